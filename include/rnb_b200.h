@@ -548,6 +548,55 @@ int rnb_b200_decoder_prefill(rnb_b200_decoder *d, const uint32_t *tokens, int n,
 /* Logits of the last step or prefill (this rank's vocab slice), for tests. */
 int rnb_b200_decoder_read_logits(rnb_b200_decoder *d, float *out, size_t n);
 
+/* ---- mixed stacks: a decoder whose layers are listed one by one --------------------------------
+ * Each layer names its mixer (token mixing) and may have a dense gated feed-forward
+ * W_down(gelu_tanh(W_gate h) * W_up h).  Sublayers are normed on both sides,
+ * x <- x + residual_mult * norm_b(sublayer(norm_a(x))), norms are x / sqrt(mean x^2 + eps) * (1 + w),
+ * and the LM head is the embedding table.  Layers loop_start .. loop_stop - 1 run loop_times times in
+ * a row, each pass with its own state; the embedding output is added to x before every pass but the
+ * first.  Weights are bf16 matrices; the residual, norms, rotations, attention weights and recurrent
+ * states are f32.  f32_math: activations and all matrix products in f32 too (no tensor cores).
+ * The functions of the decoder above work on it: step, step_dev, prefill, read_logits, time_steps, ... */
+#define RNB_B200_MIXER_WKV 1              /* RWKV-style time mixing: heads x dim, low-rank decay */
+#define RNB_B200_MIXER_RETENTION 2        /* heads x dim keys, heads x vdim values, decay per head */
+#define RNB_B200_MIXER_LATENT_ATTENTION 3 /* latent of kv_rank plus a shared rotated key part of rot_dim */
+typedef struct {
+    int32_t dims;        /* rotated dimensions of a head's vector (0: none) */
+    int32_t interleaved; /* pairs (2i, 2i + 1); otherwise (i, i + dims / 2) */
+    double base;
+    int32_t scaled;      /* YaRN: the four values below apply */
+    double factor, original, fast, slow;
+} rnb_b200_rotation;
+typedef struct {
+    int32_t mixer;
+    int32_t heads, dim, vdim, rot_dim, kv_rank;
+    int32_t decay_rank;  /* time mixing: rows of the low-rank decay matrix (0: as the tensor has) */
+    float scale;         /* latent attention: multiplies the scores */
+    rnb_b200_rotation rot;
+    const double *decay; /* retention: [heads], copied */
+    int32_t n_ff;        /* 0: no feed-forward */
+} rnb_b200_mixer_cfg;
+typedef struct {
+    int32_t n_layer, width, vocab, max_ctx;
+    int32_t loop_start, loop_stop, loop_times; /* loop_times <= 1: every layer runs once */
+    float norm_eps, residual_mult;
+    int32_t f32_math;
+} rnb_b200_stack_cfg;
+int rnb_b200_decoder_create_stack(const rnb_b200_stack_cfg *cfg, const rnb_b200_mixer_cfg *layers, rnb_b200_decoder **out);
+/* One weight by name ("embed", "final.norm", "l3.mix.q", "l0.mlp.down", ...), row-major [out, in];
+ * type: GGML id, 30 = BF16 (matrices and vectors) or 0 = F32 (vectors only). */
+int rnb_b200_decoder_set_tensor(rnb_b200_decoder *d, const char *name, uint32_t type, const void *data, const uint64_t *shape, uint32_t n_dims);
+/* Forget the sequence: the next position is 0.  A step or prefill at position 0 does this by itself. */
+int rnb_b200_decoder_reset(rnb_b200_decoder *d);
+/* Prefill as above, plus the logits at chosen places of this call's tokens: want[i] in 0..n-1,
+ * logits_out [n_want][vocab].  Any stack and any decoder on one GPU. */
+int rnb_b200_decoder_prefill_logits(rnb_b200_decoder *d, const uint32_t *tokens, int n, int pos0, const int32_t *want, int n_want,
+                                    float *logits_out, uint32_t *next_token);
+/* Mixed stacks, for tests: the next prefill calls also write the residual rows after every layer run,
+ * [runs][n][width] f32, to `out` (n must fit one internal piece); null switches it off. */
+int rnb_b200_decoder_trace_residual(rnb_b200_decoder *d, float *out);
+int rnb_b200_decoder_n_runs(rnb_b200_decoder *d, int32_t *n_runs);
+
 /* Multi-GPU exchange over peer memory (the alternative to the NCCL communicator above, which
  * measured 3-10 % faster per token on 2-8 GPUs): every rank exports the CUDA IPC handle of its exchange arena, the host side
  * all-gathers the 64-byte handles, every rank attaches the full list (rank order).  After

@@ -52,6 +52,25 @@ class GgufTensorInfo(C.Structure):
                 ("offset", C.c_uint64), ("n_elements", C.c_uint64), ("n_bytes", C.c_uint64), ("data", C.c_void_p)]
 
 
+MIXER_WKV, MIXER_RETENTION, MIXER_LATENT_ATTENTION = 1, 2, 3
+TYPE_F32, TYPE_BF16 = 0, 30
+
+
+class Rotation(C.Structure):
+    _fields_ = [("dims", C.c_int32), ("interleaved", C.c_int32), ("base", C.c_double), ("scaled", C.c_int32)] + \
+               [(n, C.c_double) for n in ("factor", "original", "fast", "slow")]
+
+
+class MixerCfg(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "dim", "vdim", "rot_dim", "kv_rank", "decay_rank")] + \
+               [("scale", C.c_float), ("rot", Rotation), ("decay", C.POINTER(C.c_double)), ("n_ff", C.c_int32)]
+
+
+class StackCfg(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("n_layer", "width", "vocab", "max_ctx", "loop_start", "loop_stop", "loop_times")] + \
+               [("norm_eps", C.c_float), ("residual_mult", C.c_float), ("f32_math", C.c_int32)]
+
+
 class LayerWeights(C.Structure):
     _fields_ = [("attn_norm", C.c_void_p), ("ffn_norm", C.c_void_p)] + \
                [(n, QWeight) for n in ("wq", "wk", "wv", "wo", "gate", "up", "down")] + \
@@ -168,6 +187,12 @@ def load() -> C.CDLL:
         "rnb_b200_nccl_unique_id": [vp],
         "rnb_b200_decoder_attach_nccl": [vp, vp],
         "rnb_b200_decoder_prefill": [vp, vp, i32, i32, vp, vp],
+        "rnb_b200_decoder_create_stack": [vp, vp, vp],
+        "rnb_b200_decoder_set_tensor": [vp, C.c_char_p, u32, vp, vp, u32],
+        "rnb_b200_decoder_reset": [vp],
+        "rnb_b200_decoder_prefill_logits": [vp, vp, i32, i32, vp, i32, vp, vp],
+        "rnb_b200_decoder_trace_residual": [vp, vp],
+        "rnb_b200_decoder_n_runs": [vp, vp],
         "rnb_b200_decoder_read_logits": [vp, vp, sz],
         "rnb_b200_decoder_exchange_handle": [vp, vp],
         "rnb_b200_decoder_attach_peers": [vp, vp],

@@ -14,11 +14,11 @@ PKG = Path(__file__).resolve().parent
 CSRC = PKG / "csrc"
 LIB = PKG / "librnb_b200.so"
 STATIC_LIB = PKG / "librnb_b200.a"
-SOURCES = ["api.cu", "noalloc.cu", "gguf.cu", "expert_cache.cu"]
+SOURCES = ["api.cu", "layer_stack.cu", "noalloc.cu", "gguf.cu", "expert_cache.cu"]
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "-Xcompiler", "-fPIC", "-Xcompiler", "-Wall", "-Xcompiler", "-Wno-unused-function",
-    "--expt-relaxed-constexpr", "-cudart", "shared",
+    "--expt-relaxed-constexpr", "-cudart", "shared", "--threads", "0",
 ]
 
 

@@ -5,6 +5,7 @@
 #include <algorithm>
 
 #include "launch.hpp"
+#include "layer_stack.hpp"
 #include "prefill.cuh"
 #include "attention_wide.cuh"
 

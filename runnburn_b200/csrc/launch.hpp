@@ -710,10 +710,10 @@ inline int launch_attention_decode(cudaStream_t s, const float *q, const uint16_
 // Tensor-core prefill matmul: converts the f32 token rows to bf16 (scratch `xb`, seq*cols
 // elements) and runs the tcgen05 kernel.  y is [seq][rows] f32.
 int prefill_gemm_setup();   // raises the kernels' dynamic shared-memory limit once
-// Descriptor of the bf16 token matrix [seq][cols] for the kernel's tiled copies: boxes of
-// 64 columns x 256 tokens, 128-byte swizzle, zeros past the last token.  The encoder is a driver
+// Descriptor of a bf16 matrix [seq][cols] (row pitch ld elements, 0: cols) for the kernels' tiled copies:
+// boxes of 64 columns x box_rows rows (256 tokens), 128-byte swizzle, zeros past either end.  The encoder is a driver
 // entry point, looked up once through the runtime.
-inline int encode_token_map(PgTensorMap *out, const uint16_t *xb, size_t seq, size_t cols) {
+inline int encode_token_map(PgTensorMap *out, const uint16_t *xb, size_t seq, size_t cols, size_t ld = 0, int box_rows = PG_BOX_ROWS) {
     static_assert(sizeof(PgTensorMap) == sizeof(CUtensorMap) && alignof(PgTensorMap) >= alignof(CUtensorMap), "descriptor size");
     typedef CUresult (*EncodeTiled)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *, const cuuint64_t *, const cuuint32_t *,
                                     const cuuint32_t *, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
@@ -726,8 +726,8 @@ inline int encode_token_map(PgTensorMap *out, const uint16_t *xb, size_t seq, si
         encode = reinterpret_cast<EncodeTiled>(fn);
     }
     const cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)seq};
-    const cuuint64_t strides[1] = {(cuuint64_t)cols * 2};
-    const cuuint32_t box[2] = {(cuuint32_t)PG_K, (cuuint32_t)PG_BOX_ROWS};
+    const cuuint64_t strides[1] = {(cuuint64_t)(ld ? ld : cols) * 2};
+    const cuuint32_t box[2] = {(cuuint32_t)PG_K, (cuuint32_t)box_rows};
     const cuuint32_t estr[2] = {1, 1};
     const CUresult r = encode(reinterpret_cast<CUtensorMap *>(out), CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<uint16_t *>(xb), dims, strides, box, estr,
                               CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);

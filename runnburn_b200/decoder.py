@@ -40,6 +40,10 @@ class ModelConfig:
             setattr(c, k, v)
         return c
 
+    def create(self, handle) -> None:
+        c = self.to_c()
+        check(load().rnb_b200_decoder_create(C.byref(c), C.byref(handle)))
+
 
 # Published shapes of the configurations the bench and tests use (random-init, synthetic).
 LLAMA3_8B = dict(n_layer=32, hidden=4096, n_head=32, n_kv_head=8, n_ff=14336, vocab=128256)
@@ -66,11 +70,12 @@ def _fp(a, keep):
 
 
 class Decoder:
-    def __init__(self, cfg: ModelConfig):
+    """`cfg`: a ModelConfig (quantised Llama / Qwen-style stack) or a StackConfig (mixed stack)."""
+
+    def __init__(self, cfg):
         self.cfg = cfg
         self._h = C.c_void_p()
-        c = cfg.to_c()
-        check(load().rnb_b200_decoder_create(C.byref(c), C.byref(self._h)))
+        cfg.create(self._h)
 
     # -- weights --
     def load_description(self, desc: dict) -> None:
@@ -87,6 +92,17 @@ class Decoder:
         keep = []
         check(load().rnb_b200_decoder_set_globals(self._h, _qw(desc["token_embd"], keep), _fp(desc["out_norm"], keep),
                                                   _qw(desc["output"], keep)))
+
+    def set_tensor(self, name: str, dtype: str, data, shape) -> None:
+        """One weight of a mixed stack; `data`: the tensor's bytes, `dtype`: "BF16" or "F32"."""
+        a = np.frombuffer(data, np.uint8)
+        dims = (C.c_uint64 * max(len(shape), 1))(*shape)
+        t = {"BF16": _lib.TYPE_BF16, "F32": _lib.TYPE_F32}.get(dtype)
+        if t is None:
+            raise ValueError(f"tensor {name!r}: dtype {dtype} is not supported (BF16, F32)")
+        if a.size != int(np.prod(shape, dtype=np.int64)) * (2 if t == _lib.TYPE_BF16 else 4):
+            raise ValueError(f"tensor {name!r}: {a.size} bytes do not fit shape {list(shape)}")
+        check(load().rnb_b200_decoder_set_tensor(self._h, name.encode(), t, a.ctypes.data_as(C.c_void_p), dims, len(shape)))
 
     def set_exact_attention_max(self, max_positions: int) -> None:
         """Contexts up to `max_positions` use the reference-order attention kernel (bit-identical to
@@ -125,8 +141,45 @@ class Decoder:
                                               C.byref(ms) if timed else None))
         return (nxt.value, ms.value) if timed else nxt.value
 
+    def prefill_logits(self, tokens, pos0: int, want):
+        """Like prefill, and returns (logits [len(want), vocab] at the places `want` of `tokens`, next token)."""
+        t = np.ascontiguousarray(np.asarray(tokens, dtype=np.uint32))
+        w = np.ascontiguousarray(np.asarray(want, dtype=np.int32))
+        out = np.empty((w.size, self.cfg.vocab), np.float32)
+        nxt = C.c_uint32()
+        check(load().rnb_b200_decoder_prefill_logits(self._h, t.ctypes.data_as(C.c_void_p), int(t.size), int(pos0), w.ctypes.data_as(C.c_void_p), int(w.size),
+                                                     out.ctypes.data_as(C.c_void_p), C.byref(nxt)))
+        return out, nxt.value
+
+    def reset(self) -> None:
+        """Forget the sequence (recurrent states to zero); the next position is 0."""
+        check(load().rnb_b200_decoder_reset(self._h))
+
+    def generate(self, prompt, n: int, stop: int | None = None) -> list:
+        """Greedy continuation: the prompt through prefill from position 0, then up to `n` tokens step by step."""
+        if n < 1:
+            return []
+        out = [self.prefill(prompt, 0)]
+        pos = len(prompt)
+        while len(out) < n and out[-1] != stop and pos < self.cfg.max_ctx:
+            out.append(self.step(out[-1], pos))
+            pos += 1
+        return out
+
+    def trace_residual(self, tokens, pos0: int = 0) -> np.ndarray:
+        """Mixed stacks: prefills `tokens` and returns the residual rows after every layer run, [runs, n, width]."""
+        runs = C.c_int32()
+        check(load().rnb_b200_decoder_n_runs(self._h, C.byref(runs)))
+        out = np.empty((runs.value, len(tokens), self.cfg.width), np.float32)
+        check(load().rnb_b200_decoder_trace_residual(self._h, out.ctypes.data_as(C.c_void_p)))
+        try:
+            self.prefill(tokens, pos0)
+        finally:
+            check(load().rnb_b200_decoder_trace_residual(self._h, None))
+        return out
+
     def read_logits(self) -> np.ndarray:
-        out = np.empty(self.cfg.vocab // self.cfg.world_size, np.float32)
+        out = np.empty(self.cfg.vocab // getattr(self.cfg, "world_size", 1), np.float32)
         check(load().rnb_b200_decoder_read_logits(self._h, out.ctypes.data_as(C.c_void_p), out.size))
         return out
 
