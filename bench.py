@@ -41,6 +41,30 @@ WORKLOADS = {
                                                n_ff_expert=768, rope_neox=1), 8192),
     "tiny-llama-ctx256": (dict(n_layer=2, hidden=512, n_head=4, n_kv_head=2, n_ff=1024, vocab=2048), 256),
 }
+
+
+def punisun_shape(n_layer: int, width: int, n_ff: int, vocab: int, loop=(0, 0, 1)) -> dict:
+    """A mixed stack (Punisun design) of the widths of a common dense model, in bf16: every group of four
+    layers is time mixing (64-wide heads), retention (128-wide heads), time mixing, latent attention
+    (128 + 64 query dimensions, latent of 512)."""
+    h64, h128 = width // 64, width // 128
+    wkv = dict(mixer="wkv", heads=h64, dim=64, decay_rank=64, n_ff=n_ff)
+    ret = dict(mixer="retention", heads=h128, dim=128, vdim=128, rot=dict(dims=128, base=1e6),
+               decay=[1.0 - 2.0 ** (-5.0 - 7.0 * i / max(h128 - 1, 1)) for i in range(h128)], n_ff=n_ff)
+    lat = dict(mixer="latent_attention", heads=h128, dim=128, vdim=128, rot_dim=64, kv_rank=512, scale=192 ** -0.5,
+               rot=dict(dims=64, base=5e4, scaling=dict(factor=8.0, original=4096.0, fast=32.0, slow=1.0)), n_ff=n_ff)
+    return dict(stack=[(wkv, ret, wkv, lat)[i % 4] for i in range(n_layer)], n_layer=n_layer, hidden=width, vocab=vocab, loop=loop)
+
+
+WORKLOADS.update({
+    # the layer widths of the 8B shape above; two layers run twice
+    "punisun-8b-ctx4096": (punisun_shape(32, 4096, 14336, 128256, (0, 2, 2)), 4096),
+    "punisun-1b-ctx4096": (punisun_shape(16, 2048, 8192, 128256, (0, 2, 2)), 4096),
+    # one group of four layers of the 8B widths: the capture-sized case for ncu
+    "punisun-4layers-ctx4096": (punisun_shape(4, 4096, 14336, 32768), 4096),
+    # the 1B widths of the closest other model, for the comparison at equal size
+    "llama3-1b-q4km-ctx4096": (dict(n_layer=16, hidden=2048, n_head=16, n_kv_head=8, n_ff=8192, vocab=128256), 4096),
+})
 DRAM_TRAFFIC_OVER_ALGORITHMIC = 459.77 / 456.19   # ncu, gemv_mma_kernel_1: LM head + q/k/v + o launches (profiles/gemv_mma_kernel_llama3-8b-2layers-ctx4096.md)
 REPEATS = 5
 METRIC = "decode_tok_per_s_batch1"
@@ -57,7 +81,28 @@ def q8k_bytes(cols: int) -> int:
 
 def algorithmic_bytes_per_token(shape: dict, ctx: int) -> dict:
     """Bytes one decode token must move (Q4_K_M convention: attn_v, ffn_down, LM head in
-    Q6_K): weights once, the visible KV rows once, activations (Q8_K in, f32 out)."""
+    Q6_K): weights once, the visible KV rows once, activations (Q8_K in, f32 out).  Mixed stacks:
+    bf16 weights, the recurrent states read and written, the visible latent rows; once per layer run."""
+    if "stack" in shape:
+        a, b, times = shape["loop"]
+        runs = list(range(a)) + list(range(a, b)) * times + list(range(b, len(shape["stack"])))
+        H, w, state, act = shape["hidden"], shape["vocab"] * shape["hidden"] * 2, 0, shape["vocab"] * 4
+        for i in runs:
+            m = shape["stack"][i]
+            hd, hv = m["heads"] * m["dim"], m["heads"] * m.get("vdim", m["dim"])
+            if m["mixer"] == "latent_attention":
+                row = m["kv_rank"] + m["rot_dim"]
+                mats = [(m["heads"] * (m["dim"] + m["rot_dim"]), H), (row, H), (hd, m["kv_rank"]), (hv, m["kv_rank"]), (H, hv)]
+                state += (ctx + 1) * row * 2
+            else:
+                mats = [(hd, H), (hd, H), (hv, H), (hv, H), (H, hv)]
+                if m["mixer"] == "wkv":
+                    mats += [(m["decay_rank"], H), (hd, m["decay_rank"])]
+                state += 2 * hd * m.get("vdim", m["dim"]) * 4
+            mats += [(m["n_ff"], H), (m["n_ff"], H), (H, m["n_ff"])]
+            w += sum(r * c for r, c in mats) * 2
+            act += sum(r + c for r, c in mats) * 4
+        return {"weights": w, "kv": state, "activations": act, "total": w + state + act}
     H, qd, kvd, ff, V, L = shape["hidden"], shape["n_head"] * 128, shape["n_kv_head"] * 128, shape["n_ff"], shape["vocab"], shape["n_layer"]
     if shape.get("n_expert", 0):
         # attention in Q6_K, f32 router, the k routed experts' gate/up/down in Q4_K
@@ -426,7 +471,15 @@ def run_gpu(args, shape, ctx, name, rank, world, local_rank):
     K, W = args.steps, args.warmup
     R = REPEATS                                   # the timed region runs R times; the median is reported
     max_ctx = ctx + (R + 1) * K + 2 * max(W, 3) + 8
-    cfg = r.ModelConfig(max_ctx=max_ctx, world_size=world, rank=rank, **shape)
+    stack = "stack" in shape
+    if stack:
+        if world > 1:
+            raise SystemExit("mixed stacks run on one GPU")
+        from runnburn_b200.stack import MixerLayer
+        cfg = r.StackConfig(width=shape["hidden"], vocab=shape["vocab"], layers=[MixerLayer(**m) for m in shape["stack"]], norm_eps=1e-6,
+                            residual_mult=0.5, loop=shape["loop"], max_ctx=max_ctx)
+    else:
+        cfg = r.ModelConfig(max_ctx=max_ctx, world_size=world, rank=rank, **shape)
     dec = r.Decoder(cfg)
     # "peer": producers store their slices into the peers' buffers (measured: 11.3 against 12.1 ms per token at 4 GPUs);
     # "nccl": ncclAllGather (13.0 against 13.8 ms at 2 GPUs, where one peer makes the gather a single copy)
@@ -545,8 +598,8 @@ def run_gpu(args, shape, ctx, name, rank, world, local_rank):
         "metric": METRIC, "value": value, "unit": UNIT, "n_gpus": world, "steps": K, "warmup": max(W, 3),
         "ms_per_step": ms / K, "repeats": R, "ms_per_step_all": [m / K for m in all_ms], "timing": "median of %d timed regions of %d steps each, max over ranks per region" % (R, K),
         "higher_is_better": True, "scaling": "strong" if world > 1 else "weak",
-        "vs_baseline": None, "dtype": "int8xint4->int32, f32 accumulate", "data": "synthetic",
-        "config": {"workload": name, "context": ctx, "kv_cache": "f16", "weights": ("random-init N(0,0.02): attention and LM head Q6_K, f32 router, experts Q4_K, generated on device" if shape.get("n_expert", 0) else "random-init N(0,0.02), Q4_K_M layout (attn_v/ffn_down/output Q6_K), generated on device"),
+        "vs_baseline": None, "dtype": "bf16 weights, f32 activations and accumulate" if stack else "int8xint4->int32, f32 accumulate", "data": "synthetic",
+        "config": {"workload": name, "context": ctx, "kv_cache": "bf16 latent rows, f32 recurrent states" if stack else "f16", "weights": "random-init N(0,0.02), bf16, generated on device" if stack else ("random-init N(0,0.02): attention and LM head Q6_K, f32 router, experts Q4_K, generated on device" if shape.get("n_expert", 0) else "random-init N(0,0.02), Q4_K_M layout (attn_v/ffn_down/output Q6_K), generated on device"),
                    "parallelism": (f"row-sharded x{world}, all-gather by " + ("ncclAllGather" if transport == "nccl" else "peer-memory stores over NVLink from the producing kernels' epilogues, consumers wait on arrival flags (no exchange launch)")) if world > 1 else "single GPU",
                    "l2": "each step streams its whole weight set and KV cache (GBs), far more than the 126 MB L2: no flush needed",
                    "algorithmic_bytes_per_token": alg},
@@ -565,7 +618,11 @@ def run_gpu(args, shape, ctx, name, rank, world, local_rank):
         per_launch_bytes = mv["bytes_per_iter"] / mv["launches_per_iter"]
         per_launch_s = mv["ms"] / 1000.0 / (mv["iters"] * mv["launches_per_iter"])
         ach = per_launch_bytes / per_launch_s / 1e9
-        out["roofline"] = {"kernel": "gemv_mma_kernel_1 (q/k/v, o, down, LM head: integer tensor-core matvec) and gemv_pair_q4k_kernel (gate/up)", "bound": "hbm", "achieved": ach, "peak": peaks["hbm_gbs"], "unit": "GB/s",
+        out["roofline"] = {"kernel": "dense_gemv_kernel (every projection and the LM head)", "bound": "hbm", "achieved": ach, "peak": peaks["hbm_gbs"], "unit": "GB/s",
+                           "frac": ach / peaks["hbm_gbs"], "peak_source": peaks["source"], "launches_per_step": mv["launches_per_iter"],
+                           "algorithmic_bytes_per_launch": per_launch_bytes, "avg_launch_us": per_launch_s * 1e6,
+                           "how": "CUDA events around all matvec launches of a step on the decoder stream, model's own weights"} if stack else {
+                           "kernel": "gemv_mma_kernel_1 (q/k/v, o, down, LM head: integer tensor-core matvec) and gemv_pair_q4k_kernel (gate/up)", "bound": "hbm", "achieved": ach, "peak": peaks["hbm_gbs"], "unit": "GB/s",
                            "frac": ach / peaks["hbm_gbs"], "frac_of_8TBs_nominal": ach / 8000.0, "peak_source": peaks["source"],
                            # DRAM read+write bytes per launch: the ncu capture of three matvec launches (LM head, q/k/v, o)
                            # gave 459.8 MB of traffic for 456.2 MB of algorithmic bytes (summary under profiles/)
@@ -583,7 +640,8 @@ def run_gpu(args, shape, ctx, name, rank, world, local_rank):
             dec.prefill(ids, 0, timed=True)
             _, pms = dec.prefill(ids, 0, timed=True)
             out["prefill"] = {"tokens": int(n_tok), "ms": pms, "tok_per_s": n_tok / (pms / 1000.0),
-                              "what": "embed, 32 x (RMSNorm, q/k/v matmul, RoPE + f16 KV append, causal attention, o_proj, RMSNorm, gate/up, SiLU*up, down), "
+                              "what": "embed, layers (projections and feed-forward on tcgen05 in bf16, chunked recurrences in f32, causal latent attention on mma.sync), "
+                                      "final norm + LM head + argmax of the last token" if stack else "embed, 32 x (RMSNorm, q/k/v matmul, RoPE + f16 KV append, causal attention, o_proj, RMSNorm, gate/up, SiLU*up, down), "
                                       "final norm + LM head + argmax of the last token; matmuls on tcgen05 (bf16), causal attention on mma.sync tensor cores (split-f16 operands, fp32 accumulate)"}
         except Exception as e:   # a secondary figure must not lose the headline line
             out["prefill"] = {"error": str(e)[:200]}
@@ -613,6 +671,9 @@ def main():
         args.gpus = world
     name = args.workload or ("llama3-8b-q4km-ctx4096" if args.gpus == 1 else "llama3-70b-q4km-ctx32768")
     shape, ctx = WORKLOADS[name]
+    if args.impl == "reference" and "stack" in shape:
+        print(json.dumps({"impl": "reference", "unavailable": "the reference has no model of this design"}), flush=True)
+        return
     if args.impl == "reference":
         out = run_reference(args, shape, ctx, name, rank, world)
         if out is not None:
@@ -624,12 +685,12 @@ def main():
     out = run_gpu(args, shape, ctx, name, rank, world, local_rank)
     if out is None:
         return
-    if world == 1 and shape.get("hidden") == 4096 and not args.no_prefill:
+    if world == 1 and shape.get("hidden") == 4096 and "stack" not in shape and not args.no_prefill:
         try:
             out["prefill_gemm"] = prefill_gemm_bench(shape, 2048)
         except Exception as e:   # a secondary figure must not lose the headline line
             out["prefill_gemm"] = {"error": str(e)[:200]}
-    if world == 1 and "roofline" in out and not args.no_per_shape:
+    if world == 1 and "roofline" in out and "stack" not in shape and not args.no_per_shape:
         # the layer's and the LM head's matvec shapes each timed alone
         try:
             ps = matvec_shape_bench([(12, 4096, 4096), (12, 14336, 4096), (12, 4096, 14336), (14, 1024, 4096), (14, 4096, 14336), (14, 128256, 4096)]
@@ -646,7 +707,7 @@ def main():
             out["moe"] = moe_decode_bench(args)
         except Exception as e:
             out["moe"] = {"error": str(e)[:200]}
-    if world == 1 and not args.no_cpu_baseline:
+    if world == 1 and "stack" not in shape and not args.no_cpu_baseline:
         s, layer, head = cpu_baseline(shape, ctx, reps=5, warmup=1, min_seconds=10.0)   # about 10 s of CPU work
         out["cpu_baseline"] = {"value": s.tok_per_s(min(layer), min(head)), "unit": UNIT, "cores": s.threads, "kind": "port",
                                "sample": s.describe() + "; %d repetitions, %.1f s of CPU time, best repetition used" % (len(layer), sum(layer))}
