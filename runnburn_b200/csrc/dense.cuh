@@ -45,11 +45,11 @@ struct DenseVecJob {
 };
 struct DenseVecJobs {
     DenseVecJob j[DENSE_MAX_JOBS];
-    int n;
+    int n, ksplit;   // ksplit (1, 2, 4): warps that share a pair of rows, each taking every ksplit-th 1024 columns
 };
 constexpr int DV_WARPS = 4, DV_UNROLL = 4;
 
-// A warp owns two output rows (or the gate and the up row of one output).  T = tokens, 1 .. 8.
+// ksplit warps own two output rows (or the gate and the up row of one output).  T = tokens, 1 .. 8.
 template <int T>
 RNB_GLOBAL void __launch_bounds__(DV_WARPS * 32)
 dense_gemv_kernel(const __grid_constant__ DenseVecJobs jobs) {
@@ -59,7 +59,9 @@ dense_gemv_kernel(const __grid_constant__ DenseVecJobs jobs) {
         if ((int)blockIdx.x >= jobs.j[i].cta0) js = i;
     const DenseVecJob &job = jobs.j[js];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int unit = ((int)blockIdx.x - job.cta0) * DV_WARPS + warp;
+    const int ks = jobs.ksplit, part = warp & (ks - 1);
+    const int unit = ((int)blockIdx.x - job.cta0) * (DV_WARPS / ks) + warp / ks;
+    __shared__ float s_part[DV_WARPS][2][T];
     const bool pair = job.w2 != nullptr;
     const int r0 = pair ? unit : 2 * unit, rows = job.rows, cols = job.cols;
     const bool live = r0 < rows, two = pair || r0 + 1 < rows;
@@ -79,13 +81,14 @@ dense_gemv_kernel(const __grid_constant__ DenseVecJobs jobs) {
                 b1[u] = k < cols ? ldg_nc_u4(w1 + k) : z4;
             }
         };
-        fetch(0);        // weights do not depend on the previous launch
+        const int step = 256 * DV_UNROLL * ks;
+        fetch(part * 256 * DV_UNROLL);        // weights do not depend on the previous launch
         pdl_wait();
-        for (int k0 = 0; k0 < cols; k0 += 256 * DV_UNROLL) {
+        for (int k0 = part * 256 * DV_UNROLL; k0 < cols; k0 += step) {
             uint4 c0[DV_UNROLL], c1[DV_UNROLL];
 #pragma unroll
             for (int u = 0; u < DV_UNROLL; u++) c0[u] = b0[u], c1[u] = b1[u];
-            if (k0 + 256 * DV_UNROLL < cols) fetch(k0 + 256 * DV_UNROLL);
+            if (k0 + step < cols) fetch(k0 + step);
 #pragma unroll
             for (int u = 0; u < DV_UNROLL; u++) {
                 const int k = k0 + u * 256 + lane * 8;
@@ -108,7 +111,7 @@ dense_gemv_kernel(const __grid_constant__ DenseVecJobs jobs) {
         }
     } else {
         pdl_wait();
-        for (int k = lane; k < cols; k += 32) {
+        for (int k = part * 32 + lane; k < cols; k += 32 * ks) {
             const float p = to_f32(w0[k]), q = to_f32(w1[k]);
 #pragma unroll
             for (int t = 0; t < T; t++) {
@@ -120,7 +123,17 @@ dense_gemv_kernel(const __grid_constant__ DenseVecJobs jobs) {
     }
 #pragma unroll
     for (int t = 0; t < T; t++) a0[t] = warp_sum(a0[t]), a1[t] = warp_sum(a1[t]);
-    if (lane == 0 && live) {
+    if (ks > 1) {
+        if (lane == 0)
+#pragma unroll
+            for (int t = 0; t < T; t++) s_part[warp][0][t] = a0[t], s_part[warp][1][t] = a1[t];
+        __syncthreads();
+        if (lane == 0 && part == 0)
+            for (int w = 1; w < ks; w++)
+#pragma unroll
+                for (int t = 0; t < T; t++) a0[t] += s_part[warp + w][0][t], a1[t] += s_part[warp + w][1][t];
+    }
+    if (lane == 0 && live && part == 0) {
 #pragma unroll
         for (int t = 0; t < T; t++) {
             float *y = job.y + (size_t)t * rows + r0;
@@ -148,6 +161,7 @@ constexpr size_t DG_SMEM = (size_t)DG_STAGES * DG_STAGE_BYTES + 1024;
 
 struct DenseGemmJob {
     void *y;             // [seq][ld]
+    const float *decay_bias;   // not null: y = exp(-exp(w x + bias[row]))
     int rows, cols, tile0, out_bf16, pair, ld;
 };
 struct DenseGemmJobs {
@@ -274,6 +288,11 @@ dense_gemm_kernel(const __grid_constant__ DenseGemmJobs jobs, const __grid_const
                 uint32_t v[32];
                 pg_tmem_ld32(tmem + ((uint32_t)(q * 32) << 16) + (uint32_t)(cc * 32), v);
                 if (row < rows) {
+                    if (job.decay_bias) {
+                        const float b = job.decay_bias[row];
+#pragma unroll
+                        for (int i = 0; i < 32; i++) v[i] = __float_as_uint(expf(-expf(__uint_as_float(v[i]) + b)));
+                    }
 #pragma unroll
                     for (int i = 0; i < 32; i++) {
                         const int tok = m0 + cc * 32 + i;

@@ -9,6 +9,7 @@
 // attention on tensor cores.
 #pragma once
 #include "layer_glue.cuh"
+#include "mma_bf16.cuh"
 
 namespace rnb {
 
@@ -38,8 +39,10 @@ latent_append_kernel(const float *__restrict__ y, const float *__restrict__ w, f
     latent_append_row<CT>(y + (size_t)blockIdx.x * (d.rank + d.rot_dim), w, eps, d, rot, *pos0 + (int)blockIdx.x, cache, red);
 }
 
-// grid = (heads + 1, tokens, ceil(rank / 256)), 128 threads.  Head h: qf[t][h] = [W_uk_h^T q | rotated q];
-// the extra column of CTAs appends the token's cache row.  Dynamic shared memory: dim floats.
+// grid = (heads + 1, tokens, ceil(rank / 512)), 512 threads.  Head h: qf[t][h] = [W_uk_h^T q | rotated q];
+// the extra column of CTAs appends the token's cache row.  64 threads hold 8 columns each, 8 groups of them
+// share the key dimensions; the first rows of W_uk are loaded ahead of the dependency wait.
+// Dynamic shared memory: dim + 8 * 512 floats.
 struct LatentPrepareArgs {
     const float *q, *y, *w;      // [tokens][heads * (dim + rot)], [tokens][rank + rot], [rank]
     const bf16 *uk;              // [heads * dim][rank]
@@ -50,47 +53,74 @@ struct LatentPrepareArgs {
     LatentDims d;
     Rotation rot;
 };
+constexpr int LP_THREADS = 512, LP_COLS = 512, LP_BATCH = 8;
 template <class CT>
-RNB_GLOBAL void __launch_bounds__(128)
+RNB_GLOBAL void __launch_bounds__(LP_THREADS)
 latent_prepare_kernel(const __grid_constant__ LatentPrepareArgs a) {
-    extern __shared__ __align__(16) float lp_q[];
+    extern __shared__ __align__(16) float lp_smem[];
     __shared__ float red[32];
     pdl_launch_dependents();
-    pdl_wait();
     const LatentDims &d = a.d;
-    const int h = blockIdx.x, t = blockIdx.y, pos = *a.pos0 + t, E = d.rank + d.rot_dim;
+    const int h = blockIdx.x, t = blockIdx.y, E = d.rank + d.rot_dim, tid = threadIdx.x;
     if (h == d.heads) {
+        pdl_wait();
         if (blockIdx.z == 0)
-            latent_append_row<CT>(a.y + (size_t)t * E, a.w, a.eps, d, a.rot, pos, reinterpret_cast<CT *>(a.cache), red);
+            latent_append_row<CT>(a.y + (size_t)t * E, a.w, a.eps, d, a.rot, *a.pos0 + t, reinterpret_cast<CT *>(a.cache), red);
         return;
     }
+    float *sq = lp_smem, *sr = lp_smem + ((d.dim + 3) & ~3);
+    const int grp = tid >> 6, c = blockIdx.z * LP_COLS + (tid & 63) * 8;
+    const bool vec = d.rank % 8 == 0, in = c < d.rank;
+    const bf16 *w = a.uk + (size_t)h * d.dim * d.rank + c;
+    uint4 b[LP_BATCH];
+    auto fetch = [&](int i0) {
+#pragma unroll
+        for (int k = 0; k < LP_BATCH; k++) {
+            const int i = i0 + 8 * k + grp;
+            b[k] = vec && in && i < d.dim ? ldg_nc_u4(w + (size_t)i * d.rank) : make_uint4(0u, 0u, 0u, 0u);
+        }
+    };
+    fetch(0);
+    pdl_wait();
     const float *q = a.q + ((size_t)t * d.heads + h) * (d.dim + d.rot_dim);
     float *out = a.qf + ((size_t)t * d.heads + h) * E;
-    for (int i = threadIdx.x; i < d.dim; i += 128) lp_q[i] = q[i];
+    for (int i = tid; i < d.dim; i += LP_THREADS) sq[i] = q[i];
     if (blockIdx.z == 0)
-        for (int i = threadIdx.x; i < d.rot_dim; i += 128) out[d.rank + i] = rotated_element(a.rot, pos, i, [&](int e) { return q[d.dim + e]; });
+        for (int i = tid; i < d.rot_dim; i += LP_THREADS) out[d.rank + i] = rotated_element(a.rot, *a.pos0 + t, i, [&](int e) { return q[d.dim + e]; });
     __syncthreads();
-    const int c = blockIdx.z * 256 + 2 * threadIdx.x;
-    if (c >= d.rank) return;
-    const bf16 *w = a.uk + (size_t)h * d.dim * d.rank + c;
-    float s0 = 0.f, s1 = 0.f;
-    if (d.rank % 2 == 0) {
-#pragma unroll 8
-        for (int i = 0; i < d.dim; i++) {
-            const uint32_t p = __ldg(reinterpret_cast<const uint32_t *>(w + (size_t)i * d.rank));
-            s0 = fmaf(bf16_lo(p), lp_q[i], s0);
-            s1 = fmaf(bf16_hi(p), lp_q[i], s1);
+    if (!vec) {
+        for (int e = blockIdx.z * LP_COLS + tid; e < min(d.rank, (int)(blockIdx.z + 1) * LP_COLS); e += LP_THREADS) {
+            const bf16 *col = a.uk + (size_t)h * d.dim * d.rank + e;
+            float s = 0.f;
+            for (int i = 0; i < d.dim; i++) s = fmaf(to_f32(col[(size_t)i * d.rank]), sq[i], s);
+            out[e] = s;
         }
-        out[c] = s0;
-        out[c + 1] = s1;
-    } else {
-        const bool two = c + 1 < d.rank;
-        for (int i = 0; i < d.dim; i++) {
-            s0 = fmaf(to_f32(w[(size_t)i * d.rank]), lp_q[i], s0);
-            if (two) s1 = fmaf(to_f32(w[(size_t)i * d.rank + 1]), lp_q[i], s1);
+        return;
+    }
+    float acc[8] = {};
+    for (int i0 = 0; i0 < d.dim; i0 += 8 * LP_BATCH) {
+        if (i0) fetch(i0);
+#pragma unroll
+        for (int k = 0; k < LP_BATCH; k++) {
+            const int i = i0 + 8 * k + grp;
+            const float qv = i < d.dim ? sq[i] : 0.f;
+            const uint32_t p[4] = {b[k].x, b[k].y, b[k].z, b[k].w};
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                acc[2 * e] = fmaf(bf16_lo(p[e]), qv, acc[2 * e]);
+                acc[2 * e + 1] = fmaf(bf16_hi(p[e]), qv, acc[2 * e + 1]);
+            }
         }
-        out[c] = s0;
-        if (two) out[c + 1] = s1;
+    }
+#pragma unroll
+    for (int e = 0; e < 8; e++) sr[grp * LP_COLS + (tid & 63) * 8 + e] = acc[e];
+    __syncthreads();
+    const int e = blockIdx.z * LP_COLS + tid;
+    if (e < d.rank) {
+        float s = 0.f;
+#pragma unroll
+        for (int k = 0; k < 8; k++) s += sr[k * LP_COLS + tid];
+        out[e] = s;
     }
 }
 
@@ -101,9 +131,11 @@ __device__ __forceinline__ void latent_chunk_range(int n, int chunks, int c, int
     hi = min(lo + per, n);
 }
 
+__host__ __device__ __forceinline__ int latent_part_ld(int rank) { return ((rank + 3) & ~3) + 4; }
+
 // Absorbed attention over one chunk of the cache on the CUDA cores.  grid = (chunks, heads, tokens), 128
-// threads; a warp takes every fourth key, lane l elements l + 32 q of a row.  part[t][h][chunk] holds the
-// unnormalised latent sum (rank), the maximum and the sum of the weights.
+// threads; a warp takes every fourth key, lane l elements l + 32 q of a row.  part[t][h][chunk] (latent_part_ld
+// floats) holds the unnormalised latent sum (rank), the maximum and the sum of the weights.
 template <class CT, int NQ>
 RNB_GLOBAL void __launch_bounds__(128)
 latent_attend_kernel(const float *__restrict__ qf, const CT *__restrict__ cache, const LatentDims d, float scale, const int *__restrict__ pos0,
@@ -149,55 +181,65 @@ latent_attend_kernel(const float *__restrict__ qf, const CT *__restrict__ cache,
         f[w] = s_m[w] == -INFINITY ? 0.f : expf(s_m[w] - M);
         L = fmaf(f[w], s_l[w], L);
     }
-    float *out = part + (((size_t)t * d.heads + h) * gridDim.x + blockIdx.x) * (d.rank + 2);
+    float *out = part + (((size_t)t * d.heads + h) * gridDim.x + blockIdx.x) * latent_part_ld(d.rank);
     for (int e = threadIdx.x; e < d.rank; e += 128) out[e] = f[0] * s_o[0][e] + f[1] * s_o[1][e] + f[2] * s_o[2][e] + f[3] * s_o[3][e];
     if (threadIdx.x == 0) out[d.rank] = M, out[d.rank + 1] = L;
 }
 
-// act[t][h * vdim + v] = W_uv_h (merged latent result).  grid = (heads, tokens, row blocks), 128 threads;
-// dynamic shared memory rank + chunks floats.
+// act[t][h * vdim + v] = W_uv_h (merged latent result).  grid = (heads, tokens, row blocks), 512 threads: four
+// groups of 128 share the chunks, 16 warps share the rows.  Dynamic shared memory 5 * rank4 + chunks floats.
+constexpr int LO_THREADS = 512;
 template <class HT>
-RNB_GLOBAL void __launch_bounds__(128)
+RNB_GLOBAL void __launch_bounds__(LO_THREADS)
 latent_output_kernel(const float *__restrict__ part, const bf16 *__restrict__ uv, const LatentDims d, int chunks, int rows_per_cta, HT *__restrict__ act) {
     extern __shared__ __align__(16) float lo_smem[];
     __shared__ float s_inv;
     pdl_launch_dependents();
+    const int h = blockIdx.x, t = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, R4 = (d.rank + 3) & ~3, ld = latent_part_ld(d.rank);
+    const int v0 = blockIdx.z * rows_per_cta, v1 = min(v0 + rows_per_cta, d.vdim);
+    if (gridDim.y == 1) prefetch_l2(uv + ((size_t)h * d.vdim + v0) * d.rank, (size_t)(v1 - v0) * d.rank * 2, threadIdx.x, LO_THREADS);
     pdl_wait();
-    float *ol = lo_smem, *f = lo_smem + d.rank;
-    const int h = blockIdx.x, t = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const float *p = part + ((size_t)t * d.heads + h) * chunks * (d.rank + 2);
+    float *ol = lo_smem, *grp = lo_smem + R4, *f = grp + 4 * R4;
+    const float *p = part + ((size_t)t * d.heads + h) * chunks * ld;
     if (warp == 0) {
         float M = -INFINITY, L = 0.f;
-        for (int c = lane; c < chunks; c += 32) M = fmaxf(M, p[(size_t)c * (d.rank + 2) + d.rank]);
+        for (int c = lane; c < chunks; c += 32) M = fmaxf(M, p[(size_t)c * ld + d.rank]);
         M = warp_max(M);
         for (int c = lane; c < chunks; c += 32) {
-            const float m = p[(size_t)c * (d.rank + 2) + d.rank], e = m == -INFINITY ? 0.f : expf(m - M);
+            const float m = p[(size_t)c * ld + d.rank], e = m == -INFINITY ? 0.f : expf(m - M);
             f[c] = e;
-            L = fmaf(e, p[(size_t)c * (d.rank + 2) + d.rank + 1], L);
+            L = fmaf(e, p[(size_t)c * ld + d.rank + 1], L);
         }
         L = warp_sum(L);
         if (lane == 0) s_inv = 1.0f / L;
     }
     __syncthreads();
-    for (int e = threadIdx.x; e < d.rank; e += 128) {
-        float s = 0.f;
-#pragma unroll 4
-        for (int c = 0; c < chunks; c++) s = fmaf(f[c], p[(size_t)c * (d.rank + 2) + e], s);
-        ol[e] = s * s_inv;
+    const int q = threadIdx.x >> 7;
+    for (int e = (threadIdx.x & 127) * 4; e < R4; e += 512) {
+        float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+        for (int c = q; c < chunks; c += 4) {
+            const float4 x = *reinterpret_cast<const float4 *>(p + (size_t)c * ld + e);
+            const float w = f[c];
+            if (w != 0.f) s.x = fmaf(w, x.x, s.x), s.y = fmaf(w, x.y, s.y), s.z = fmaf(w, x.z, s.z), s.w = fmaf(w, x.w, s.w);
+        }
+        *reinterpret_cast<float4 *>(grp + q * R4 + e) = s;
     }
     __syncthreads();
-    const int v0 = blockIdx.z * rows_per_cta, v1 = min(v0 + rows_per_cta, d.vdim);
-    for (int v = v0 + warp; v < v1; v += 4) {
+    for (int e = threadIdx.x; e < d.rank; e += LO_THREADS) ol[e] = (grp[e] + grp[R4 + e] + grp[2 * R4 + e] + grp[3 * R4 + e]) * s_inv;
+    __syncthreads();
+    for (int v = v0 + warp; v < v1; v += LO_THREADS / 32) {
         const bf16 *w = uv + ((size_t)h * d.vdim + v) * d.rank;
         float s = 0.f;
         if (d.rank % 8 == 0) {
+#pragma unroll 2
             for (int e = lane * 8; e < d.rank; e += 256) {
                 const uint4 b = ldg_nc_u4(w + e);
-                const uint32_t q[4] = {b.x, b.y, b.z, b.w};
+                const uint32_t x[4] = {b.x, b.y, b.z, b.w};
 #pragma unroll
                 for (int i = 0; i < 4; i++) {
-                    s = fmaf(bf16_lo(q[i]), ol[e + 2 * i], s);
-                    s = fmaf(bf16_hi(q[i]), ol[e + 2 * i + 1], s);
+                    s = fmaf(bf16_lo(x[i]), ol[e + 2 * i], s);
+                    s = fmaf(bf16_hi(x[i]), ol[e + 2 * i + 1], s);
                 }
             }
         } else {
@@ -208,24 +250,161 @@ latent_output_kernel(const float *__restrict__ part, const bf16 *__restrict__ uv
     }
 }
 
-// ---- prompts: causal attention over expanded keys and values on tensor cores ---------------------
-__device__ __forceinline__ void la_ldmatrix_x4(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+// ---- the same over a bf16 cache on tensor cores ---------------------------------------------------
+// The 16 rows of the products are 16 heads (they share every cache row).  Tiles of 64 keys, two stages;
+// 8 warps: scores of 8 keys each, then 1/8 of the latent columns each (8 NT per warp).  The query enters in
+// bf16, the weights as bf16 hi + lo parts.  grid = (chunks, ceil(heads / 16), tokens); rank and cache rows
+// multiples of 8.
+constexpr int LM_KEYS = 64, LM_THREADS = 256;
+struct LatentMmaSmem {
+    uint32_t pitch, q, s, phi, plo, stat, bytes;
+};
+__host__ __device__ inline LatentMmaSmem latent_mma_smem(const LatentDims &d) {
+    LatentMmaSmem L;
+    const uint32_t ep = (uint32_t)((d.rank + d.rot_dim + 31) & ~31);   // two k-steps per B load
+    L.pitch = (ep + 8) * 2;
+    L.q = 2 * LM_KEYS * L.pitch;
+    L.s = L.q + 16 * L.pitch;
+    L.phi = L.s + 16 * (LM_KEYS + 4) * 4;
+    L.plo = L.phi + 16 * (LM_KEYS + 8) * 2;
+    L.stat = L.plo + 16 * (LM_KEYS + 8) * 2;
+    L.bytes = L.stat + 3 * 16 * 4;
+    return L;
 }
-__device__ __forceinline__ void la_ldmatrix_x4_trans(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void la_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-// (x, y) as packed bf16 plus what the rounding left over, again in bf16
-__device__ __forceinline__ void la_split(float x, float y, uint32_t &hi, uint32_t &lo) {
-    hi = pg_pack_bf16(x, y);
-    lo = pg_pack_bf16(x - bf16_lo(hi), y - bf16_hi(hi));
+template <int NT>
+RNB_GLOBAL void __launch_bounds__(LM_THREADS)
+latent_attend_mma_kernel(const float *__restrict__ qf, const bf16 *__restrict__ cache, const LatentDims d, float scale, const int *__restrict__ pos0,
+                         float *__restrict__ part) {
+    extern __shared__ __align__(128) uint8_t lm_smem[];
+    pdl_launch_dependents();
+    pdl_wait();
+    const LatentMmaSmem L = latent_mma_smem(d);
+    const uint32_t base = smem_u32(lm_smem);
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h0 = blockIdx.y * 16, t = blockIdx.z, E = d.rank + d.rot_dim;
+    const int EP = (int)(L.pitch / 2) - 8, ld = latent_part_ld(d.rank);
+    int lo, hi;
+    latent_chunk_range(*pos0 + t + 1, gridDim.x, blockIdx.x, lo, hi);
+    float *ss = reinterpret_cast<float *>(lm_smem + L.s), *s_m = reinterpret_cast<float *>(lm_smem + L.stat), *s_l = s_m + 16, *s_c = s_l + 16;
+    bf16 *qs = reinterpret_cast<bf16 *>(lm_smem + L.q), *phi = reinterpret_cast<bf16 *>(lm_smem + L.phi), *plo = reinterpret_cast<bf16 *>(lm_smem + L.plo);
+    constexpr int PE = LM_KEYS + 8, SE = LM_KEYS + 4;
+    auto load_tile = [&](int i) {
+        const int k0 = lo + i * LM_KEYS, per = EP / 8;
+        const uint32_t st = base + (uint32_t)(i & 1) * LM_KEYS * L.pitch;
+        for (int x = tid; x < LM_KEYS * per; x += LM_THREADS) {
+            const int r = x / per, q = x % per, key = k0 + r;
+            // the row's padding (up to ld) is never written by an append; what lies past E meets zero query columns, so it
+            // only has to be finite: it is taken as zero
+            const bool in = key < hi && q * 8 < E;
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(st + (uint32_t)r * L.pitch + (uint32_t)q * 16u),
+                         "l"(cache + (size_t)min(key, hi - 1) * d.ld + min(q * 8, d.ld - 8)), "r"(in ? (uint32_t)min(16, (E - q * 8) * 2) : 0u)
+                         : "memory");
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    const int n_tiles = (hi - lo + LM_KEYS - 1) / LM_KEYS;
+    if (n_tiles > 0) load_tile(0);
+    for (int x = tid; x < 16 * EP; x += LM_THREADS) {
+        const int r = x / EP, e = x % EP;
+        qs[r * (EP + 8) + e] = from_f32<bf16>(h0 + r < d.heads && e < E ? qf[((size_t)t * d.heads + h0 + r) * E + e] : 0.f);
+    }
+    if (tid < 16) s_m[tid] = -INFINITY, s_l[tid] = 0.f;
+    float o[NT][4];
+#pragma unroll
+    for (int n = 0; n < NT; n++) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+    const int g = lane >> 2, tq = lane & 3, mi = lane >> 3, mr = lane & 7, c0 = warp * 8 * NT;
+    const uint32_t a_off = (uint32_t)((mi & 1) * 8 + mr), a_col = (uint32_t)(mi >> 1) * 16u;
+    for (int it = 0; it < n_tiles; it++) {
+        if (it + 1 < n_tiles) {
+            load_tile(it + 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+        const uint32_t st = base + (uint32_t)(it & 1) * LM_KEYS * L.pitch;
+        {   // scores of keys 8 warp .. + 7; independent accumulators hide the MMA latency
+            float s[4][4] = {};
+            const uint32_t qa = base + L.q + a_off * L.pitch + a_col, ka = st + (uint32_t)(warp * 8 + mr) * L.pitch + (uint32_t)mi * 16u;
+#pragma unroll 2
+            for (int k = 0; k < EP / 32; k++) {
+                uint32_t b[4], a0[4], a1[4];
+                lt_ldmatrix_x4(b, ka + (uint32_t)k * 64u);
+                lt_ldmatrix_x4(a0, qa + (uint32_t)k * 64u);
+                lt_ldmatrix_x4(a1, qa + (uint32_t)k * 64u + 32u);
+                lt_mma(s[2 * (k & 1)], a0, b[0], b[1]);
+                lt_mma(s[2 * (k & 1) + 1], a1, b[2], b[3]);
+            }
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const int key = lo + it * LM_KEYS + warp * 8 + 2 * tq + (e & 1);
+                const float v = (s[0][e] + s[1][e]) + (s[2][e] + s[3][e]);
+                ss[(g + 8 * (e >> 1)) * SE + warp * 8 + 2 * tq + (e & 1)] = key < hi ? v * scale : -INFINITY;
+            }
+        }
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < 2; i++) {   // softmax bookkeeping of heads 2 warp, 2 warp + 1
+            const int r = 2 * warp + i;
+            const float x0 = ss[r * SE + lane], x1 = ss[r * SE + lane + 32], m_old = s_m[r];
+            const float m = fmaxf(m_old, warp_max(fmaxf(x0, x1)));
+            const float p0 = expf(x0 - m), p1 = expf(x1 - m), sum = warp_sum(p0 + p1);
+            lt_split_store(phi + r * PE + lane, plo + r * PE + lane, p0);
+            lt_split_store(phi + r * PE + lane + 32, plo + r * PE + lane + 32, p1);
+            if (lane == 0) {
+                const float c = expf(m_old - m);
+                s_c[r] = c;
+                s_m[r] = m;
+                s_l[r] = fmaf(s_l[r], c, sum);
+            }
+        }
+        __syncthreads();
+        const float c_lo = s_c[g], c_hi = s_c[g + 8];
+#pragma unroll
+        for (int n = 0; n < NT; n++) {
+            o[n][0] *= c_lo;
+            o[n][1] *= c_lo;
+            o[n][2] *= c_hi;
+            o[n][3] *= c_hi;
+        }
+#pragma unroll
+        for (int kk = 0; kk < LM_KEYS / 16; kk++) {
+            uint32_t ah[4], al[4];
+            const uint32_t pa = a_off * (PE * 2) + (uint32_t)kk * 32u + a_col;
+            lt_ldmatrix_x4(ah, base + L.phi + pa);
+            lt_ldmatrix_x4(al, base + L.plo + pa);
+            const uint32_t va = st + (uint32_t)(kk * 16 + (mi & 1) * 8 + mr) * L.pitch + (uint32_t)(mi >> 1) * 16u + (uint32_t)c0 * 2u;
+#pragma unroll
+            for (int np = 0; np < (NT + 1) / 2; np++) {
+                if (c0 + np * 16 >= EP) break;
+                uint32_t b[4];
+                lt_ldmatrix_x4_trans(b, va + (uint32_t)np * 32u);
+                lt_mma(o[2 * np], ah, b[0], b[1]);
+                lt_mma(o[2 * np], al, b[0], b[1]);
+                if (2 * np + 1 < NT) {
+                    lt_mma(o[2 * np + 1], ah, b[2], b[3]);
+                    lt_mma(o[2 * np + 1], al, b[2], b[3]);
+                }
+            }
+        }
+        __syncthreads();
+    }
+    __syncthreads();
+    float *out = part + (((size_t)t * d.heads + h0) * gridDim.x + blockIdx.x) * ld;
+    const size_t hs = (size_t)gridDim.x * ld;
+#pragma unroll
+    for (int n = 0; n < NT; n++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+            const int r = g + 8 * (e >> 1), c = c0 + n * 8 + 2 * tq + (e & 1);
+            if (h0 + r < d.heads && c < d.rank) out[r * hs + c] = o[n][e];
+        }
+    if (tid < 16 && h0 + tid < d.heads) {
+        out[tid * hs + d.rank] = s_m[tid];
+        out[tid * hs + d.rank + 1] = s_l[tid];
+    }
 }
 
+// ---- prompts: causal attention over expanded keys and values on tensor cores ---------------------
 constexpr int LA_ROWS = 128, LA_KEYS = 64, LA_THREADS = 256;
 __host__ __device__ inline int la_pad16(int n) { return (n + 15) & ~15; }
 __host__ inline size_t latent_prefill_smem(const LatentDims &d, int dvp) {
@@ -336,13 +515,13 @@ latent_prefill_kernel(const __grid_constant__ LatentPrefillArgs a) {
         const uint32_t kb = k_st + (uint32_t)((mi >> 1) * 8 + mr) * kpitch + (uint32_t)(mi & 1) * 16u;
         for (int kk = 0; kk < KS; kk++) {
             uint32_t af[4];
-            la_ldmatrix_x4(af, q_addr + (uint32_t)kk * 32u);
+            lt_ldmatrix_x4(af, q_addr + (uint32_t)kk * 32u);
 #pragma unroll
             for (int jp = 0; jp < 4; jp++) {
                 uint32_t b[4];
-                la_ldmatrix_x4(b, kb + (uint32_t)(jp * 16) * kpitch + (uint32_t)kk * 32u);
-                la_mma(s[2 * jp], af, b[0], b[1]);
-                la_mma(s[2 * jp + 1], af, b[2], b[3]);
+                lt_ldmatrix_x4(b, kb + (uint32_t)(jp * 16) * kpitch + (uint32_t)kk * 32u);
+                lt_mma(s[2 * jp], af, b[0], b[1]);
+                lt_mma(s[2 * jp + 1], af, b[2], b[3]);
             }
         }
         const int key0 = t * LA_KEYS + 2 * tq;
@@ -374,8 +553,8 @@ latent_prefill_kernel(const __grid_constant__ LatentPrefillArgs a) {
             const float p2 = exp2f(s[j][2] - m_use[1]), p3 = exp2f(s[j][3] - m_use[1]);
             rs[0] += p0 + p1;
             rs[1] += p2 + p3;
-            la_split(p0, p1, ph[j >> 1][2 * (j & 1)], pl[j >> 1][2 * (j & 1)]);
-            la_split(p2, p3, ph[j >> 1][2 * (j & 1) + 1], pl[j >> 1][2 * (j & 1) + 1]);
+            lt_split(p0, p1, ph[j >> 1][2 * (j & 1)], pl[j >> 1][2 * (j & 1)]);
+            lt_split(p2, p3, ph[j >> 1][2 * (j & 1) + 1], pl[j >> 1][2 * (j & 1) + 1]);
         }
 #pragma unroll
         for (int e = 0; e < 2; e++) {
@@ -396,11 +575,11 @@ latent_prefill_kernel(const __grid_constant__ LatentPrefillArgs a) {
 #pragma unroll
             for (int jp = 0; jp < DVJ / 2; jp++) {
                 uint32_t b[4];
-                la_ldmatrix_x4_trans(b, vb + (uint32_t)jp * 32u);
-                la_mma(o[2 * jp], ph[kk], b[0], b[1]);
-                la_mma(o[2 * jp], pl[kk], b[0], b[1]);
-                la_mma(o[2 * jp + 1], ph[kk], b[2], b[3]);
-                la_mma(o[2 * jp + 1], pl[kk], b[2], b[3]);
+                lt_ldmatrix_x4_trans(b, vb + (uint32_t)jp * 32u);
+                lt_mma(o[2 * jp], ph[kk], b[0], b[1]);
+                lt_mma(o[2 * jp], pl[kk], b[0], b[1]);
+                lt_mma(o[2 * jp + 1], ph[kk], b[2], b[3]);
+                lt_mma(o[2 * jp + 1], pl[kk], b[2], b[3]);
             }
         }
         __syncthreads();

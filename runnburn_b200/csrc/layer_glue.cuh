@@ -17,6 +17,12 @@ __device__ __forceinline__ float block_sum(float v, float *red) {
     return warp_sum(v);
 }
 
+// Weights do not depend on the launch before: asking for them ahead of the dependency wait hides their DRAM latency.
+__device__ __forceinline__ void prefetch_l2(const void *p, size_t bytes, int tid, int nthreads) {
+    if (!p) return;
+    for (size_t i = (size_t)tid * 128; i < bytes; i += (size_t)nthreads * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"((const char *)p + i));
+}
+
 // grid = tokens.  x and (when kept for later passes) emb: [tokens][width] f32
 RNB_GLOBAL void __launch_bounds__(256)
 dense_embed_kernel(const bf16 *__restrict__ table, const uint32_t *__restrict__ token, int width, float *__restrict__ x, float *__restrict__ emb) {
@@ -51,6 +57,11 @@ residual_norm_kernel(const __grid_constant__ ResidualNormArgs a) {
     extern __shared__ __align__(16) float rn_smem[];
     __shared__ float red[32];
     pdl_launch_dependents();
+    if (gridDim.x == 1) {
+        prefetch_l2(a.wb, (size_t)a.width * 4, threadIdx.x, blockDim.x);
+        prefetch_l2(a.wn, (size_t)a.width * 4, threadIdx.x, blockDim.x);
+        prefetch_l2(a.mu, (size_t)a.width * 4 * a.n_mix, threadIdx.x, blockDim.x);
+    }
     pdl_wait();
     struct alignas(4 * V) Vec { float v[V]; };
     struct alignas(sizeof(HT) * V) HVec { HT v[V]; };

@@ -145,8 +145,8 @@ int LayerStack::init(const rnb_b200_mixer_cfg *layers) {
     }
     RNB_TRY(alloc((void **)&counters_, (size_t)max_heads * 4));
     RNB_CU(cudaMemset(counters_, 0, (size_t)max_heads * 4));
-    // a chunk of at least 32 keys per CTA, and about two CTAs per SM over the heads
-    attend_chunks_ = std::max(1, std::min((c.max_ctx + 31) / 32, 64));
+    // at least one tile of keys per chunk; more chunks mean more CTAs but more partial results to merge
+    attend_chunks_ = std::max(1, std::min((c.max_ctx + 63) / 64, 48));
     return RNB_B200_OK;
 }
 
@@ -345,7 +345,17 @@ int LayerStack::piece() const {
     return p;
 }
 
-static int linear_chunk(int tokens) { return tokens <= 96 ? tokens : tokens <= 1024 ? 64 : 128; }
+// Tokens per chunk: long chunks move less state, short ones give more CTAs.
+static int linear_chunk(int tokens, int ctas_per_chunk) {
+    if (tokens <= 96) return tokens;
+    for (int c = 256; c > 64; c /= 2)
+        if ((tokens + c - 1) / c * ctas_per_chunk >= 256) return c;
+    return 64;
+}
+static bool linear_tiled(const rnb_b200_mixer_cfg &m) { return m.dim % 8 == 0 && m.vdim % 8 == 0 && m.dim <= 256; }
+static int linear_tile_warps(int vdim) { return std::min((vdim + 15) / 16, 8); }
+// CTAs that work on one chunk of tokens
+static int linear_ctas(const rnb_b200_mixer_cfg &m) { const int w = 16 * linear_tile_warps(m.vdim); return m.heads * ((m.vdim + w - 1) / w); }
 
 int LayerStack::alloc_scratch(StackScratch &b, int cap) {
     for (void *p : b.allocs) cudaFree(p);
@@ -362,7 +372,7 @@ int LayerStack::alloc_scratch(StackScratch &b, int cap) {
             zw = std::max(zw, (size_t)(m.kv_rank + m.rot_dim));
             if (absorbed(L, cap)) {
                 qfw = std::max(qfw, (size_t)m.heads * (m.kv_rank + m.rot_dim));
-                partw = std::max(partw, (size_t)m.heads * (small ? attend_chunks_ : 1) * (m.kv_rank + 2));
+                partw = std::max(partw, (size_t)m.heads * (small ? attend_chunks_ : 1) * latent_part_ld(m.kv_rank));
             } else {
                 kn = std::max(kn, (size_t)cfg.max_ctx * hd);
                 vx = std::max(vx, (size_t)cfg.max_ctx * hv);
@@ -376,8 +386,11 @@ int LayerStack::alloc_scratch(StackScratch &b, int cap) {
                 ww = std::max(ww, hd);
             }
             if (!small) {
-                // most chunks any token count up to cap can have
-                const size_t nc = std::max((T + 127) / 128, (std::min<size_t>(T, 1024) + 63) / 64);
+                size_t nc = 1;   // most chunks any token count up to cap can have
+                for (int t = 1; t <= cap; t++) {
+                    const int c = linear_chunk(t, linear_ctas(m));
+                    nc = std::max(nc, (size_t)((t + c - 1) / c));
+                }
                 st = std::max(st, nc * hd * m.vdim);
                 dc = std::max(dc, nc * hd);
             }
@@ -397,6 +410,7 @@ int LayerStack::alloc_scratch(StackScratch &b, int cap) {
     RNB_TRY(get(&b.part, T * partw * 4));
     RNB_TRY(get(&b.starts, st * 4));
     RNB_TRY(get(&b.decays, dc * 4));
+    if (!small && narrow(cap) && streams == 5) RNB_TRY(get(&b.th, T * zw * 2 * 2));
     RNB_TRY(get(&b.kn, kn * 2));
     RNB_TRY(get(&b.vx, vx * 2));
     RNB_TRY(get(&b.rows, T * 4));
@@ -437,6 +451,31 @@ int LayerStack::ready(cudaStream_t s) {
                          (const void *)linear_state_step_kernel<64>, (const void *)latent_prefill_kernel<4>, (const void *)latent_prefill_kernel<8>,
                          (const void *)latent_prefill_kernel<16>, (const void *)latent_prefill_kernel<32>};
     for (const void *f : fns) RNB_TRY(raise(f));
+    const void *tile[] = {
+#define RNB_LT(DT) (const void *)linear_state_tile_kernel<DT, false, false>, (const void *)linear_state_tile_kernel<DT, false, true>, \
+                   (const void *)linear_state_tile_kernel<DT, true, false>, (const void *)linear_state_tile_kernel<DT, true, true>
+        RNB_LT(2), RNB_LT(4), RNB_LT(8), RNB_LT(16)
+#undef RNB_LT
+    };
+    for (const void *f : tile) RNB_TRY(raise(f));
+    const void *lat[] = {(const void *)latent_attend_mma_kernel<1>, (const void *)latent_attend_mma_kernel<2>, (const void *)latent_attend_mma_kernel<4>,
+                         (const void *)latent_attend_mma_kernel<8>, (const void *)latent_attend_mma_kernel<10>, (const void *)latent_prepare_kernel<float>,
+                         (const void *)latent_prepare_kernel<bf16>, (const void *)latent_output_kernel<float>, (const void *)latent_output_kernel<bf16>};
+    for (const void *f : lat) RNB_TRY(raise(f));
+    for (StackLayer &L : layers_)
+        if (L.w2.w && L.w2.cols % 4 == 0 && !cfg.f32_math) {
+            DenseMat &m = L.w2x;
+            const size_t pitch = (size_t)L.w2.cols * 2;
+            RNB_TRY(alloc((void **)&m.w, (size_t)L.w2.rows * pitch * 2));
+            for (int half = 0; half < 2; half++)
+                RNB_CU(cudaMemcpy2DAsync((char *)m.w + half * pitch, 2 * pitch, L.w2.w, pitch, pitch, (size_t)L.w2.rows, cudaMemcpyDeviceToDevice, s));
+            m.rows = L.w2.rows;
+            m.cols = 2 * L.w2.cols;
+            m.tiled = true;
+            PgTensorMap t;
+            RNB_TRY(encode_token_map(&t, m.w, (size_t)m.rows, (size_t)m.cols, (size_t)m.cols, 64));
+            memcpy(m.map, &t, sizeof(m.map));
+        }
     RNB_TRY(alloc_scratch(small_, SMALL));
     RNB_TRY(reset(s));
     ready_ = true;
@@ -466,7 +505,14 @@ int LayerStack::matmul(cudaStream_t s, int n, const Mm *jobs, int n_jobs, int *e
         DenseVecJobs J;
         memset(&J, 0, sizeof(J));
         J.n = n_jobs;
-        int ctas = 0;
+        int ctas = 0, all = 0, cols = 1 << 30;
+        for (int i = 0; i < n_jobs; i++) {
+            all += jobs[i].w2 ? jobs[i].w->rows : (jobs[i].w->rows + 1) / 2;
+            cols = std::min(cols, jobs[i].w->cols);
+        }
+        // few rows: several warps share a pair of them, so that every SM has loads in flight to the end
+        J.ksplit = all <= 4096 && cols >= 4096 ? 4 : all <= 12288 && cols >= 2048 ? 2 : 1;
+        const int per_cta = DV_WARPS / J.ksplit;
         for (int i = 0; i < n_jobs; i++) {
             DenseVecJob &j = J.j[i];
             j.w = reinterpret_cast<const bf16 *>(jobs[i].w->w);
@@ -478,7 +524,7 @@ int LayerStack::matmul(cudaStream_t s, int n, const Mm *jobs, int n_jobs, int *e
             j.cta0 = ctas;
             j.vec = jobs[i].w->cols % 8 == 0 && ((uintptr_t)j.x & 15) == 0;
             const int units = j.w2 ? j.rows : (j.rows + 1) / 2;
-            ctas += (units + DV_WARPS - 1) / DV_WARPS;
+            ctas += (units + per_cta - 1) / per_cta;
         }
         const dim3 grid((unsigned)ctas), block(DV_WARPS * 32);
         if (n == 1) RNB_CU(launch_k(dense_gemv_kernel<1>, grid, block, 0, s, J));
@@ -500,6 +546,7 @@ int LayerStack::matmul(cudaStream_t s, int n, const Mm *jobs, int n_jobs, int *e
         for (int i = 0; i < n_jobs; i++) {
             DenseGemmJob &j = J.j[i];
             j.y = jobs[i].y;
+            j.decay_bias = jobs[i].decay_bias;
             j.rows = j.ld = jobs[i].w->rows;
             j.cols = jobs[i].w->cols;
             j.tile0 = tiles;
@@ -581,8 +628,33 @@ int LayerStack::boundary(cudaStream_t s, int n, StackScratch &b, int &cur, const
     return RNB_B200_OK;
 }
 
+// linear_state_scan_kernel between the two passes over the chunks
+static int launch_linear_scan(cudaStream_t s, const LinearChunkArgs &a) {
+    const size_t n = (size_t)a.heads * a.dim * a.vdim;
+    const float *decays = a.w ? a.decays : nullptr;
+    if (a.vdim % 4 == 0) RNB_CU(launch_k(linear_state_scan_kernel<4>, dim3((unsigned)((n / 4 + 255) / 256)), dim3(256), 0, s, (const float *)a.state, a.starts, decays, a.decay, a.heads, a.dim, a.vdim, a.chunk, a.n_chunks));
+    else RNB_CU(launch_k(linear_state_scan_kernel<1>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, s, (const float *)a.state, a.starts, decays, a.decay, a.heads, a.dim, a.vdim, a.chunk, a.n_chunks));
+    return RNB_B200_OK;
+}
+template <int DT>
+static int launch_linear_tiles(cudaStream_t s, const LinearChunkArgs &a) {
+    const int nw = linear_tile_warps(a.vdim);
+    const unsigned zb = (unsigned)((a.vdim + 16 * nw - 1) / (16 * nw));
+    const size_t smem = linear_tile_smem(DT, nw).bytes;
+    const dim3 block((unsigned)(32 * nw));
+    if (a.n_chunks > 1) {
+        const dim3 grid((unsigned)(a.n_chunks - 1), (unsigned)a.heads, zb);
+        if (a.w) RNB_CU(launch_k(linear_state_tile_kernel<DT, false, false>, grid, block, smem, s, a));
+        else RNB_CU(launch_k(linear_state_tile_kernel<DT, false, true>, grid, block, smem, s, a));
+        RNB_TRY(launch_linear_scan(s, a));
+    }
+    const dim3 grid((unsigned)a.n_chunks, (unsigned)a.heads, zb);
+    if (a.w) RNB_CU(launch_k(linear_state_tile_kernel<DT, true, false>, grid, block, smem, s, a));
+    else RNB_CU(launch_k(linear_state_tile_kernel<DT, true, true>, grid, block, smem, s, a));
+    return RNB_B200_OK;
+}
 template <class AT>
-static int launch_linear_chunks(cudaStream_t s, LinearChunkArgs a, const float *decay) {
+static int launch_linear_chunks(cudaStream_t s, LinearChunkArgs a) {
     const bool cw = a.w == nullptr;
     a.G = round_pow2((a.dim + LS_TI - 1) / LS_TI);
     a.JG = std::min((a.vdim + 3) / 4, 256 / a.G);
@@ -593,9 +665,7 @@ static int launch_linear_chunks(cudaStream_t s, LinearChunkArgs a, const float *
         const dim3 grid((unsigned)(a.n_chunks - 1), (unsigned)a.heads, zb);
         if (cw) RNB_CU(launch_k(linear_state_chunk_kernel<AT, false, true>, grid, block, smem, s, a));
         else RNB_CU(launch_k(linear_state_chunk_kernel<AT, false, false>, grid, block, smem, s, a));
-        const size_t n = (size_t)a.heads * a.dim * a.vdim;
-        RNB_CU(launch_k(linear_state_scan_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, s, (const float *)a.state, a.starts,
-                        cw ? (const float *)nullptr : (const float *)a.decays, decay, a.heads, a.dim, a.vdim, a.chunk, a.n_chunks));
+        RNB_TRY(launch_linear_scan(s, a));
     }
     const dim3 grid((unsigned)a.n_chunks, (unsigned)a.heads, zb);
     if (cw) RNB_CU(launch_k(linear_state_chunk_kernel<AT, true, true>, grid, block, smem, s, a));
@@ -645,7 +715,13 @@ int LayerStack::mixer_linear(cudaStream_t s, int n, StackScratch &b, StackLayer 
     }
     if (wkv) {
         const int ch = m.heads * m.dim, rank = L.w1.rows;
-        RNB_CU(launch_k(decay_rows_kernel, dim3((unsigned)((ch + 127) / 128), (unsigned)((n + 15) / 16)), dim3(128), (size_t)rank * 64, s, (const float *)b.z,
+        if (nb && L.w2x.w) {
+            const size_t nz = (size_t)n * rank;
+            RNB_CU(launch_k(tanh_split_kernel, dim3((unsigned)((nz + 255) / 256)), dim3(256), 0, s, (const float *)b.z, rank, nz, reinterpret_cast<bf16 *>(b.th)));
+            const Mm dj = {&L.w2x, nullptr, b.th, (size_t)2 * rank, b.w, true, L.w0};
+            RNB_TRY(matmul(s, n, &dj, 1, err));
+        } else
+            RNB_CU(launch_k(decay_rows_kernel, dim3((unsigned)((ch + 127) / 128), (unsigned)((n + 15) / 16)), dim3(128), (size_t)rank * 64, s, (const float *)b.z,
                         reinterpret_cast<const bf16 *>(L.w2.w), (const float *)L.w0, n, rank, ch, b.w));
     } else {
         RotateArgs r;
@@ -665,16 +741,32 @@ int LayerStack::mixer_linear(cudaStream_t s, int n, StackScratch &b, StackLayer 
     a.decay = L.decay, a.u = L.u;
     a.state = R.state, a.o = b.o, a.starts = b.starts, a.decays = b.decays;
     a.tokens = n, a.heads = m.heads, a.dim = m.dim, a.vdim = m.vdim;
-    a.chunk = linear_chunk(n);
+    a.chunk = linear_chunk(n, linear_ctas(m));
     a.n_chunks = (n + a.chunk - 1) / a.chunk;
     if (nb) {
-        RNB_TRY(launch_linear_chunks<bf16>(s, a, L.decay));
+        if (!linear_tiled(m)) RNB_TRY(launch_linear_chunks<bf16>(s, a));
+        else if (m.dim <= 32) RNB_TRY(launch_linear_tiles<2>(s, a));
+        else if (m.dim <= 64) RNB_TRY(launch_linear_tiles<4>(s, a));
+        else if (m.dim <= 128) RNB_TRY(launch_linear_tiles<8>(s, a));
+        else RNB_TRY(launch_linear_tiles<16>(s, a));
         return launch_head_norm_gate<bf16>(s, b.o, L.head_norm, b.p[3], cfg.norm_eps, n, m.heads, m.vdim, b.act);
     }
-    RNB_TRY(launch_linear_chunks<float>(s, a, L.decay));
+    RNB_TRY(launch_linear_chunks<float>(s, a));
     return launch_head_norm_gate<float>(s, b.o, L.head_norm, b.p[3], cfg.norm_eps, n, m.heads, m.vdim, b.act);
 }
 
+static bool latent_mma_fits(const LatentDims &d) { return d.rank % 8 == 0 && d.rank <= 640 && latent_mma_smem(d).bytes <= 220 * 1024; }
+static int launch_latent_attend_mma(cudaStream_t s, const float *qf, const bf16 *cache, const LatentDims &d, float scale, const int *pos, float *part, int n, int chunks) {
+    const dim3 grid((unsigned)chunks, (unsigned)((d.heads + 15) / 16), (unsigned)n), block(LM_THREADS);
+    const size_t smem = latent_mma_smem(d).bytes;
+    const int nt = (d.rank + 63) / 64;
+    if (nt <= 1) RNB_CU(launch_k(latent_attend_mma_kernel<1>, grid, block, smem, s, qf, cache, d, scale, pos, part));
+    else if (nt <= 2) RNB_CU(launch_k(latent_attend_mma_kernel<2>, grid, block, smem, s, qf, cache, d, scale, pos, part));
+    else if (nt <= 4) RNB_CU(launch_k(latent_attend_mma_kernel<4>, grid, block, smem, s, qf, cache, d, scale, pos, part));
+    else if (nt <= 8) RNB_CU(launch_k(latent_attend_mma_kernel<8>, grid, block, smem, s, qf, cache, d, scale, pos, part));
+    else RNB_CU(launch_k(latent_attend_mma_kernel<10>, grid, block, smem, s, qf, cache, d, scale, pos, part));
+    return RNB_B200_OK;
+}
 template <class CT>
 static int launch_latent_attend(cudaStream_t s, const float *qf, const CT *cache, const LatentDims &d, float scale, const int *pos, float *part, int n, int chunks) {
     const dim3 grid((unsigned)chunks, (unsigned)d.heads, (unsigned)n), block(128);
@@ -701,22 +793,24 @@ int LayerStack::mixer_latent(cudaStream_t s, int n, StackScratch &b, StackLayer 
         a.q = (const float *)b.p[0], a.y = b.z, a.w = L.dkv_norm;
         a.uk = reinterpret_cast<const bf16 *>(L.uk.w);
         a.qf = b.qf, a.cache = R.cache, a.pos0 = pos_dev, a.eps = cfg.norm_eps, a.d = d, a.rot = rot;
-        const dim3 grid((unsigned)(m.heads + 1), (unsigned)n, (unsigned)((m.kv_rank + 255) / 256));
+        const dim3 grid((unsigned)(m.heads + 1), (unsigned)n, (unsigned)((m.kv_rank + LP_COLS - 1) / LP_COLS)), pb(LP_THREADS);
+        const size_t psmem = ((size_t)((m.dim + 3) & ~3) + 8 * LP_COLS) * 4;
         const int chunks = n <= SMALL ? attend_chunks_ : 1;
         if (cfg.f32_math) {
-            RNB_CU(launch_k(latent_prepare_kernel<float>, grid, dim3(128), (size_t)m.dim * 4, s, a));
+            RNB_CU(launch_k(latent_prepare_kernel<float>, grid, pb, psmem, s, a));
             RNB_TRY(launch_latent_attend<float>(s, b.qf, (const float *)R.cache, d, m.scale, pos_dev, b.part, n, chunks));
         } else {
-            RNB_CU(launch_k(latent_prepare_kernel<bf16>, grid, dim3(128), (size_t)m.dim * 4, s, a));
-            RNB_TRY(launch_latent_attend<bf16>(s, b.qf, (const bf16 *)R.cache, d, m.scale, pos_dev, b.part, n, chunks));
+            RNB_CU(launch_k(latent_prepare_kernel<bf16>, grid, pb, psmem, s, a));
+            if (latent_mma_fits(d)) RNB_TRY(launch_latent_attend_mma(s, b.qf, (const bf16 *)R.cache, d, m.scale, pos_dev, b.part, n, chunks));
+            else RNB_TRY(launch_latent_attend<bf16>(s, b.qf, (const bf16 *)R.cache, d, m.scale, pos_dev, b.part, n, chunks));
         }
         // a few CTAs per head share its value rows
         const int split = n <= SMALL ? std::max(1, std::min((m.vdim + 15) / 16, sm_ / std::max(1, m.heads * n))) : 1;
         const int rows = (m.vdim + split - 1) / split;
         const dim3 og((unsigned)m.heads, (unsigned)n, (unsigned)split);
-        const size_t smem = (size_t)(m.kv_rank + chunks) * 4;
-        if (nb) RNB_CU(launch_k(latent_output_kernel<bf16>, og, dim3(128), smem, s, (const float *)b.part, reinterpret_cast<const bf16 *>(L.uv.w), d, chunks, rows, (bf16 *)b.act));
-        else RNB_CU(launch_k(latent_output_kernel<float>, og, dim3(128), smem, s, (const float *)b.part, reinterpret_cast<const bf16 *>(L.uv.w), d, chunks, rows, (float *)b.act));
+        const size_t smem = ((size_t)5 * ((m.kv_rank + 3) & ~3) + chunks) * 4;
+        if (nb) RNB_CU(launch_k(latent_output_kernel<bf16>, og, dim3(LO_THREADS), smem, s, (const float *)b.part, reinterpret_cast<const bf16 *>(L.uv.w), d, chunks, rows, (bf16 *)b.act));
+        else RNB_CU(launch_k(latent_output_kernel<float>, og, dim3(LO_THREADS), smem, s, (const float *)b.part, reinterpret_cast<const bf16 *>(L.uv.w), d, chunks, rows, (float *)b.act));
         return RNB_B200_OK;
     }
     RNB_CU(launch_k(latent_append_kernel<bf16>, dim3((unsigned)n), dim3(128), 0, s, (const float *)b.z, (const float *)L.dkv_norm, cfg.norm_eps, d, rot, pos_dev, (bf16 *)R.cache));

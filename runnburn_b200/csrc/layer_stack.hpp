@@ -20,7 +20,7 @@ struct StackLayer {
     rnb_b200_mixer_cfg c;
     std::vector<float> decay_host;
     float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr;
-    DenseMat r, k, v, g, w1, w2, q, dkv, uk, uv, o, gate, up, down;
+    DenseMat r, k, v, g, w1, w2, w2x /* [w2 | w2] */, q, dkv, uk, uv, o, gate, up, down;
     float *mu = nullptr, *w0 = nullptr, *u = nullptr, *head_norm = nullptr, *dkv_norm = nullptr, *decay = nullptr;
     const void *rot_table = nullptr;   // float2 [max_ctx][dims / 2]
 };
@@ -37,6 +37,7 @@ struct StackScratch {
     int cap = 0;   // tokens
     float *x[2] = {nullptr, nullptr}, *emb = nullptr, *y = nullptr, *z = nullptr, *w = nullptr, *o = nullptr, *qf = nullptr, *part = nullptr, *starts = nullptr,
           *decays = nullptr, *logits = nullptr;
+    uint16_t *th = nullptr;   // tanh of the low-rank decay input as bf16 hi + lo
     void *h = nullptr, *p[4] = {nullptr, nullptr, nullptr, nullptr}, *act = nullptr;
     uint16_t *kn = nullptr, *vx = nullptr;
     int *rows = nullptr;
@@ -87,6 +88,7 @@ private:
         size_t ldx;
         void *y;
         bool f32_out;
+        const float *decay_bias = nullptr;
     };
     explicit LayerStack(const rnb_b200_stack_cfg &c) : cfg(c) {}
     int init(const rnb_b200_mixer_cfg *layers);

@@ -9,9 +9,12 @@
 //       OUT = false: every chunk but the last accumulates its own contribution from a zero state;
 //       linear_state_scan_kernel turns these into the state at the start of every chunk;
 //       OUT = true: every chunk runs again from its start state and writes its outputs.
-//     Decays enter as products of w, never as ratios of products: nothing can overflow.
+//   linear_state_tile_kernel    the same two passes on tensor cores for bf16 projections: 16 tokens at a time
+//     (the state stays in f32 accumulators and enters products as bf16 hi + lo parts).
+//   Decays enter as products of w, never as ratios of products: nothing can overflow.
 #pragma once
 #include "layer_glue.cuh"
+#include "mma_bf16.cuh"
 
 namespace rnb {
 
@@ -149,24 +152,38 @@ linear_state_chunk_kernel(const __grid_constant__ LinearChunkArgs a) {
     }
 }
 
-// starts[c] <- the state at the start of chunk c, from the chunks' own contributions.  One thread per state element.
+// starts[c] <- the state at the start of chunk c, from the chunks' own contributions.  One thread per V state
+// elements of a channel's row; the contributions of eight chunks are in flight at a time.
+template <int V>
 RNB_GLOBAL void __launch_bounds__(256)
-linear_state_scan_kernel(const float *__restrict__ state, float *__restrict__ starts, const float *__restrict__ decays, const float *__restrict__ decay,
-                         int heads, int dim, int vdim, int chunk, int n_chunks) {
+linear_state_scan_kernel(const float *__restrict__ state, float *starts, const float *__restrict__ decays, const float *__restrict__ decay, int heads, int dim,
+                         int vdim, int chunk, int n_chunks) {
     pdl_launch_dependents();
     pdl_wait();
-    const size_t n = (size_t)heads * dim * vdim, i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    struct alignas(4 * V) Vec { float v[V]; };
+    const size_t n = (size_t)heads * dim * vdim, i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * V;
     if (i >= n) return;
-    const size_t row = i / vdim;
-    float S = state[i];
+    const size_t row = i / vdim, rows = (size_t)heads * dim;
+    Vec S = *reinterpret_cast<const Vec *>(state + i);
     const float p0 = decays ? 0.f : powf(decay[row / dim], (float)chunk);
-#pragma unroll 4
-    for (int c = 0; c < n_chunks - 1; c++) {
-        const float add = starts[(size_t)c * n + i], p = decays ? decays[(size_t)c * heads * dim + row] : p0;
-        starts[(size_t)c * n + i] = S;
-        S = fmaf(p, S, add);
+    for (int c0 = 0; c0 < n_chunks - 1; c0 += 8) {
+        Vec add[8];
+        float p[8];
+#pragma unroll
+        for (int q = 0; q < 8; q++)
+            if (c0 + q < n_chunks - 1) {
+                add[q] = *reinterpret_cast<const Vec *>(starts + (size_t)(c0 + q) * n + i);
+                p[q] = decays ? decays[(size_t)(c0 + q) * rows + row] : p0;
+            }
+#pragma unroll
+        for (int q = 0; q < 8; q++)
+            if (c0 + q < n_chunks - 1) {
+                *reinterpret_cast<Vec *>(starts + (size_t)(c0 + q) * n + i) = S;
+#pragma unroll
+                for (int e = 0; e < V; e++) S.v[e] = fmaf(p[q], S.v[e], add[q].v[e]);
+            }
     }
-    starts[(size_t)(n_chunks - 1) * n + i] = S;
+    *reinterpret_cast<Vec *>(starts + (size_t)(n_chunks - 1) * n + i) = S;
 }
 
 // Decays of time mixing: out[t][c] = exp(-exp(sum_j w2[c][j] tanh(z[t][j]) + w0[c])).
@@ -205,6 +222,311 @@ decay_rows_kernel(const float *__restrict__ z, const bf16 *__restrict__ w2, cons
         if (t0 + t < tokens) out[(size_t)(t0 + t) * channels + c] = expf(-expf(acc[t] + b));
 }
 
+// z [tokens][rank] f32 -> [tanh z rounded to bf16 | what the rounding left] [tokens][2 rank]: against [w2 | w2] the
+// tensor-core matmul gives w2 tanh(z) to f32 accuracy.
+RNB_GLOBAL void __launch_bounds__(256)
+tanh_split_kernel(const float *__restrict__ z, int rank, size_t n, bf16 *__restrict__ out) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n) return;
+    const float v = tanhf(z[i]);
+    const bf16 hi = from_f32<bf16>(v);
+    bf16 *row = out + (i / rank) * 2 * rank + i % rank;
+    row[0] = hi;
+    row[rank] = from_f32<bf16>(v - to_f32(hi));
+}
+
+// ---- many tokens on tensor cores -----------------------------------------------------------------
+// Shared memory of a CTA of NW warps (16 value columns each): two stages of raw rows, then the processed ones.
+struct LinearTileSmem {
+    uint32_t kp, vp, stage, k, w, v, rhi, rlo, khi, klo, ahi, alo, d, p, pw, bytes;
+};
+__host__ __device__ inline LinearTileSmem linear_tile_smem(int DT, int NW) {
+    LinearTileSmem s;
+    s.kp = (uint32_t)(16 * DT + 8) * 2;
+    s.vp = (uint32_t)(16 * NW + 8) * 2;
+    s.k = 16 * s.kp;
+    s.w = s.k + 16 * s.kp;
+    s.v = s.w + 16 * 16 * DT * 4;
+    s.stage = s.v + 16 * s.vp;
+    s.rhi = 2 * s.stage;
+    s.rlo = s.rhi + 16 * s.kp;
+    s.khi = s.rlo + 16 * s.kp;
+    s.klo = s.khi + 16 * s.kp;
+    s.ahi = s.klo + 16 * s.kp;
+    s.alo = s.ahi + 16 * 48;
+    s.d = s.alo + 16 * 48;
+    s.p = s.d + 16 * DT * 4;
+    s.pw = s.p + 16 * DT * 4;
+    s.bytes = s.pw + 32 * 4;
+    return s;
+}
+// Per tile of 16 tokens, with S^T (value column x channel) in each warp's accumulators:
+//   o^T = S^T r~^T + v^T A^T          r~_t = r_t times the decays before t,  A: pairs inside the tile
+//   S^T <- S^T D + v^T k~             k~_t = k_t times the decays after t,   D: all decays of the tile
+// Time mixing computes A below the diagonal pair by pair (running products of w), with r u k on it;
+// retention masks and scales q k^T by powers of its decay, and scales S^T q^T by them afterwards.
+// grid = (chunks, heads, column blocks), blockDim = 32 * NW.  dim <= 16 DT, dim and vdim multiples of 8.
+template <int DT, bool OUT, bool CONST_W>
+RNB_GLOBAL void __launch_bounds__(256)
+linear_state_tile_kernel(const __grid_constant__ LinearChunkArgs a) {
+    extern __shared__ __align__(128) uint8_t lt_smem[];
+    pdl_launch_dependents();
+    pdl_wait();
+    constexpr int DP = 16 * DT;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nthr = blockDim.x, NW = nthr >> 5;
+    const LinearTileSmem L = linear_tile_smem(DT, NW);
+    const uint32_t base = smem_u32(lt_smem);
+    const int c = blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * 16 * NW;
+    const int t_begin = c * a.chunk, t_end = min(t_begin + a.chunk, a.tokens), n_tiles = (t_end - t_begin + 15) / 16;
+    const bf16 *rp = reinterpret_cast<const bf16 *>(a.r) + (size_t)h * a.dim, *kp = reinterpret_cast<const bf16 *>(a.k) + (size_t)h * a.dim;
+    const bf16 *vp = reinterpret_cast<const bf16 *>(a.v) + (size_t)h * a.vdim;
+    const float *wp = CONST_W ? nullptr : a.w + (size_t)h * a.dim;
+    const size_t ldk = (size_t)a.heads * a.dim, ldv = (size_t)a.heads * a.vdim;
+    float *sD = reinterpret_cast<float *>(lt_smem + L.d), *sP = reinterpret_cast<float *>(lt_smem + L.p), *pw = reinterpret_cast<float *>(lt_smem + L.pw);
+    auto cp16 = [&](uint32_t dst, const void *src, bool in) {
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(in ? 16u : 0u) : "memory");
+    };
+    auto load_tile = [&](int i) {
+        const uint32_t st = base + (uint32_t)(i & 1) * L.stage;
+        const int t0 = t_begin + 16 * i;
+        constexpr int CK = DP / 8, CWF = DP / 4;
+        const int cv = 2 * NW, per = (OUT ? 2 : 1) * CK + (CONST_W ? 0 : CWF) + cv;
+        for (int x = tid; x < 16 * per; x += nthr) {
+            const int t = x / per, tok = t0 + t, row = min(tok, t_end - 1);
+            int q = x % per;
+            const bool in = tok < t_end;
+            if (q < CK) {
+                cp16(st + L.k + (uint32_t)t * L.kp + (uint32_t)q * 16u, kp + (size_t)row * ldk + min(q * 8, a.dim - 8), in && q * 8 < a.dim);
+                continue;
+            }
+            q -= CK;
+            if (OUT) {
+                if (q < CK) {
+                    cp16(st + (uint32_t)t * L.kp + (uint32_t)q * 16u, rp + (size_t)row * ldk + min(q * 8, a.dim - 8), in && q * 8 < a.dim);
+                    continue;
+                }
+                q -= CK;
+            }
+            if (!CONST_W) {
+                if (q < CWF) {
+                    cp16(st + L.w + (uint32_t)(t * DP + q * 4) * 4u, wp + (size_t)row * ldk + min(q * 4, a.dim - 4), in && q * 4 < a.dim);
+                    continue;
+                }
+                q -= CWF;
+            }
+            const int col = j0 + q * 8;
+            cp16(st + L.v + (uint32_t)t * L.vp + (uint32_t)q * 16u, vp + (size_t)row * ldv + min(col, a.vdim - 8), in && col < a.vdim);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    load_tile(0);
+    const float cw = CONST_W ? a.decay[h] : 1.f;
+    if (CONST_W && tid <= 16) pw[tid] = powf(cw, (float)tid);
+    if (!OUT && !CONST_W)
+        for (int i = tid; i < DP; i += nthr) sP[i] = 1.f;
+    const int g = lane >> 2, tq = lane & 3, mi = lane >> 3, mr = lane & 7, jw = j0 + warp * 16;
+    float S[2 * DT][4];
+    const size_t cs = (size_t)a.heads * a.dim * a.vdim;
+    auto state_io = [&](float *b, bool store) {
+#pragma unroll
+        for (int n = 0; n < 2 * DT; n++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const int ch = n * 8 + 2 * tq + (e & 1), j = jw + g + 8 * (e >> 1);
+                const bool in = ch < a.dim && j < a.vdim;
+                float *p = b + ((size_t)h * a.dim + ch) * a.vdim + j;
+                if (store) {
+                    if (in) *p = S[n][e];
+                } else {
+                    S[n][e] = in ? *p : 0.f;
+                }
+            }
+    };
+    if (OUT) state_io(a.n_chunks > 1 ? a.starts + (size_t)c * cs : a.state, false);
+    else
+#pragma unroll
+        for (int n = 0; n < 2 * DT; n++) S[n][0] = S[n][1] = S[n][2] = S[n][3] = 0.f;
+    // fragment addresses that do not change from tile to tile
+    const uint32_t b_plain = (uint32_t)((mi >> 1) * 8 + mr) * L.kp + (uint32_t)(mi & 1) * 16u;        // rows (n), k contiguous
+    const uint32_t b_trans = (uint32_t)((mi & 1) * 8 + mr) * L.kp + (uint32_t)(mi >> 1) * 16u;        // rows (k), n contiguous
+    for (int it = 0; it < n_tiles; it++) {
+        if (it + 1 < n_tiles) {
+            load_tile(it + 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();   // raw rows are in; the previous tile's processed rows are free
+        uint8_t *raw = lt_smem + (size_t)(it & 1) * L.stage;
+        const int t0 = t_begin + 16 * it, nt = min(16, t_end - t0);
+        const bf16 *rr = reinterpret_cast<const bf16 *>(raw), *kk = reinterpret_cast<const bf16 *>(raw + L.k);
+        const float *ww = reinterpret_cast<const float *>(raw + L.w);
+        bf16 *rhi = reinterpret_cast<bf16 *>(lt_smem + L.rhi), *rlo = reinterpret_cast<bf16 *>(lt_smem + L.rlo);
+        bf16 *khi = reinterpret_cast<bf16 *>(lt_smem + L.khi), *klo = reinterpret_cast<bf16 *>(lt_smem + L.klo);
+        bf16 *ahi = reinterpret_cast<bf16 *>(lt_smem + L.ahi), *alo = reinterpret_cast<bf16 *>(lt_smem + L.alo);
+        constexpr int KE = DP + 8;
+        if (CONST_W) {
+            for (int x = tid; x < 16 * DP; x += nthr) {
+                const int t = x / DP, ch = x % DP;
+                lt_split_store(khi + t * KE + ch, klo + t * KE + ch, t < nt ? to_f32(kk[t * KE + ch]) * pw[nt - 1 - t] : 0.f);
+            }
+            if (OUT && warp == 0) {
+                float q[2][4] = {};
+                const uint32_t ra = base + (uint32_t)(it & 1) * L.stage + (uint32_t)((mi & 1) * 8 + mr) * L.kp + (uint32_t)(mi >> 1) * 16u;
+                const uint32_t kb = base + (uint32_t)(it & 1) * L.stage + L.k + b_plain;
+#pragma unroll
+                for (int ks = 0; ks < DT; ks++) {
+                    uint32_t ra4[4], kb4[4];
+                    lt_ldmatrix_x4(ra4, ra + (uint32_t)ks * 32u);
+                    lt_ldmatrix_x4(kb4, kb + (uint32_t)ks * 32u);
+                    lt_mma(q[0], ra4, kb4[0], kb4[1]);
+                    lt_mma(q[1], ra4, kb4[2], kb4[3]);
+                }
+#pragma unroll
+                for (int n = 0; n < 2; n++)
+#pragma unroll
+                    for (int e = 0; e < 4; e++) {
+                        const int t = g + 8 * (e >> 1), s = n * 8 + 2 * tq + (e & 1);
+                        lt_split_store(ahi + t * 24 + s, alo + t * 24 + s, s <= t ? q[n][e] * pw[t - s] : 0.f);
+                    }
+            }
+        } else {
+            // decays before each token (for r) and after it (for k), channel by channel
+            for (int x = tid; x < 2 * DP; x += nthr) {
+                const int ch = x % DP;
+                if (x < DP) {
+                    float p = 1.f;
+#pragma unroll
+                    for (int t = 15; t >= 0; t--) {
+                        lt_split_store(khi + t * KE + ch, klo + t * KE + ch, to_f32(kk[t * KE + ch]) * p);
+                        if (t < nt) p *= ww[t * DP + ch];
+                    }
+                    sD[ch] = p;
+                    if (!OUT) sP[ch] *= p;
+                } else if (OUT) {
+                    float p = 1.f;
+#pragma unroll
+                    for (int t = 0; t < 16; t++) {
+                        lt_split_store(rhi + t * KE + ch, rlo + t * KE + ch, to_f32(rr[t * KE + ch]) * p);
+                        if (t < nt) p *= ww[t * DP + ch];
+                    }
+                }
+            }
+            if (OUT) {
+                // eight lanes share a column s of A; lane q takes channels q, q + 8, ...; a warp's four columns lie four apart
+                constexpr int CH = DP / 8;
+                const int q = lane & 7;
+                for (int s0 = warp; s0 < 4; s0 += NW) {
+                    const int s = s0 + 4 * (lane >> 3);
+                    float x[CH], b = 0.f;
+#pragma unroll
+                    for (int i = 0; i < CH; i++) {
+                        const int ch = q + 8 * i;
+                        x[i] = to_f32(kk[s * KE + ch]);
+                        const float u = ch < a.dim ? a.u[h * a.dim + ch] : 0.f;
+                        b = fmaf(to_f32(rr[s * KE + ch]) * u, x[i], b);
+                    }
+#pragma unroll
+                    for (int t = 0; t < 16; t++) {
+                        float v = t == s ? b : 0.f;
+                        if (t > s) {
+#pragma unroll
+                            for (int i = 0; i < CH; i++) {
+                                const int ch = q + 8 * i;
+                                v = fmaf(to_f32(rr[t * KE + ch]), x[i], v);
+                                x[i] *= ww[t * DP + ch];
+                            }
+                        }
+                        v += __shfl_xor_sync(0xffffffffu, v, 1);
+                        v += __shfl_xor_sync(0xffffffffu, v, 2);
+                        v += __shfl_xor_sync(0xffffffffu, v, 4);
+                        if (q == (t & 7)) lt_split_store(ahi + t * 24 + s, alo + t * 24 + s, v);
+                    }
+                }
+            }
+        }
+        __syncthreads();
+        // v^T fragments: (columns, tokens) from [token][column] rows
+        uint32_t va[4];
+        lt_ldmatrix_x4_trans(va, base + (uint32_t)(it & 1) * L.stage + L.v + (uint32_t)((mi >> 1) * 8 + mr) * L.vp + (uint32_t)(warp * 32 + (mi & 1) * 16));
+        if (OUT) {
+            float o[2][4] = {};
+            const uint32_t rb = CONST_W ? base + (uint32_t)(it & 1) * L.stage : base + L.rhi;
+#pragma unroll
+            for (int ks = 0; ks < DT; ks++) {
+                uint32_t sh[4], sl[4], r4[4];
+                lt_split(S[2 * ks][0], S[2 * ks][1], sh[0], sl[0]);
+                lt_split(S[2 * ks][2], S[2 * ks][3], sh[1], sl[1]);
+                lt_split(S[2 * ks + 1][0], S[2 * ks + 1][1], sh[2], sl[2]);
+                lt_split(S[2 * ks + 1][2], S[2 * ks + 1][3], sh[3], sl[3]);
+                lt_ldmatrix_x4(r4, rb + b_plain + (uint32_t)ks * 32u);
+                lt_mma(o[0], sh, r4[0], r4[1]);
+                lt_mma(o[1], sh, r4[2], r4[3]);
+                lt_mma(o[0], sl, r4[0], r4[1]);
+                lt_mma(o[1], sl, r4[2], r4[3]);
+                if (!CONST_W) {
+                    lt_ldmatrix_x4(r4, base + L.rlo + b_plain + (uint32_t)ks * 32u);
+                    lt_mma(o[0], sh, r4[0], r4[1]);
+                    lt_mma(o[1], sh, r4[2], r4[3]);
+                }
+            }
+            if (CONST_W) {
+#pragma unroll
+                for (int n = 0; n < 2; n++)
+#pragma unroll
+                    for (int e = 0; e < 4; e++) o[n][e] *= pw[n * 8 + 2 * tq + (e & 1) + 1];
+            }
+            uint32_t ab[4];
+            const uint32_t aa = (uint32_t)((mi >> 1) * 8 + mr) * 48u + (uint32_t)(mi & 1) * 16u;
+            lt_ldmatrix_x4(ab, base + L.ahi + aa);
+            lt_mma(o[0], va, ab[0], ab[1]);
+            lt_mma(o[1], va, ab[2], ab[3]);
+            lt_ldmatrix_x4(ab, base + L.alo + aa);
+            lt_mma(o[0], va, ab[0], ab[1]);
+            lt_mma(o[1], va, ab[2], ab[3]);
+#pragma unroll
+            for (int n = 0; n < 2; n++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    const int t = n * 8 + 2 * tq + (e & 1), j = jw + g + 8 * (e >> 1);
+                    if (t < nt && j < a.vdim) a.o[((size_t)(t0 + t) * a.heads + h) * a.vdim + j] = o[n][e];
+                }
+        }
+#pragma unroll
+        for (int np = 0; np < DT; np++) {
+            uint32_t kb[4];
+            float d0[2], d1[2];
+            if (CONST_W) {
+                d0[0] = d0[1] = d1[0] = d1[1] = pw[nt];
+            } else {
+                const float2 x = *reinterpret_cast<const float2 *>(sD + np * 16 + 2 * tq), y = *reinterpret_cast<const float2 *>(sD + np * 16 + 8 + 2 * tq);
+                d0[0] = x.x, d0[1] = x.y, d1[0] = y.x, d1[1] = y.y;
+            }
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                S[2 * np][e] *= d0[e & 1];
+                S[2 * np + 1][e] *= d1[e & 1];
+            }
+            lt_ldmatrix_x4_trans(kb, base + L.khi + b_trans + (uint32_t)np * 32u);
+            lt_mma(S[2 * np], va, kb[0], kb[1]);
+            lt_mma(S[2 * np + 1], va, kb[2], kb[3]);
+            lt_ldmatrix_x4_trans(kb, base + L.klo + b_trans + (uint32_t)np * 32u);
+            lt_mma(S[2 * np], va, kb[0], kb[1]);
+            lt_mma(S[2 * np + 1], va, kb[2], kb[3]);
+        }
+        __syncthreads();   // this stage and the processed rows may be overwritten now
+    }
+    if (OUT) {
+        if (c == a.n_chunks - 1) state_io(a.state, true);
+    } else {
+        state_io(a.starts + (size_t)c * cs, true);
+        if (!CONST_W && blockIdx.z == 0)
+            for (int ch = tid; ch < a.dim; ch += nthr) a.decays[((size_t)c * a.heads + h) * a.dim + ch] = sP[ch];
+    }
+}
+
 // ---- few tokens: everything between the projections in one launch -------------------------------
 struct LinearStepArgs {
     const float *r, *k, *v, *g;      // projections of the tokens, f32: [tokens][heads * dim] (v, g: heads * vdim)
@@ -229,13 +551,26 @@ linear_state_step_kernel(const __grid_constant__ LinearStepArgs a) {
     extern __shared__ __align__(16) float st_smem[];
     __shared__ int s_last;
     pdl_launch_dependents();
-    pdl_wait();
     const int T = a.tokens, dim = a.dim, vdim = a.vdim, h = blockIdx.x, j0 = blockIdx.y * 32;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, j = j0 + lane;
     const bool live = j < vdim;
     float *sr = st_smem, *sk = sr + T * dim, *sw = sk + T * dim, *sz = sw + T * dim, *sv = sz + T * a.rank, *sb = sv + T * 32, *red = sb + T;
-    float S[TI];
+    // four lanes per channel of the decay product; the first 64 channels' weights are loaded ahead of the wait
+    const int dch = tid >> 2, dl = tid & 3, seg = a.rank / 4;
+    const bool dvec = !a.decay && a.rank % 32 == 0 && a.rank <= 128;
+    uint4 dw[4];
+    if (dvec && dch < dim)
+#pragma unroll
+        for (int i = 0; i < 4; i++)
+            if (i * 8 < seg) dw[i] = ldg_nc_u4(a.w2 + ((size_t)h * dim + dch) * a.rank + dl * seg + i * 8);
     float *sp = a.state + (size_t)h * dim * vdim + j;
+    if (vdim * 4 >= 128) {
+        for (int ch = tid; ch < dim; ch += 256) asm volatile("prefetch.global.L2 [%0];" ::"l"(a.state + ((size_t)h * dim + ch) * vdim + j0));
+    } else if (blockIdx.y == 0) {
+        prefetch_l2(a.state + (size_t)h * dim * vdim, (size_t)dim * vdim * 4, tid, 256);
+    }
+    pdl_wait();
+    float S[TI];
 #pragma unroll
     for (int q = 0; q < TI; q++) {
         const int ch = warp + 8 * q;
@@ -255,7 +590,32 @@ linear_state_step_kernel(const __grid_constant__ LinearStepArgs a) {
     }
     for (int i = tid; i < T * a.rank; i += 256) sz[i] = tanhf(a.z[i]);
     __syncthreads();
-    if (!a.decay) {
+    if (dvec) {
+        for (int ch = dch; ch < (dim + 63) / 64 * 64; ch += 64) {
+            if (ch != dch && ch < dim)
+#pragma unroll
+                for (int i = 0; i < 4; i++)
+                    if (i * 8 < seg) dw[i] = ldg_nc_u4(a.w2 + ((size_t)h * dim + ch) * a.rank + dl * seg + i * 8);
+            for (int t = 0; t < T; t++) {
+                float s = 0.f;
+                const float *z = sz + t * a.rank + dl * seg;
+                if (ch < dim)
+#pragma unroll
+                    for (int i = 0; i < 4; i++)
+                        if (i * 8 < seg) {
+                            const uint32_t p[4] = {dw[i].x, dw[i].y, dw[i].z, dw[i].w};
+#pragma unroll
+                            for (int e = 0; e < 4; e++) {
+                                s = fmaf(bf16_lo(p[e]), z[i * 8 + 2 * e], s);
+                                s = fmaf(bf16_hi(p[e]), z[i * 8 + 2 * e + 1], s);
+                            }
+                        }
+                s += __shfl_xor_sync(0xffffffffu, s, 1);
+                s += __shfl_xor_sync(0xffffffffu, s, 2);
+                if (dl == 0 && ch < dim) sw[t * dim + ch] = expf(-expf(s + a.w0[h * dim + ch]));
+            }
+        }
+    } else if (!a.decay) {
         for (int ch = warp; ch < dim; ch += 8) {
             const bf16 *w = a.w2 + ((size_t)h * dim + ch) * a.rank;
             for (int t = 0; t < T; t++) {

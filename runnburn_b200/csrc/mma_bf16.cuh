@@ -1,0 +1,29 @@
+// Warp-level bf16 tensor-core helpers: fragments, m16n8k16 products, and the split of an f32 value into
+// a bf16 and what its rounding left (again bf16), which keeps about 16 bits of it in a product.
+#pragma once
+#include "dense.cuh"
+
+namespace rnb {
+
+__device__ __forceinline__ void lt_ldmatrix_x4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void lt_ldmatrix_x4_trans(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void lt_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void lt_split(float x, float y, uint32_t &hi, uint32_t &lo) {
+    hi = pg_pack_bf16(x, y);
+    lo = pg_pack_bf16(x - bf16_lo(hi), y - bf16_hi(hi));
+}
+__device__ __forceinline__ void lt_split_store(bf16 *hi, bf16 *lo, float v) {
+    const bf16 h = from_f32<bf16>(v);
+    *hi = h;
+    *lo = from_f32<bf16>(v - to_f32(h));
+}
+
+}  // namespace rnb

@@ -325,7 +325,7 @@ def test_many_wanted_places():
         places = [5, 5] + list(range(299, -1, -1))
         got, nxt = dec.prefill_logits(toks, 0, places)
         assert not _bad(got, want[places], dtype)
-        assert nxt == int(np.argmax(got[2])) or su.rel(got[2:3], want[299:300]) > 0
+        assert dtype == "bfloat16" or nxt == int(np.argmax(want[299]))
         dec.close()
 
 
