@@ -46,7 +46,8 @@ latent_append_kernel(const float *__restrict__ y, const float *__restrict__ w, f
 struct LatentPrepareArgs {
     const float *q, *y, *w;      // [tokens][heads * (dim + rot)], [tokens][rank + rot], [rank]
     const bf16 *uk;              // [heads * dim][rank]
-    float *qf;                   // [tokens][heads][rank + rot]
+    void *qf;                    // [tokens][heads][qld] of QT, zeros from rank + rot on
+    int qld;
     void *cache;
     const int *pos0;
     float eps;
@@ -54,7 +55,7 @@ struct LatentPrepareArgs {
     Rotation rot;
 };
 constexpr int LP_THREADS = 512, LP_COLS = 512, LP_BATCH = 8;
-template <class CT>
+template <class CT, class QT>
 RNB_GLOBAL void __launch_bounds__(LP_THREADS)
 latent_prepare_kernel(const __grid_constant__ LatentPrepareArgs a) {
     extern __shared__ __align__(16) float lp_smem[];
@@ -83,17 +84,18 @@ latent_prepare_kernel(const __grid_constant__ LatentPrepareArgs a) {
     fetch(0);
     pdl_wait();
     const float *q = a.q + ((size_t)t * d.heads + h) * (d.dim + d.rot_dim);
-    float *out = a.qf + ((size_t)t * d.heads + h) * E;
+    QT *out = reinterpret_cast<QT *>(a.qf) + ((size_t)t * d.heads + h) * a.qld;
     for (int i = tid; i < d.dim; i += LP_THREADS) sq[i] = q[i];
     if (blockIdx.z == 0)
-        for (int i = tid; i < d.rot_dim; i += LP_THREADS) out[d.rank + i] = rotated_element(a.rot, *a.pos0 + t, i, [&](int e) { return q[d.dim + e]; });
+        for (int i = tid; i < a.qld - d.rank; i += LP_THREADS)
+            out[d.rank + i] = from_f32<QT>(i < d.rot_dim ? rotated_element(a.rot, *a.pos0 + t, i, [&](int e) { return q[d.dim + e]; }) : 0.f);
     __syncthreads();
     if (!vec) {
         for (int e = blockIdx.z * LP_COLS + tid; e < min(d.rank, (int)(blockIdx.z + 1) * LP_COLS); e += LP_THREADS) {
             const bf16 *col = a.uk + (size_t)h * d.dim * d.rank + e;
             float s = 0.f;
             for (int i = 0; i < d.dim; i++) s = fmaf(to_f32(col[(size_t)i * d.rank]), sq[i], s);
-            out[e] = s;
+            out[e] = from_f32<QT>(s);
         }
         return;
     }
@@ -120,7 +122,7 @@ latent_prepare_kernel(const __grid_constant__ LatentPrepareArgs a) {
         float s = 0.f;
 #pragma unroll
         for (int k = 0; k < 8; k++) s += sr[k * LP_COLS + tid];
-        out[e] = s;
+        out[e] = from_f32<QT>(s);
     }
 }
 
@@ -273,7 +275,7 @@ __host__ __device__ inline LatentMmaSmem latent_mma_smem(const LatentDims &d) {
 }
 template <int NT>
 RNB_GLOBAL void __launch_bounds__(LM_THREADS)
-latent_attend_mma_kernel(const float *__restrict__ qf, const bf16 *__restrict__ cache, const LatentDims d, float scale, const int *__restrict__ pos0,
+latent_attend_mma_kernel(const bf16 *__restrict__ qf, const bf16 *__restrict__ cache, const LatentDims d, float scale, const int *__restrict__ pos0,
                          float *__restrict__ part) {
     extern __shared__ __align__(128) uint8_t lm_smem[];
     pdl_launch_dependents();
@@ -285,7 +287,7 @@ latent_attend_mma_kernel(const float *__restrict__ qf, const bf16 *__restrict__ 
     int lo, hi;
     latent_chunk_range(*pos0 + t + 1, gridDim.x, blockIdx.x, lo, hi);
     float *ss = reinterpret_cast<float *>(lm_smem + L.s), *s_m = reinterpret_cast<float *>(lm_smem + L.stat), *s_l = s_m + 16, *s_c = s_l + 16;
-    bf16 *qs = reinterpret_cast<bf16 *>(lm_smem + L.q), *phi = reinterpret_cast<bf16 *>(lm_smem + L.phi), *plo = reinterpret_cast<bf16 *>(lm_smem + L.plo);
+    bf16 *phi = reinterpret_cast<bf16 *>(lm_smem + L.phi), *plo = reinterpret_cast<bf16 *>(lm_smem + L.plo);
     constexpr int PE = LM_KEYS + 8, SE = LM_KEYS + 4;
     auto load_tile = [&](int i) {
         const int k0 = lo + i * LM_KEYS, per = EP / 8;
@@ -302,10 +304,15 @@ latent_attend_mma_kernel(const float *__restrict__ qf, const bf16 *__restrict__ 
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     const int n_tiles = (hi - lo + LM_KEYS - 1) / LM_KEYS;
-    if (n_tiles > 0) load_tile(0);
-    for (int x = tid; x < 16 * EP; x += LM_THREADS) {
-        const int r = x / EP, e = x % EP;
-        qs[r * (EP + 8) + e] = from_f32<bf16>(h0 + r < d.heads && e < E ? qf[((size_t)t * d.heads + h0 + r) * E + e] : 0.f);
+    if (n_tiles > 0) {
+        // query rows (pitch EP in memory), part of the first tile's copy group
+        for (int x = tid; x < 16 * (EP / 8); x += LM_THREADS) {
+            const int r = x / (EP / 8), q = x % (EP / 8);
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(base + L.q + (uint32_t)r * L.pitch + (uint32_t)q * 16u),
+                         "l"(qf + ((size_t)t * d.heads + min(h0 + r, d.heads - 1)) * EP + q * 8), "r"(h0 + r < d.heads ? 16u : 0u)
+                         : "memory");
+        }
+        load_tile(0);
     }
     if (tid < 16) s_m[tid] = -INFINITY, s_l[tid] = 0.f;
     float o[NT][4];

@@ -205,21 +205,39 @@ rotate_heads_kernel(const __grid_constant__ RotateArgs a) {
         }
 }
 
-// act = (o / rms(o over the head)) * w * silu(g); w null: 1.  One warp per (token, head).
-template <class GT, class HT>
+// act = (o / rms(o over the head)) * w * silu(g); w null: 1.  `lanes` (a power of two up to 32) per
+// (token, head), V elements per access (4 when vdim % 4 == 0, else 1).
+template <class GT, class HT, int V>
 RNB_GLOBAL void __launch_bounds__(256)
-head_norm_gate_kernel(const float *__restrict__ o, const float *__restrict__ w, const GT *__restrict__ g, float eps, int tokens, int heads, int vdim,
+head_norm_gate_kernel(const float *__restrict__ o, const float *__restrict__ w, const GT *__restrict__ g, float eps, size_t units, int heads, int vdim, int lanes,
                       HT *__restrict__ act) {
     pdl_launch_dependents();
     pdl_wait();
-    const int unit = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (unit >= tokens * heads) return;
-    const size_t at = (size_t)unit * vdim;
-    const int hw = (unit % heads) * vdim;
+    struct alignas(4 * V) Vec { float v[V]; };
+    struct alignas(sizeof(GT) * V) GVec { GT v[V]; };
+    struct alignas(sizeof(HT) * V) HVec { HT v[V]; };
+    const size_t unit = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) / lanes;
+    const int l = threadIdx.x & (lanes - 1);
+    const bool in = unit < units;
+    const size_t at = (in ? unit : 0) * vdim;
+    const int hw = (int)((in ? unit : 0) % heads) * vdim;
     float ss = 0.f;
-    for (int j = lane; j < vdim; j += 32) ss = fmaf(o[at + j], o[at + j], ss);
-    const float r = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + eps);
-    for (int j = lane; j < vdim; j += 32) act[at + j] = from_f32<HT>(o[at + j] * r * (w ? w[hw + j] : 1.0f) * silu_f32(to_f32(g[at + j])));
+    for (int j = l * V; j < vdim; j += lanes * V) {
+        const Vec x = *reinterpret_cast<const Vec *>(o + at + j);
+#pragma unroll
+        for (int e = 0; e < V; e++) ss = fmaf(x.v[e], x.v[e], ss);
+    }
+    for (int d = 1; d < lanes; d <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
+    const float r = 1.0f / sqrtf(ss / (float)vdim + eps);
+    if (!in) return;
+    for (int j = l * V; j < vdim; j += lanes * V) {
+        const Vec x = *reinterpret_cast<const Vec *>(o + at + j);
+        const GVec y = *reinterpret_cast<const GVec *>(g + at + j);
+        HVec out;
+#pragma unroll
+        for (int e = 0; e < V; e++) out.v[e] = from_f32<HT>(x.v[e] * r * (w ? w[hw + j + e] : 1.0f) * silu_f32(to_f32(y.v[e])));
+        *reinterpret_cast<HVec *>(act + at + j) = out;
+    }
 }
 
 }  // namespace rnb

@@ -371,7 +371,7 @@ int LayerStack::alloc_scratch(StackScratch &b, int cap) {
             proj = std::max(proj, (size_t)m.heads * (m.dim + m.rot_dim) * (absorbed(L, cap) && es == 2 ? 2 : 1));
             zw = std::max(zw, (size_t)(m.kv_rank + m.rot_dim));
             if (absorbed(L, cap)) {
-                qfw = std::max(qfw, (size_t)m.heads * (m.kv_rank + m.rot_dim));
+                qfw = std::max(qfw, (size_t)m.heads * (m.kv_rank + m.rot_dim + 32));
                 partw = std::max(partw, (size_t)m.heads * (small ? attend_chunks_ : 1) * latent_part_ld(m.kv_rank));
             } else {
                 kn = std::max(kn, (size_t)cfg.max_ctx * hd);
@@ -459,8 +459,8 @@ int LayerStack::ready(cudaStream_t s) {
     };
     for (const void *f : tile) RNB_TRY(raise(f));
     const void *lat[] = {(const void *)latent_attend_mma_kernel<1>, (const void *)latent_attend_mma_kernel<2>, (const void *)latent_attend_mma_kernel<4>,
-                         (const void *)latent_attend_mma_kernel<8>, (const void *)latent_attend_mma_kernel<10>, (const void *)latent_prepare_kernel<float>,
-                         (const void *)latent_prepare_kernel<bf16>, (const void *)latent_output_kernel<float>, (const void *)latent_output_kernel<bf16>};
+                         (const void *)latent_attend_mma_kernel<8>, (const void *)latent_attend_mma_kernel<10>, (const void *)latent_prepare_kernel<float, float>,
+                         (const void *)latent_prepare_kernel<bf16, float>, (const void *)latent_prepare_kernel<bf16, bf16>, (const void *)latent_output_kernel<float>, (const void *)latent_output_kernel<bf16>};
     for (const void *f : lat) RNB_TRY(raise(f));
     for (StackLayer &L : layers_)
         if (L.w2.w && L.w2.cols % 4 == 0 && !cfg.f32_math) {
@@ -674,7 +674,11 @@ static int launch_linear_chunks(cudaStream_t s, LinearChunkArgs a) {
 }
 template <class HT>
 static int launch_head_norm_gate(cudaStream_t s, const float *o, const float *w, const void *g, float eps, int n, int heads, int vdim, void *act) {
-    RNB_CU(launch_k(head_norm_gate_kernel<HT, HT>, dim3((unsigned)(((size_t)n * heads + 7) / 8)), dim3(256), 0, s, o, w, (const HT *)g, eps, n, heads, vdim, (HT *)act));
+    const int v = vdim % 4 == 0 ? 4 : 1, lanes = std::min(32, round_pow2((vdim + v - 1) / v));
+    const size_t units = (size_t)n * heads;
+    const dim3 grid((unsigned)((units * lanes + 255) / 256));
+    if (v == 4) RNB_CU(launch_k(head_norm_gate_kernel<HT, HT, 4>, grid, dim3(256), 0, s, o, w, (const HT *)g, eps, units, heads, vdim, lanes, (HT *)act));
+    else RNB_CU(launch_k(head_norm_gate_kernel<HT, HT, 1>, grid, dim3(256), 0, s, o, w, (const HT *)g, eps, units, heads, vdim, lanes, (HT *)act));
     return RNB_B200_OK;
 }
 
@@ -756,7 +760,7 @@ int LayerStack::mixer_linear(cudaStream_t s, int n, StackScratch &b, StackLayer 
 }
 
 static bool latent_mma_fits(const LatentDims &d) { return d.rank % 8 == 0 && d.rank <= 640 && latent_mma_smem(d).bytes <= 220 * 1024; }
-static int launch_latent_attend_mma(cudaStream_t s, const float *qf, const bf16 *cache, const LatentDims &d, float scale, const int *pos, float *part, int n, int chunks) {
+static int launch_latent_attend_mma(cudaStream_t s, const bf16 *qf, const bf16 *cache, const LatentDims &d, float scale, const int *pos, float *part, int n, int chunks) {
     const dim3 grid((unsigned)chunks, (unsigned)((d.heads + 15) / 16), (unsigned)n), block(LM_THREADS);
     const size_t smem = latent_mma_smem(d).bytes;
     const int nt = (d.rank + 63) / 64;
@@ -792,16 +796,18 @@ int LayerStack::mixer_latent(cudaStream_t s, int n, StackScratch &b, StackLayer 
         memset(&a, 0, sizeof(a));
         a.q = (const float *)b.p[0], a.y = b.z, a.w = L.dkv_norm;
         a.uk = reinterpret_cast<const bf16 *>(L.uk.w);
-        a.qf = b.qf, a.cache = R.cache, a.pos0 = pos_dev, a.eps = cfg.norm_eps, a.d = d, a.rot = rot;
+        const bool mma = !cfg.f32_math && latent_mma_fits(d);
+        a.qf = b.qf, a.qld = mma ? (m.kv_rank + m.rot_dim + 31) & ~31 : m.kv_rank + m.rot_dim, a.cache = R.cache, a.pos0 = pos_dev, a.eps = cfg.norm_eps, a.d = d, a.rot = rot;
         const dim3 grid((unsigned)(m.heads + 1), (unsigned)n, (unsigned)((m.kv_rank + LP_COLS - 1) / LP_COLS)), pb(LP_THREADS);
         const size_t psmem = ((size_t)((m.dim + 3) & ~3) + 8 * LP_COLS) * 4;
         const int chunks = n <= SMALL ? attend_chunks_ : 1;
         if (cfg.f32_math) {
-            RNB_CU(launch_k(latent_prepare_kernel<float>, grid, pb, psmem, s, a));
+            RNB_CU(launch_k(latent_prepare_kernel<float, float>, grid, pb, psmem, s, a));
             RNB_TRY(launch_latent_attend<float>(s, b.qf, (const float *)R.cache, d, m.scale, pos_dev, b.part, n, chunks));
         } else {
-            RNB_CU(launch_k(latent_prepare_kernel<bf16>, grid, pb, psmem, s, a));
-            if (latent_mma_fits(d)) RNB_TRY(launch_latent_attend_mma(s, b.qf, (const bf16 *)R.cache, d, m.scale, pos_dev, b.part, n, chunks));
+            if (mma) RNB_CU(launch_k(latent_prepare_kernel<bf16, bf16>, grid, pb, psmem, s, a));
+            else RNB_CU(launch_k(latent_prepare_kernel<bf16, float>, grid, pb, psmem, s, a));
+            if (mma) RNB_TRY(launch_latent_attend_mma(s, (const bf16 *)b.qf, (const bf16 *)R.cache, d, m.scale, pos_dev, b.part, n, chunks));
             else RNB_TRY(launch_latent_attend<bf16>(s, b.qf, (const bf16 *)R.cache, d, m.scale, pos_dev, b.part, n, chunks));
         }
         // a few CTAs per head share its value rows

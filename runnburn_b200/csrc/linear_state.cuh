@@ -415,28 +415,46 @@ linear_state_tile_kernel(const __grid_constant__ LinearChunkArgs a) {
                 }
             }
             if (OUT) {
-                // eight lanes share a column s of A; lane q takes channels q, q + 8, ...; a warp's four columns lie four apart
-                constexpr int CH = DP / 8;
+                // eight lanes share a column s of A; lane q takes channels 4 q .. 4 q + 3, 4 (q + 8) .., ...; a warp's four
+                // columns lie four apart
+                constexpr int C4 = DP / 32;
                 const int q = lane & 7;
                 for (int s0 = warp; s0 < 4; s0 += NW) {
                     const int s = s0 + 4 * (lane >> 3);
-                    float x[CH], b = 0.f;
+                    float x[C4][4], b = 0.f;
+                    auto row4 = [&](const bf16 *p, int i, float (&o)[4]) {
+                        const uint2 w = *reinterpret_cast<const uint2 *>(p + 4 * (q + 8 * i));
+                        o[0] = bf16_lo(w.x), o[1] = bf16_hi(w.x), o[2] = bf16_lo(w.y), o[3] = bf16_hi(w.y);
+                    };
 #pragma unroll
-                    for (int i = 0; i < CH; i++) {
-                        const int ch = q + 8 * i;
-                        x[i] = to_f32(kk[s * KE + ch]);
-                        const float u = ch < a.dim ? a.u[h * a.dim + ch] : 0.f;
-                        b = fmaf(to_f32(rr[s * KE + ch]) * u, x[i], b);
+                    for (int i = 0; i < C4; i++) {
+                        const int ch = 4 * (q + 8 * i);
+                        float r4[4];
+                        row4(kk + s * KE, i, x[i]);
+                        row4(rr + s * KE, i, r4);
+                        const float4 u4 = ch < a.dim ? *reinterpret_cast<const float4 *>(a.u + h * a.dim + ch) : make_float4(0.f, 0.f, 0.f, 0.f);
+                        b = fmaf(r4[0] * u4.x, x[i][0], b);
+                        b = fmaf(r4[1] * u4.y, x[i][1], b);
+                        b = fmaf(r4[2] * u4.z, x[i][2], b);
+                        b = fmaf(r4[3] * u4.w, x[i][3], b);
                     }
 #pragma unroll
                     for (int t = 0; t < 16; t++) {
                         float v = t == s ? b : 0.f;
                         if (t > s) {
 #pragma unroll
-                            for (int i = 0; i < CH; i++) {
-                                const int ch = q + 8 * i;
-                                v = fmaf(to_f32(rr[t * KE + ch]), x[i], v);
-                                x[i] *= ww[t * DP + ch];
+                            for (int i = 0; i < C4; i++) {
+                                float r4[4];
+                                row4(rr + t * KE, i, r4);
+                                const float4 w4 = *reinterpret_cast<const float4 *>(ww + t * DP + 4 * (q + 8 * i));
+                                v = fmaf(r4[0], x[i][0], v);
+                                v = fmaf(r4[1], x[i][1], v);
+                                v = fmaf(r4[2], x[i][2], v);
+                                v = fmaf(r4[3], x[i][3], v);
+                                x[i][0] *= w4.x;
+                                x[i][1] *= w4.y;
+                                x[i][2] *= w4.z;
+                                x[i][3] *= w4.w;
                             }
                         }
                         v += __shfl_xor_sync(0xffffffffu, v, 1);
