@@ -160,6 +160,8 @@ dense_gemv_kernel(const __grid_constant__ DenseVecJobs jobs) {
 // one's epilogue overlaps the other's matmul.  Warp 0 issues the copies, warp 1 the MMAs, warps 2-5
 // read the accumulators back.  Every wait is bounded; after a timeout the error flag is set, the
 // copies in flight are waited for and the tensor memory is freed.
+// grid = (token tiles, row tiles of all jobs): CTAs that run together share weight rows, so a weight matrix
+// larger than L2 still crosses DRAM once.
 constexpr int DG_TOK = 256, DG_ROWS = 128, DG_K = 64, DG_STAGES = 2, DG_THREADS = 192;
 constexpr uint32_t DG_X_BYTES = DG_TOK * 128, DG_W_BYTES = DG_ROWS * 128, DG_STAGE_BYTES = DG_X_BYTES + DG_W_BYTES;
 constexpr size_t DG_SMEM = (size_t)DG_STAGES * DG_STAGE_BYTES + 1024;
@@ -191,11 +193,11 @@ dense_gemm_kernel(const __grid_constant__ DenseGemmJobs jobs, const __grid_const
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     int js = 0;
     for (int i = 1; i < jobs.n; i++)
-        if ((int)blockIdx.x >= jobs.j[i].tile0) js = i;
+        if ((int)blockIdx.y >= jobs.j[i].tile0) js = i;
     const DenseGemmJob &job = jobs.j[js];
     const bool pair = job.pair != 0;
     const int rows = job.rows, seq = jobs.seq;
-    const int n0 = ((int)blockIdx.x - job.tile0) * (pair ? DG_ROWS / 2 : DG_ROWS), m0 = blockIdx.y * DG_TOK;
+    const int n0 = ((int)blockIdx.y - job.tile0) * (pair ? DG_ROWS / 2 : DG_ROWS), m0 = blockIdx.x * DG_TOK;
     const int KT = (job.cols + DG_K - 1) / DG_K;
     if (tid == 0) {
         for (int s = 0; s < DG_STAGES; s++) {

@@ -290,10 +290,9 @@ latent_attend_mma_kernel(const bf16 *__restrict__ qf, const bf16 *__restrict__ c
     bf16 *phi = reinterpret_cast<bf16 *>(lm_smem + L.phi), *plo = reinterpret_cast<bf16 *>(lm_smem + L.plo);
     constexpr int PE = LM_KEYS + 8, SE = LM_KEYS + 4;
     auto load_tile = [&](int i) {
-        const int k0 = lo + i * LM_KEYS, per = EP / 8;
         const uint32_t st = base + (uint32_t)(i & 1) * LM_KEYS * L.pitch;
-        for (int x = tid; x < LM_KEYS * per; x += LM_THREADS) {
-            const int r = x / per, q = x % per, key = k0 + r;
+        const int r = tid >> 2, key = lo + i * LM_KEYS + r;   // four threads walk along a row
+        for (int q = tid & 3; q < EP / 8; q += 4) {
             // the row's padding (up to ld) is never written by an append; what lies past E meets zero query columns, so it
             // only has to be finite: it is taken as zero
             const bool in = key < hi && q * 8 < E;
@@ -306,8 +305,8 @@ latent_attend_mma_kernel(const bf16 *__restrict__ qf, const bf16 *__restrict__ c
     const int n_tiles = (hi - lo + LM_KEYS - 1) / LM_KEYS;
     if (n_tiles > 0) {
         // query rows (pitch EP in memory), part of the first tile's copy group
-        for (int x = tid; x < 16 * (EP / 8); x += LM_THREADS) {
-            const int r = x / (EP / 8), q = x % (EP / 8);
+        const int r = tid >> 4;
+        for (int q = tid & 15; q < EP / 8; q += 16) {
             asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(base + L.q + (uint32_t)r * L.pitch + (uint32_t)q * 16u),
                          "l"(qf + ((size_t)t * d.heads + min(h0 + r, d.heads - 1)) * EP + q * 8), "r"(h0 + r < d.heads ? 16u : 0u)
                          : "memory");
@@ -458,24 +457,17 @@ latent_prefill_kernel(const __grid_constant__ LatentPrefillArgs a) {
     auto load_tile = [&](int t) {
         const int st = t & 1, key0 = t * LA_KEYS;
         if (a.vec) {
-            const int cn = d.dim / 8, cr = d.rot_dim / 8, cv = d.vdim / 8, per = cn + cr + cv;
-            for (int i = tid; i < LA_KEYS * per; i += LA_THREADS) {
-                const int r = i / per, c = i % per, key = key0 + r, kk = min(key, kv_len - 1);
-                const bf16 *src;
-                uint32_t dst;
-                if (c < cn) {
-                    src = a.kn + ((size_t)kk * d.heads + h) * d.dim + c * 8;
-                    dst = k_base + (uint32_t)(st * LA_KEYS + r) * kpitch + (uint32_t)c * 16u;
-                } else if (c < cn + cr) {
-                    src = a.kr + (size_t)kk * d.ld + (c - cn) * 8;
-                    dst = k_base + (uint32_t)(st * LA_KEYS + r) * kpitch + (uint32_t)c * 16u;
-                } else {
-                    src = a.v + ((size_t)kk * d.heads + h) * d.vdim + (c - cn - cr) * 8;
-                    dst = v_base + (uint32_t)(st * LA_KEYS + r) * vpitch + (uint32_t)(c - cn - cr) * 16u;
-                }
-                const uint32_t nbytes = key < kv_len ? 16u : 0u;
-                asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(nbytes) : "memory");
-            }
+            // four threads walk along a key's rows
+            const int r = tid >> 2, q0 = tid & 3, key = key0 + r, kk = min(key, kv_len - 1);
+            const uint32_t nbytes = key < kv_len ? 16u : 0u;
+            auto row = [&](uint32_t dst, const bf16 *src, int chunks) {
+                for (int c = q0; c < chunks; c += 4)
+                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst + (uint32_t)c * 16u), "l"(src + c * 8), "r"(nbytes) : "memory");
+            };
+            const uint32_t kdst = k_base + (uint32_t)(st * LA_KEYS + r) * kpitch;
+            row(kdst, a.kn + ((size_t)kk * d.heads + h) * d.dim, d.dim / 8);
+            row(kdst + (uint32_t)d.dim * 2u, a.kr + (size_t)kk * d.ld, d.rot_dim / 8);
+            row(v_base + (uint32_t)(st * LA_KEYS + r) * vpitch, a.v + ((size_t)kk * d.heads + h) * d.vdim, d.vdim / 8);
         } else {
             const int per = dk + d.vdim;
             for (int i = tid; i < LA_KEYS * per; i += LA_THREADS) {
@@ -520,6 +512,7 @@ latent_prefill_kernel(const __grid_constant__ LatentPrefillArgs a) {
         for (int j = 0; j < 8; j++) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
         // B fragments of two key tiles per ldmatrix: (keys 0-7, k 0-7), (keys 0-7, k 8-15), (keys 8-15, k 0-7), (keys 8-15, k 8-15)
         const uint32_t kb = k_st + (uint32_t)((mi >> 1) * 8 + mr) * kpitch + (uint32_t)(mi & 1) * 16u;
+#pragma unroll 4
         for (int kk = 0; kk < KS; kk++) {
             uint32_t af[4];
             lt_ldmatrix_x4(af, q_addr + (uint32_t)kk * 32u);

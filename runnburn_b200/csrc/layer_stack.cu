@@ -558,7 +558,7 @@ int LayerStack::matmul(cudaStream_t s, int n, const Mm *jobs, int n_jobs, int *e
             memcpy(&M.w[i], jobs[i].w->map, sizeof(PgTensorMap));
             if (j.pair) memcpy(&M.w2[i], jobs[i].w2->map, sizeof(PgTensorMap));
         }
-        RNB_CU(launch_k(dense_gemm_kernel, dim3((unsigned)tiles, (unsigned)((n + DG_TOK - 1) / DG_TOK)), dim3(DG_THREADS), DG_SMEM, s, J, M, err));
+        RNB_CU(launch_k(dense_gemm_kernel, dim3((unsigned)((n + DG_TOK - 1) / DG_TOK), (unsigned)tiles), dim3(DG_THREADS), DG_SMEM, s, J, M, err));
         return RNB_B200_OK;
     }
     DenseSimtJobs J;

@@ -292,32 +292,24 @@ linear_state_tile_kernel(const __grid_constant__ LinearChunkArgs a) {
         const uint32_t st = base + (uint32_t)(i & 1) * L.stage;
         const int t0 = t_begin + 16 * i;
         constexpr int CK = DP / 8, CWF = DP / 4;
-        const int cv = 2 * NW, per = (OUT ? 2 : 1) * CK + (CONST_W ? 0 : CWF) + cv;
-        for (int x = tid; x < 16 * per; x += nthr) {
-            const int t = x / per, tok = t0 + t, row = min(tok, t_end - 1);
-            int q = x % per;
+        // eight threads walk along a row; 256 threads put two such groups on each row
+        const int groups = nthr == 256 ? 2 : 1, q0 = (tid & 7) + (groups == 2 ? 8 * (tid >> 7) : 0), qs = 8 * groups;
+        for (int t = (groups == 2 ? tid & 127 : tid) >> 3; t < 16; t += nthr / (8 * groups)) {
+            const int tok = t0 + t;
+            const size_t row = (size_t)min(tok, t_end - 1);
             const bool in = tok < t_end;
-            if (q < CK) {
-                cp16(st + L.k + (uint32_t)t * L.kp + (uint32_t)q * 16u, kp + (size_t)row * ldk + min(q * 8, a.dim - 8), in && q * 8 < a.dim);
-                continue;
+            for (int q = q0; q < CK; q += qs) {
+                const bool ok = in && q * 8 < a.dim;
+                const int at = min(q * 8, a.dim - 8);
+                cp16(st + L.k + (uint32_t)t * L.kp + (uint32_t)q * 16u, kp + row * ldk + at, ok);
+                if (OUT) cp16(st + (uint32_t)t * L.kp + (uint32_t)q * 16u, rp + row * ldk + at, ok);
             }
-            q -= CK;
-            if (OUT) {
-                if (q < CK) {
-                    cp16(st + (uint32_t)t * L.kp + (uint32_t)q * 16u, rp + (size_t)row * ldk + min(q * 8, a.dim - 8), in && q * 8 < a.dim);
-                    continue;
-                }
-                q -= CK;
+            if (!CONST_W)
+                for (int q = q0; q < CWF; q += qs) cp16(st + L.w + (uint32_t)(t * DP + q * 4) * 4u, wp + row * ldk + min(q * 4, a.dim - 4), in && q * 4 < a.dim);
+            for (int q = q0; q < 2 * NW; q += qs) {
+                const int col = j0 + q * 8;
+                cp16(st + L.v + (uint32_t)t * L.vp + (uint32_t)q * 16u, vp + row * ldv + min(col, a.vdim - 8), in && col < a.vdim);
             }
-            if (!CONST_W) {
-                if (q < CWF) {
-                    cp16(st + L.w + (uint32_t)(t * DP + q * 4) * 4u, wp + (size_t)row * ldk + min(q * 4, a.dim - 4), in && q * 4 < a.dim);
-                    continue;
-                }
-                q -= CWF;
-            }
-            const int col = j0 + q * 8;
-            cp16(st + L.v + (uint32_t)t * L.vp + (uint32_t)q * 16u, vp + (size_t)row * ldv + min(col, a.vdim - 8), in && col < a.vdim);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -368,9 +360,17 @@ linear_state_tile_kernel(const __grid_constant__ LinearChunkArgs a) {
         bf16 *ahi = reinterpret_cast<bf16 *>(lt_smem + L.ahi), *alo = reinterpret_cast<bf16 *>(lt_smem + L.alo);
         constexpr int KE = DP + 8;
         if (CONST_W) {
-            for (int x = tid; x < 16 * DP; x += nthr) {
-                const int t = x / DP, ch = x % DP;
-                lt_split_store(khi + t * KE + ch, klo + t * KE + ch, t < nt ? to_f32(kk[t * KE + ch]) * pw[nt - 1 - t] : 0.f);
+            for (int x = tid; x < 16 * (DP / 8); x += nthr) {
+                const int t = x / (DP / 8), at = t * KE + x % (DP / 8) * 8;
+                const uint4 b = *reinterpret_cast<const uint4 *>(kk + at);
+                const float p = t < nt ? pw[nt - 1 - t] : 0.f;
+                uint4 hi, lo;
+                lt_split(bf16_lo(b.x) * p, bf16_hi(b.x) * p, hi.x, lo.x);
+                lt_split(bf16_lo(b.y) * p, bf16_hi(b.y) * p, hi.y, lo.y);
+                lt_split(bf16_lo(b.z) * p, bf16_hi(b.z) * p, hi.z, lo.z);
+                lt_split(bf16_lo(b.w) * p, bf16_hi(b.w) * p, hi.w, lo.w);
+                *reinterpret_cast<uint4 *>(khi + at) = hi;
+                *reinterpret_cast<uint4 *>(klo + at) = lo;
             }
             if (OUT && warp == 0) {
                 float q[2][4] = {};
@@ -396,21 +396,29 @@ linear_state_tile_kernel(const __grid_constant__ LinearChunkArgs a) {
             // decays before each token (for r) and after it (for k), channel by channel
             for (int x = tid; x < 2 * DP; x += nthr) {
                 const int ch = x % DP;
+                if (!OUT && x >= DP) break;
+                // everything is read before anything is written, so that the loads overlap
+                const bf16 *src = x < DP ? kk : rr;
+                float raw16[16], w16[16];
+#pragma unroll
+                for (int t = 0; t < 16; t++) {
+                    raw16[t] = to_f32(src[t * KE + ch]);
+                    w16[t] = t < nt ? ww[t * DP + ch] : 1.f;
+                }
+                float p = 1.f;
                 if (x < DP) {
-                    float p = 1.f;
 #pragma unroll
                     for (int t = 15; t >= 0; t--) {
-                        lt_split_store(khi + t * KE + ch, klo + t * KE + ch, to_f32(kk[t * KE + ch]) * p);
-                        if (t < nt) p *= ww[t * DP + ch];
+                        lt_split_store(khi + t * KE + ch, klo + t * KE + ch, raw16[t] * p);
+                        p *= w16[t];
                     }
                     sD[ch] = p;
                     if (!OUT) sP[ch] *= p;
-                } else if (OUT) {
-                    float p = 1.f;
+                } else {
 #pragma unroll
                     for (int t = 0; t < 16; t++) {
-                        lt_split_store(rhi + t * KE + ch, rlo + t * KE + ch, to_f32(rr[t * KE + ch]) * p);
-                        if (t < nt) p *= ww[t * DP + ch];
+                        lt_split_store(rhi + t * KE + ch, rlo + t * KE + ch, raw16[t] * p);
+                        p *= w16[t];
                     }
                 }
             }
@@ -438,30 +446,38 @@ linear_state_tile_kernel(const __grid_constant__ LinearChunkArgs a) {
                         b = fmaf(r4[2] * u4.z, x[i][2], b);
                         b = fmaf(r4[3] * u4.w, x[i][3], b);
                     }
+                    float v[16];
 #pragma unroll
                     for (int t = 0; t < 16; t++) {
-                        float v = t == s ? b : 0.f;
+                        v[t] = t == s ? b : 0.f;
                         if (t > s) {
 #pragma unroll
                             for (int i = 0; i < C4; i++) {
                                 float r4[4];
                                 row4(rr + t * KE, i, r4);
                                 const float4 w4 = *reinterpret_cast<const float4 *>(ww + t * DP + 4 * (q + 8 * i));
-                                v = fmaf(r4[0], x[i][0], v);
-                                v = fmaf(r4[1], x[i][1], v);
-                                v = fmaf(r4[2], x[i][2], v);
-                                v = fmaf(r4[3], x[i][3], v);
+                                v[t] = fmaf(r4[0], x[i][0], v[t]);
+                                v[t] = fmaf(r4[1], x[i][1], v[t]);
+                                v[t] = fmaf(r4[2], x[i][2], v[t]);
+                                v[t] = fmaf(r4[3], x[i][3], v[t]);
                                 x[i][0] *= w4.x;
                                 x[i][1] *= w4.y;
                                 x[i][2] *= w4.z;
                                 x[i][3] *= w4.w;
                             }
                         }
-                        v += __shfl_xor_sync(0xffffffffu, v, 1);
-                        v += __shfl_xor_sync(0xffffffffu, v, 2);
-                        v += __shfl_xor_sync(0xffffffffu, v, 4);
-                        if (q == (t & 7)) lt_split_store(ahi + t * 24 + s, alo + t * 24 + s, v);
                     }
+                    // sums over the eight lanes; lane q ends up with rows q and q + 8
+                    float keep[2] = {0.f, 0.f};
+#pragma unroll
+                    for (int t = 0; t < 16; t++) {
+                        v[t] += __shfl_xor_sync(0xffffffffu, v[t], 1);
+                        v[t] += __shfl_xor_sync(0xffffffffu, v[t], 2);
+                        v[t] += __shfl_xor_sync(0xffffffffu, v[t], 4);
+                        if (q == (t & 7)) keep[t >> 3] = v[t];
+                    }
+#pragma unroll
+                    for (int i = 0; i < 2; i++) lt_split_store(ahi + (q + 8 * i) * 24 + s, alo + (q + 8 * i) * 24 + s, keep[i]);
                 }
             }
         }
