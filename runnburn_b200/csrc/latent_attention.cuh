@@ -39,10 +39,10 @@ latent_append_kernel(const float *__restrict__ y, const float *__restrict__ w, f
     latent_append_row<CT>(y + (size_t)blockIdx.x * (d.rank + d.rot_dim), w, eps, d, rot, *pos0 + (int)blockIdx.x, cache, red);
 }
 
-// grid = (heads + 1, tokens, ceil(rank / 512)), 512 threads.  Head h: qf[t][h] = [W_uk_h^T q | rotated q];
-// the extra column of CTAs appends the token's cache row.  64 threads hold 8 columns each, 8 groups of them
+// grid = (heads + 1, tokens, ceil(rank / 128)), 512 threads.  Head h: qf[t][h] = [W_uk_h^T q | rotated q];
+// the extra column of CTAs appends the token's cache row.  16 threads hold 8 columns each, 32 groups of them
 // share the key dimensions; the first rows of W_uk are loaded ahead of the dependency wait.
-// Dynamic shared memory: dim + 8 * 512 floats.
+// Dynamic shared memory: dim + 32 * 128 floats.
 struct LatentPrepareArgs {
     const float *q, *y, *w;      // [tokens][heads * (dim + rot)], [tokens][rank + rot], [rank]
     const bf16 *uk;              // [heads * dim][rank]
@@ -54,7 +54,7 @@ struct LatentPrepareArgs {
     LatentDims d;
     Rotation rot;
 };
-constexpr int LP_THREADS = 512, LP_COLS = 512, LP_BATCH = 8;
+constexpr int LP_THREADS = 512, LP_COLS = 128, LP_GROUPS = LP_THREADS / (LP_COLS / 8), LP_BATCH = 4;
 template <class CT, class QT>
 RNB_GLOBAL void __launch_bounds__(LP_THREADS)
 latent_prepare_kernel(const __grid_constant__ LatentPrepareArgs a) {
@@ -70,14 +70,14 @@ latent_prepare_kernel(const __grid_constant__ LatentPrepareArgs a) {
         return;
     }
     float *sq = lp_smem, *sr = lp_smem + ((d.dim + 3) & ~3);
-    const int grp = tid >> 6, c = blockIdx.z * LP_COLS + (tid & 63) * 8;
+    const int grp = tid / (LP_COLS / 8), cl = tid % (LP_COLS / 8) * 8, c = blockIdx.z * LP_COLS + cl;
     const bool vec = d.rank % 8 == 0, in = c < d.rank;
     const bf16 *w = a.uk + (size_t)h * d.dim * d.rank + c;
     uint4 b[LP_BATCH];
     auto fetch = [&](int i0) {
 #pragma unroll
         for (int k = 0; k < LP_BATCH; k++) {
-            const int i = i0 + 8 * k + grp;
+            const int i = i0 + LP_GROUPS * k + grp;
             b[k] = vec && in && i < d.dim ? ldg_nc_u4(w + (size_t)i * d.rank) : make_uint4(0u, 0u, 0u, 0u);
         }
     };
@@ -100,11 +100,11 @@ latent_prepare_kernel(const __grid_constant__ LatentPrepareArgs a) {
         return;
     }
     float acc[8] = {};
-    for (int i0 = 0; i0 < d.dim; i0 += 8 * LP_BATCH) {
+    for (int i0 = 0; i0 < d.dim; i0 += LP_GROUPS * LP_BATCH) {
         if (i0) fetch(i0);
 #pragma unroll
         for (int k = 0; k < LP_BATCH; k++) {
-            const int i = i0 + 8 * k + grp;
+            const int i = i0 + LP_GROUPS * k + grp;
             const float qv = i < d.dim ? sq[i] : 0.f;
             const uint32_t p[4] = {b[k].x, b[k].y, b[k].z, b[k].w};
 #pragma unroll
@@ -115,20 +115,22 @@ latent_prepare_kernel(const __grid_constant__ LatentPrepareArgs a) {
         }
     }
 #pragma unroll
-    for (int e = 0; e < 8; e++) sr[grp * LP_COLS + (tid & 63) * 8 + e] = acc[e];
+    for (int e = 0; e < 8; e++) sr[grp * LP_COLS + cl + e] = acc[e];
     __syncthreads();
     const int e = blockIdx.z * LP_COLS + tid;
-    if (e < d.rank) {
+    if (tid < LP_COLS && e < d.rank) {
         float s = 0.f;
-#pragma unroll
-        for (int k = 0; k < 8; k++) s += sr[k * LP_COLS + tid];
+#pragma unroll 8
+        for (int k = 0; k < LP_GROUPS; k++) s += sr[k * LP_COLS + tid];
         out[e] = from_f32<QT>(s);
     }
 }
 
-// Keys [lo, hi) of chunk c when n keys are split over `chunks`.
+// n keys split over at most `chunks` CTAs: at least 128 keys each (a shorter chunk costs more in merging than it
+// saves), in whole units of 32.
+__device__ __forceinline__ int latent_chunk_keys(int n, int chunks) { return max(128, ((n + chunks - 1) / chunks + 31) & ~31); }
 __device__ __forceinline__ void latent_chunk_range(int n, int chunks, int c, int &lo, int &hi) {
-    const int per = (n + chunks - 1) / chunks;
+    const int per = latent_chunk_keys(n, chunks);
     lo = min(c * per, n);
     hi = min(lo + per, n);
 }
@@ -148,6 +150,7 @@ latent_attend_kernel(const float *__restrict__ qf, const CT *__restrict__ cache,
     const int h = blockIdx.y, t = blockIdx.z, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, E = d.rank + d.rot_dim;
     int lo, hi;
     latent_chunk_range(*pos0 + t + 1, gridDim.x, blockIdx.x, lo, hi);
+    if (lo == hi) return;   // the merge knows how many chunks hold keys
     const float *q = qf + ((size_t)t * d.heads + h) * E;
     float qv[NQ], o[NQ], m = -INFINITY, l = 0.f;
 #pragma unroll
@@ -189,11 +192,12 @@ latent_attend_kernel(const float *__restrict__ qf, const CT *__restrict__ cache,
 }
 
 // act[t][h * vdim + v] = W_uv_h (merged latent result).  grid = (heads, tokens, row blocks), 512 threads: four
-// groups of 128 share the chunks, 16 warps share the rows.  Dynamic shared memory 5 * rank4 + chunks floats.
+// groups of 128 share the chunks, 16 warps share the rows.  Dynamic shared memory 5 * rank4 + max_chunks floats.
 constexpr int LO_THREADS = 512;
 template <class HT>
 RNB_GLOBAL void __launch_bounds__(LO_THREADS)
-latent_output_kernel(const float *__restrict__ part, const bf16 *__restrict__ uv, const LatentDims d, int chunks, int rows_per_cta, HT *__restrict__ act) {
+latent_output_kernel(const float *__restrict__ part, const bf16 *__restrict__ uv, const LatentDims d, int max_chunks, const int *__restrict__ pos0, int rows_per_cta,
+                     HT *__restrict__ act) {
     extern __shared__ __align__(16) float lo_smem[];
     __shared__ float s_inv;
     pdl_launch_dependents();
@@ -202,7 +206,8 @@ latent_output_kernel(const float *__restrict__ part, const bf16 *__restrict__ uv
     if (gridDim.y == 1) prefetch_l2(uv + ((size_t)h * d.vdim + v0) * d.rank, (size_t)(v1 - v0) * d.rank * 2, threadIdx.x, LO_THREADS);
     pdl_wait();
     float *ol = lo_smem, *grp = lo_smem + R4, *f = grp + 4 * R4;
-    const float *p = part + ((size_t)t * d.heads + h) * chunks * ld;
+    const float *p = part + ((size_t)t * d.heads + h) * max_chunks * ld;
+    const int keys = *pos0 + t + 1, per = latent_chunk_keys(keys, max_chunks), chunks = (keys + per - 1) / per;
     if (warp == 0) {
         float M = -INFINITY, L = 0.f;
         for (int c = lane; c < chunks; c += 32) M = fmaxf(M, p[(size_t)c * ld + d.rank]);
@@ -286,6 +291,7 @@ latent_attend_mma_kernel(const bf16 *__restrict__ qf, const bf16 *__restrict__ c
     const int EP = (int)(L.pitch / 2) - 8, ld = latent_part_ld(d.rank);
     int lo, hi;
     latent_chunk_range(*pos0 + t + 1, gridDim.x, blockIdx.x, lo, hi);
+    if (lo == hi) return;
     float *ss = reinterpret_cast<float *>(lm_smem + L.s), *s_m = reinterpret_cast<float *>(lm_smem + L.stat), *s_l = s_m + 16, *s_c = s_l + 16;
     bf16 *phi = reinterpret_cast<bf16 *>(lm_smem + L.phi), *plo = reinterpret_cast<bf16 *>(lm_smem + L.plo);
     constexpr int PE = LM_KEYS + 8, SE = LM_KEYS + 4;

@@ -145,8 +145,7 @@ int LayerStack::init(const rnb_b200_mixer_cfg *layers) {
     }
     RNB_TRY(alloc((void **)&counters_, (size_t)max_heads * 4));
     RNB_CU(cudaMemset(counters_, 0, (size_t)max_heads * 4));
-    // at least one tile of keys per chunk; more chunks mean more CTAs but more partial results to merge
-    attend_chunks_ = std::max(1, std::min((c.max_ctx + 63) / 64, 48));
+    attend_chunks_ = std::max(1, std::min((c.max_ctx + 127) / 128, 64));
     return RNB_B200_OK;
 }
 
@@ -799,7 +798,7 @@ int LayerStack::mixer_latent(cudaStream_t s, int n, StackScratch &b, StackLayer 
         const bool mma = !cfg.f32_math && latent_mma_fits(d);
         a.qf = b.qf, a.qld = mma ? (m.kv_rank + m.rot_dim + 31) & ~31 : m.kv_rank + m.rot_dim, a.cache = R.cache, a.pos0 = pos_dev, a.eps = cfg.norm_eps, a.d = d, a.rot = rot;
         const dim3 grid((unsigned)(m.heads + 1), (unsigned)n, (unsigned)((m.kv_rank + LP_COLS - 1) / LP_COLS)), pb(LP_THREADS);
-        const size_t psmem = ((size_t)((m.dim + 3) & ~3) + 8 * LP_COLS) * 4;
+        const size_t psmem = ((size_t)((m.dim + 3) & ~3) + LP_GROUPS * LP_COLS) * 4;
         const int chunks = n <= SMALL ? attend_chunks_ : 1;
         if (cfg.f32_math) {
             RNB_CU(launch_k(latent_prepare_kernel<float, float>, grid, pb, psmem, s, a));
@@ -811,12 +810,12 @@ int LayerStack::mixer_latent(cudaStream_t s, int n, StackScratch &b, StackLayer 
             else RNB_TRY(launch_latent_attend<bf16>(s, b.qf, (const bf16 *)R.cache, d, m.scale, pos_dev, b.part, n, chunks));
         }
         // a few CTAs per head share its value rows
-        const int split = n <= SMALL ? std::max(1, std::min((m.vdim + 15) / 16, sm_ / std::max(1, m.heads * n))) : 1;
+        const int split = n <= SMALL ? std::max(1, std::min((m.vdim + 15) / 16, 2 * sm_ / std::max(1, m.heads * n))) : 1;
         const int rows = (m.vdim + split - 1) / split;
         const dim3 og((unsigned)m.heads, (unsigned)n, (unsigned)split);
         const size_t smem = ((size_t)5 * ((m.kv_rank + 3) & ~3) + chunks) * 4;
-        if (nb) RNB_CU(launch_k(latent_output_kernel<bf16>, og, dim3(LO_THREADS), smem, s, (const float *)b.part, reinterpret_cast<const bf16 *>(L.uv.w), d, chunks, rows, (bf16 *)b.act));
-        else RNB_CU(launch_k(latent_output_kernel<float>, og, dim3(LO_THREADS), smem, s, (const float *)b.part, reinterpret_cast<const bf16 *>(L.uv.w), d, chunks, rows, (float *)b.act));
+        if (nb) RNB_CU(launch_k(latent_output_kernel<bf16>, og, dim3(LO_THREADS), smem, s, (const float *)b.part, reinterpret_cast<const bf16 *>(L.uv.w), d, chunks, pos_dev, rows, (bf16 *)b.act));
+        else RNB_CU(launch_k(latent_output_kernel<float>, og, dim3(LO_THREADS), smem, s, (const float *)b.part, reinterpret_cast<const bf16 *>(L.uv.w), d, chunks, pos_dev, rows, (float *)b.act));
         return RNB_B200_OK;
     }
     RNB_CU(launch_k(latent_append_kernel<bf16>, dim3((unsigned)n), dim3(128), 0, s, (const float *)b.z, (const float *)L.dkv_norm, cfg.norm_eps, d, rot, pos_dev, (bf16 *)R.cache));
