@@ -49,10 +49,10 @@ def punisun_shape(n_layer: int, width: int, n_ff: int, vocab: int, loop=(0, 0, 1
     (128 + 64 query dimensions, latent of 512)."""
     h64, h128 = width // 64, width // 128
     wkv = dict(mixer="wkv", heads=h64, dim=64, decay_rank=64, n_ff=n_ff)
-    ret = dict(mixer="retention", heads=h128, dim=128, vdim=128, rot=dict(dims=128, base=1e6),
+    ret = dict(mixer="retention", heads=h128, dim=128, vdim=128, rot=dict(dims=128, base=1e4),
                decay=[1.0 - 2.0 ** (-5.0 - 7.0 * i / max(h128 - 1, 1)) for i in range(h128)], n_ff=n_ff)
     lat = dict(mixer="latent_attention", heads=h128, dim=128, vdim=128, rot_dim=64, kv_rank=512, scale=192 ** -0.5,
-               rot=dict(dims=64, base=5e4, scaling=dict(factor=8.0, original=4096.0, fast=32.0, slow=1.0)), n_ff=n_ff)
+               rot=dict(dims=64, base=1e5, scaling=dict(factor=4.0, original=2048.0, fast=24.0, slow=1.5)), n_ff=n_ff)
     return dict(stack=[(wkv, ret, wkv, lat)[i % 4] for i in range(n_layer)], n_layer=n_layer, hidden=width, vocab=vocab, loop=loop)
 
 

@@ -1,5 +1,5 @@
-"""Reader of safetensors files: an 8-byte little-endian header length, the JSON header
-(name -> dtype, shape, data_offsets), then the data.  The file is mapped, not copied."""
+"""Reader of safetensors files.  The JSON header follows its own length (u64, little-endian) and gives
+each tensor's dtype, shape and place in the data behind it.  The file is mapped, not copied."""
 from __future__ import annotations
 
 import json

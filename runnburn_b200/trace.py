@@ -3,7 +3,8 @@
     python -m runnburn_b200.trace --model DIR --dtype bfloat16|float32 --out DIR --max-tokens N
 
 Steps come on standard input, one JSON object a line:
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}
+    {"step": 4, "entries": [{"id": "q7", "tokens": [12, 9], "want": [1]}], "end": ["q7"]}
+`want` are places among the step's tokens; a request named in `end` is over after the step.
 For a step that wants logits, OUT/<step>.f32 receives them ([wanted, vocab], little-endian f32); after
 every step 'done <step>' is printed.  One sequence is live at a time: a request runs until it ends.
 """
