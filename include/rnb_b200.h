@@ -549,42 +549,68 @@ int rnb_b200_decoder_prefill(rnb_b200_decoder *d, const uint32_t *tokens, int n,
 int rnb_b200_decoder_read_logits(rnb_b200_decoder *d, float *out, size_t n);
 
 /* ---- mixed stacks: a decoder whose layers are listed one by one --------------------------------
- * Each layer names its mixer (token mixing) and may have a dense gated feed-forward
- * W_down(gelu_tanh(W_gate h) * W_up h).  Sublayers are normed on both sides,
- * x <- x + residual_mult * norm_b(sublayer(norm_a(x))), norms are x / sqrt(mean x^2 + eps) * (1 + w),
- * and the LM head is the embedding table.  Layers loop_start .. loop_stop - 1 run loop_times times in
- * a row, each pass with its own state; the embedding output is added to x before every pass but the
- * first.  Weights are bf16 matrices; the residual, norms, rotations, attention weights and recurrent
- * states are f32.  f32_math: activations and all matrix products in f32 too (no tensor cores).
+ * Each layer names its mixer (token mixing; up to two side by side, whose outputs are added) and may have
+ * a dense gated feed-forward W_down(act(W_gate h) * W_up h).  Two forms of a layer:
+ *   sandwich: sublayers normed on both sides, x <- x + residual_mult * norm_b(sublayer(norm_a(x)));
+ *   parallel: one norm, x <- x + residual_mult * (mixers(norm(x)) + feed_forward(norm(x))).
+ * Norms are x / sqrt(mean x^2 + eps) * (1 + w), or (parallel layers) the layer norm with weight and bias.
+ * The LM head is the embedding table, embed_scale multiplies the embedding rows only.  Layers
+ * loop_start .. loop_stop - 1 run loop_times times in a row, each pass with its own state; the embedding
+ * output is added to x before every pass but the first.  A layer may use another layer's weights with a
+ * state of its own.  Weights are bf16 matrices; the residual, norms, rotations, attention weights and
+ * recurrent states are f32.  f32_math: activations and all matrix products in f32 too (no tensor cores).
  * The functions of the decoder above work on it: step, step_dev, prefill, read_logits, time_steps, ... */
 #define RNB_B200_MIXER_WKV 1              /* RWKV-style time mixing: heads x dim, low-rank decay */
 #define RNB_B200_MIXER_RETENTION 2        /* heads x dim keys, heads x vdim values, decay per head */
 #define RNB_B200_MIXER_LATENT_ATTENTION 3 /* latent of kv_rank plus a shared rotated key part of rot_dim */
+#define RNB_B200_MIXER_GLA 4              /* gated linear attention: heads x dim keys, heads x vdim values, low-rank decay per key channel */
+#define RNB_B200_MIXER_ATTENTION 5        /* softmax attention: heads x dim queries on kv_heads keys and values, optional window, norm, gate */
+#define RNB_B200_MIXER_DELTA 6            /* gated delta rule: kv_heads x dim queries and keys, heads x vdim values, short convolutions */
+#define RNB_B200_BLOCK_SANDWICH 0
+#define RNB_B200_BLOCK_PARALLEL 1
+#define RNB_B200_NORM_RMS 0               /* x / sqrt(mean x^2 + eps) * (1 + w) */
+#define RNB_B200_NORM_LAYER 1             /* (x - mean) / sqrt(variance + eps) * w + b */
+#define RNB_B200_ACT_GELU_TANH 0
+#define RNB_B200_ACT_SILU 1
+#define RNB_B200_ROTATION_YARN 1
+#define RNB_B200_ROTATION_LINEAR 2
 typedef struct {
     int32_t dims;        /* rotated dimensions of a head's vector (0: none) */
     int32_t interleaved; /* pairs (2i, 2i + 1); otherwise (i, i + dims / 2) */
     double base;
-    int32_t scaled;      /* YaRN: the four values below apply */
+    int32_t scaled;      /* 0 none; YaRN: the four values below apply; linear: frequencies divided by factor */
     double factor, original, fast, slow;
 } rnb_b200_rotation;
 typedef struct {
     int32_t mixer;
     int32_t heads, dim, vdim, rot_dim, kv_rank;
     int32_t decay_rank;  /* time mixing: rows of the low-rank decay matrix (0: as the tensor has) */
-    float scale;         /* latent attention: multiplies the scores */
+    float scale;         /* attention, latent attention: multiplies the scores */
     rnb_b200_rotation rot;
     const double *decay; /* retention: [heads], copied */
-    int32_t n_ff;        /* 0: no feed-forward */
+    int32_t n_ff;        /* 0: no feed-forward (of a layer's first record) */
+    int32_t kv_heads;    /* attention: key/value heads; delta: query/key heads; each serves heads / kv_heads heads */
+    int32_t window;      /* attention: keys that a query sees, its own included (0: all before it) */
+    int32_t qk_norm;     /* attention: rotated queries and keys are divided by their root mean square per head */
+    int32_t head_gate;   /* attention: the output of a head times sigmoid(W_g h)_head */
+    int32_t conv;        /* delta: taps of the convolutions, the current token's included */
+    float tau;           /* gated linear attention: decay sigmoid(z)^(1 / tau) */
+    float out_scale;     /* multiplies the mixer's output */
+    int32_t join;        /* 1: one more mixer of the layer of the record before */
+    int32_t weights_of;  /* >= 0: this layer uses that (earlier) layer's tensors; -1: its own */
+    const char *prefix;  /* tensor names after "l<i>."; null: "mix." */
 } rnb_b200_mixer_cfg;
 typedef struct {
-    int32_t n_layer, width, vocab, max_ctx;
+    int32_t n_layer, width, vocab, max_ctx;    /* n_layer: records (a layer with two mixers has two) */
     int32_t loop_start, loop_stop, loop_times; /* loop_times <= 1: every layer runs once */
     float norm_eps, residual_mult;
     int32_t f32_math;
+    int32_t block, norm, act;                  /* RNB_B200_BLOCK_*, _NORM_*, _ACT_* */
+    float embed_scale;
 } rnb_b200_stack_cfg;
 int rnb_b200_decoder_create_stack(const rnb_b200_stack_cfg *cfg, const rnb_b200_mixer_cfg *layers, rnb_b200_decoder **out);
 /* One weight by name ("embed", "final.norm", "l3.mix.q", "l0.mlp.down", ...), row-major [out, in];
- * type: GGML id, 30 = BF16 (matrices and vectors) or 0 = F32 (vectors only). */
+ * type: GGML id, 30 = BF16 (matrices and vectors) or 0 = F32 (vectors, convolution taps). */
 int rnb_b200_decoder_set_tensor(rnb_b200_decoder *d, const char *name, uint32_t type, const void *data, const uint64_t *shape, uint32_t n_dims);
 /* Forget the sequence: the next position is 0.  A step or prefill at position 0 does this by itself. */
 int rnb_b200_decoder_reset(rnb_b200_decoder *d);

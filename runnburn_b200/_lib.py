@@ -52,7 +52,11 @@ class GgufTensorInfo(C.Structure):
                 ("offset", C.c_uint64), ("n_elements", C.c_uint64), ("n_bytes", C.c_uint64), ("data", C.c_void_p)]
 
 
-MIXER_WKV, MIXER_RETENTION, MIXER_LATENT_ATTENTION = 1, 2, 3
+MIXER_WKV, MIXER_RETENTION, MIXER_LATENT_ATTENTION, MIXER_GLA, MIXER_ATTENTION, MIXER_DELTA = 1, 2, 3, 4, 5, 6
+BLOCK_SANDWICH, BLOCK_PARALLEL = 0, 1
+NORM_RMS, NORM_LAYER = 0, 1
+ACT_GELU_TANH, ACT_SILU = 0, 1
+ROTATION_YARN, ROTATION_LINEAR = 1, 2
 TYPE_F32, TYPE_BF16 = 0, 30
 
 
@@ -63,12 +67,15 @@ class Rotation(C.Structure):
 
 class MixerCfg(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "dim", "vdim", "rot_dim", "kv_rank", "decay_rank")] + \
-               [("scale", C.c_float), ("rot", Rotation), ("decay", C.POINTER(C.c_double)), ("n_ff", C.c_int32)]
+               [("scale", C.c_float), ("rot", Rotation), ("decay", C.POINTER(C.c_double)), ("n_ff", C.c_int32)] + \
+               [(n, C.c_int32) for n in ("kv_heads", "window", "qk_norm", "head_gate", "conv")] + \
+               [("tau", C.c_float), ("out_scale", C.c_float), ("join", C.c_int32), ("weights_of", C.c_int32), ("prefix", C.c_char_p)]
 
 
 class StackCfg(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("n_layer", "width", "vocab", "max_ctx", "loop_start", "loop_stop", "loop_times")] + \
-               [("norm_eps", C.c_float), ("residual_mult", C.c_float), ("f32_math", C.c_int32)]
+               [("norm_eps", C.c_float), ("residual_mult", C.c_float), ("f32_math", C.c_int32)] + \
+               [(n, C.c_int32) for n in ("block", "norm", "act")] + [("embed_scale", C.c_float)]
 
 
 class LayerWeights(C.Structure):

@@ -7,7 +7,7 @@
 //                           16-byte aligned, which the tiled copies cannot describe)
 //
 // All accumulate in f32.  Matrices that go out together share a launch (jobs).  A job with w2 is a
-// gate + up pair: the result is gelu(w x) * (w2 x), gelu in its tanh form.
+// gate + up pair: the result is act(w x) * (w2 x), act the tanh form of gelu or silu.
 #pragma once
 #include <cuda_bf16.h>
 
@@ -39,14 +39,25 @@ __device__ __forceinline__ float silu_f32(float z) { return z / (1.0f + expf(-z)
 __device__ __forceinline__ float bf16_lo(uint32_t w) { return __uint_as_float(w << 16); }
 __device__ __forceinline__ float bf16_hi(uint32_t w) { return __uint_as_float(w & 0xffff0000u); }
 
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
+constexpr int ACT_GELU_TANH = 0, ACT_SILU = 1;
+__device__ __forceinline__ float gate_act(int act, float z) { return act == ACT_SILU ? silu_f32(z) : gelu_tanh_f32(z); }
+__device__ __forceinline__ float gate_act_fast(int act, float z) { return act == ACT_SILU ? silu_fast(z) : gelu_tanh_fast(z); }
+
+// A decay in (0, 1) from its projection x: exp(-exp(x)), or sigmoid(x)^inv_tau taken through the logarithm of the sigmoid.
+constexpr int DECAY_EXP = 0, DECAY_SIGMOID_ROOT = 1;
+__device__ __forceinline__ float decay_of(int kind, float x, float inv_tau) {
+    return kind == DECAY_SIGMOID_ROOT ? expf((fminf(x, 0.f) - log1pf(expf(-fabsf(x)))) * inv_tau) : expf(-expf(x));
+}
+
 constexpr int DENSE_MAX_JOBS = 6;
 
 // ---- few tokens ---------------------------------------------------------------------------------
 struct DenseVecJob {
     const bf16 *w, *w2;   // [rows][cols]; w2: the up half of a gate + up pair
-    const float *x;       // token t at x + t * cols
-    float *y;             // token t at y + t * rows
-    int rows, cols, cta0, vec;   // vec: rows of 16-byte aligned weights (cols % 8 == 0)
+    const float *x;       // token t at x + t * ldx
+    float *y;             // token t at y + t * ldy
+    int rows, cols, ldx, ldy, cta0, vec, act;   // vec: rows of 16-byte aligned weights (cols % 8 == 0) and inputs
 };
 struct DenseVecJobs {
     DenseVecJob j[DENSE_MAX_JOBS];
@@ -101,8 +112,8 @@ dense_gemv_kernel(const __grid_constant__ DenseVecJobs jobs) {
                 const uint32_t p[4] = {c0[u].x, c0[u].y, c0[u].z, c0[u].w}, q[4] = {c1[u].x, c1[u].y, c1[u].z, c1[u].w};
 #pragma unroll
                 for (int t = 0; t < T; t++) {
-                    const float4 xa = *reinterpret_cast<const float4 *>(job.x + (size_t)t * cols + k);
-                    const float4 xb = *reinterpret_cast<const float4 *>(job.x + (size_t)t * cols + k + 4);
+                    const float4 xa = *reinterpret_cast<const float4 *>(job.x + (size_t)t * job.ldx + k);
+                    const float4 xb = *reinterpret_cast<const float4 *>(job.x + (size_t)t * job.ldx + k + 4);
                     const float xv[8] = {xa.x, xa.y, xa.z, xa.w, xb.x, xb.y, xb.z, xb.w};
 #pragma unroll
                     for (int e = 0; e < 4; e++) {
@@ -120,7 +131,7 @@ dense_gemv_kernel(const __grid_constant__ DenseVecJobs jobs) {
             const float p = to_f32(w0[k]), q = to_f32(w1[k]);
 #pragma unroll
             for (int t = 0; t < T; t++) {
-                const float xv = job.x[(size_t)t * cols + k];
+                const float xv = job.x[(size_t)t * job.ldx + k];
                 a0[t] = fmaf(p, xv, a0[t]);
                 a1[t] = fmaf(q, xv, a1[t]);
             }
@@ -141,9 +152,9 @@ dense_gemv_kernel(const __grid_constant__ DenseVecJobs jobs) {
     if (lane == 0 && live && part == 0) {
 #pragma unroll
         for (int t = 0; t < T; t++) {
-            float *y = job.y + (size_t)t * rows + r0;
+            float *y = job.y + (size_t)t * job.ldy + r0;
             if (pair) {
-                y[0] = gelu_tanh_f32(a0[t]) * a1[t];
+                y[0] = gate_act(job.act, a0[t]) * a1[t];
             } else {
                 y[0] = a0[t];
                 if (two) y[1] = a1[t];
@@ -168,8 +179,9 @@ constexpr size_t DG_SMEM = (size_t)DG_STAGES * DG_STAGE_BYTES + 1024;
 
 struct DenseGemmJob {
     void *y;             // [seq][ld]
-    const float *decay_bias;   // not null: y = exp(-exp(w x + bias[row]))
-    int rows, cols, tile0, out_bf16, pair, ld;
+    const float *decay_bias;   // not null: y = decay_of(w x + bias[row])
+    float inv_tau;
+    int rows, cols, tile0, out_bf16, pair, ld, act, decay_kind;
 };
 struct DenseGemmJobs {
     DenseGemmJob j[DENSE_MAX_JOBS];
@@ -282,7 +294,7 @@ dense_gemm_kernel(const __grid_constant__ DenseGemmJobs jobs, const __grid_const
                     for (int i = 0; i < 16; i++) {
                         const int tok = m0 + cc * 32 + t_lo + i;
                         const float z = gs[lane * 33 + t_lo + i];
-                        const float a = (job.out_bf16 ? gelu_tanh_fast(z) : gelu_tanh_f32(z)) * us[lane * 33 + t_lo + i];
+                        const float a = (job.out_bf16 ? gate_act_fast(job.act, z) : gate_act(job.act, z)) * us[lane * 33 + t_lo + i];
                         if (tok < seq) {
                             if (job.out_bf16) dg_store<bf16>(job.y, (size_t)tok * job.ld + row, a);
                             else dg_store<float>(job.y, (size_t)tok * job.ld + row, a);
@@ -299,7 +311,7 @@ dense_gemm_kernel(const __grid_constant__ DenseGemmJobs jobs, const __grid_const
                     if (job.decay_bias) {
                         const float b = job.decay_bias[row];
 #pragma unroll
-                        for (int i = 0; i < 32; i++) v[i] = __float_as_uint(expf(-expf(__uint_as_float(v[i]) + b)));
+                        for (int i = 0; i < 32; i++) v[i] = __float_as_uint(decay_of(job.decay_kind, __uint_as_float(v[i]) + b, job.inv_tau));
                     }
 #pragma unroll
                     for (int i = 0; i < 32; i++) {
@@ -326,7 +338,7 @@ struct DenseSimtJob {
     const bf16 *w, *w2;
     const void *x;       // [seq][ldx] of XT
     void *y;             // [seq][ld]
-    int rows, cols, tile0, out_bf16, ldx, ld;
+    int rows, cols, tile0, out_bf16, ldx, ld, act;
 };
 struct DenseSimtJobs {
     DenseSimtJob j[DENSE_MAX_JOBS];
@@ -384,7 +396,7 @@ dense_gemm_simt_kernel(const __grid_constant__ DenseSimtJobs jobs) {
         for (int j = 0; j < 4; j++) {
             const int tok = m0 + ty * 4 + i, row = n0 + tx * 4 + j;
             if (tok >= jobs.seq || row >= job.rows) continue;
-            const float v = pair ? gelu_tanh_f32(a[i][j]) * b[i][j] : a[i][j];
+            const float v = pair ? gate_act(job.act, a[i][j]) * b[i][j] : a[i][j];
             if (job.out_bf16) dg_store<bf16>(job.y, (size_t)tok * job.ld + row, v);
             else dg_store<float>(job.y, (size_t)tok * job.ld + row, v);
         }

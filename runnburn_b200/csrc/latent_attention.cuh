@@ -5,11 +5,9 @@
 // query moves into the latent space once (latent_prepare_kernel, which also appends the tokens' cache
 // rows), attention runs over the cache rows themselves (latent_attend_kernel, split over the context),
 // and the merged latent result is taken to the value space (latent_output_kernel).
-// Prompts in bf16: keys and values are expanded by matmuls and latent_prefill_kernel runs causal
-// attention on tensor cores.
+// Prompts in bf16: keys and values are expanded by matmuls and causal_attention_kernel runs over them.
 #pragma once
-#include "layer_glue.cuh"
-#include "mma_bf16.cuh"
+#include "causal_attention.cuh"
 
 namespace rnb {
 
@@ -191,13 +189,13 @@ latent_attend_kernel(const float *__restrict__ qf, const CT *__restrict__ cache,
     if (threadIdx.x == 0) out[d.rank] = M, out[d.rank + 1] = L;
 }
 
-// act[t][h * vdim + v] = W_uv_h (merged latent result).  grid = (heads, tokens, row blocks), 512 threads: four
+// act[t * lda + h * vdim + v] = mul * W_uv_h (merged latent result).  grid = (heads, tokens, row blocks), 512 threads: four
 // groups of 128 share the chunks, 16 warps share the rows.  Dynamic shared memory 5 * rank4 + max_chunks floats.
 constexpr int LO_THREADS = 512;
 template <class HT>
 RNB_GLOBAL void __launch_bounds__(LO_THREADS)
 latent_output_kernel(const float *__restrict__ part, const bf16 *__restrict__ uv, const LatentDims d, int max_chunks, const int *__restrict__ pos0, int rows_per_cta,
-                     HT *__restrict__ act) {
+                     HT *__restrict__ act, int lda, float mul) {
     extern __shared__ __align__(16) float lo_smem[];
     __shared__ float s_inv;
     pdl_launch_dependents();
@@ -253,7 +251,7 @@ latent_output_kernel(const float *__restrict__ part, const bf16 *__restrict__ uv
             for (int e = lane; e < d.rank; e += 32) s = fmaf(to_f32(w[e]), ol[e], s);
         }
         s = warp_sum(s);
-        if (lane == 0) act[((size_t)t * d.heads + h) * d.vdim + v] = from_f32<HT>(s);
+        if (lane == 0) act[(size_t)t * lda + h * d.vdim + v] = from_f32<HT>(s * mul);
     }
 }
 
@@ -413,193 +411,6 @@ latent_attend_mma_kernel(const bf16 *__restrict__ qf, const bf16 *__restrict__ c
     if (tid < 16 && h0 + tid < d.heads) {
         out[tid * hs + d.rank] = s_m[tid];
         out[tid * hs + d.rank + 1] = s_l[tid];
-    }
-}
-
-// ---- prompts: causal attention over expanded keys and values on tensor cores ---------------------
-constexpr int LA_ROWS = 128, LA_KEYS = 64, LA_THREADS = 256;
-__host__ __device__ inline int la_pad16(int n) { return (n + 15) & ~15; }
-__host__ inline size_t latent_prefill_smem(const LatentDims &d, int dvp) {
-    return 2 * ((size_t)(LA_ROWS + 2 * LA_KEYS) * (la_pad16(d.dim + d.rot_dim) + 8) + (size_t)2 * LA_KEYS * (dvp + 8));
-}
-struct LatentPrefillArgs {
-    const bf16 *q, *kn, *kr, *v;   // [tokens][heads][dim + rot] (rotated), [keys][heads][dim], cache + rank, [keys][heads][vdim]
-    bf16 *act;                     // [tokens][heads * vdim]
-    const int *pos0;
-    float scale;
-    int tokens, vec;               // vec: every row piece is 16-byte aligned and a multiple of 8 elements
-    LatentDims d;
-};
-// grid = (ceil(tokens / 128), heads), 256 threads; warp w owns queries 16w .. 16w + 15 of the CTA's 128.
-// Keys come in tiles of 64, double-buffered; the weights enter the value product as bf16 hi + lo parts.
-// DVJ: 8-column tiles of the value dimension (vdim <= 8 DVJ).
-template <int DVJ>
-RNB_GLOBAL void __launch_bounds__(LA_THREADS, 1)
-latent_prefill_kernel(const __grid_constant__ LatentPrefillArgs a) {
-    extern __shared__ __align__(128) uint8_t la_smem[];
-    pdl_launch_dependents();
-    pdl_wait();
-    const LatentDims &d = a.d;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y;
-    const int dk = d.dim + d.rot_dim, dkp = la_pad16(dk), KS = dkp / 16;
-    constexpr int DVP = 8 * DVJ;
-    const uint32_t kpitch = (uint32_t)(dkp + 8) * 2, vpitch = (uint32_t)(DVP + 8) * 2;
-    bf16 *qs = reinterpret_cast<bf16 *>(la_smem);
-    bf16 *ks = qs + (size_t)LA_ROWS * (dkp + 8), *vs = ks + (size_t)2 * LA_KEYS * (dkp + 8);
-    const uint32_t q_base = smem_u32(qs), k_base = smem_u32(ks), v_base = smem_u32(vs);
-    const int i0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * LA_ROWS;   // long rows first
-    const int pos0 = *a.pos0, kv_len = pos0 + a.tokens;
-    const int n_keys = min(kv_len, pos0 + i0 + LA_ROWS), n_tiles = (n_keys + LA_KEYS - 1) / LA_KEYS;
-    const bf16 zero = from_f32<bf16>(0.f);
-    // queries, and zeros in the padding columns of every buffer (the copies below never touch those)
-    for (int i = tid; i < LA_ROWS * (dkp + 8); i += LA_THREADS) {
-        const int r = i / (dkp + 8), c = i % (dkp + 8);
-        qs[i] = c < dk && i0 + r < a.tokens ? a.q[((size_t)(i0 + r) * d.heads + h) * dk + c] : zero;
-    }
-    if (dkp > dk)
-        for (int i = tid; i < 2 * LA_KEYS * (dkp - dk); i += LA_THREADS) ks[(size_t)(i / (dkp - dk)) * (dkp + 8) + dk + i % (dkp - dk)] = zero;
-    if (DVP > d.vdim)
-        for (int i = tid; i < 2 * LA_KEYS * (DVP - d.vdim); i += LA_THREADS) vs[(size_t)(i / (DVP - d.vdim)) * (DVP + 8) + d.vdim + i % (DVP - d.vdim)] = zero;
-    auto load_tile = [&](int t) {
-        const int st = t & 1, key0 = t * LA_KEYS;
-        if (a.vec) {
-            // four threads walk along a key's rows
-            const int r = tid >> 2, q0 = tid & 3, key = key0 + r, kk = min(key, kv_len - 1);
-            const uint32_t nbytes = key < kv_len ? 16u : 0u;
-            auto row = [&](uint32_t dst, const bf16 *src, int chunks) {
-                for (int c = q0; c < chunks; c += 4)
-                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst + (uint32_t)c * 16u), "l"(src + c * 8), "r"(nbytes) : "memory");
-            };
-            const uint32_t kdst = k_base + (uint32_t)(st * LA_KEYS + r) * kpitch;
-            row(kdst, a.kn + ((size_t)kk * d.heads + h) * d.dim, d.dim / 8);
-            row(kdst + (uint32_t)d.dim * 2u, a.kr + (size_t)kk * d.ld, d.rot_dim / 8);
-            row(v_base + (uint32_t)(st * LA_KEYS + r) * vpitch, a.v + ((size_t)kk * d.heads + h) * d.vdim, d.vdim / 8);
-        } else {
-            const int per = dk + d.vdim;
-            for (int i = tid; i < LA_KEYS * per; i += LA_THREADS) {
-                const int r = i / per, c = i % per, key = key0 + r;
-                const bool in = key < kv_len;
-                if (c < dk)
-                    ks[(size_t)(st * LA_KEYS + r) * (dkp + 8) + c] =
-                        !in ? zero : c < d.dim ? a.kn[((size_t)key * d.heads + h) * d.dim + c] : a.kr[(size_t)key * d.ld + c - d.dim];
-                else
-                    vs[(size_t)(st * LA_KEYS + r) * (DVP + 8) + c - dk] = in ? a.v[((size_t)key * d.heads + h) * d.vdim + c - dk] : zero;
-            }
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    };
-    load_tile(0);
-    const int g = lane >> 2, tq = lane & 3, mi = lane >> 3, mr = lane & 7;
-    int qi[2], pos[2];
-    bool live[2];
-#pragma unroll
-    for (int e = 0; e < 2; e++) {
-        qi[e] = i0 + warp * 16 + g + 8 * e;
-        live[e] = qi[e] < a.tokens;
-        pos[e] = live[e] ? pos0 + qi[e] : kv_len - 1;   // rows past the end see everything and are never stored
-    }
-    float o[DVJ][4], m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
-#pragma unroll
-    for (int j = 0; j < DVJ; j++) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
-    const float sl2 = a.scale * 1.4426950408889634f;
-    // A fragments: matrices (rows 0-7, k 0-7), (rows 8-15, k 0-7), (rows 0-7, k 8-15), (rows 8-15, k 8-15)
-    const uint32_t q_addr = q_base + (uint32_t)(warp * 16 + (mi & 1) * 8 + mr) * kpitch + (uint32_t)(mi >> 1) * 16u;
-    for (int t = 0; t < n_tiles; t++) {
-        if (t + 1 < n_tiles) {
-            load_tile(t + 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        __syncthreads();
-        const uint32_t k_st = k_base + (uint32_t)(t & 1) * LA_KEYS * kpitch, v_st = v_base + (uint32_t)(t & 1) * LA_KEYS * vpitch;
-        float s[8][4];
-#pragma unroll
-        for (int j = 0; j < 8; j++) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
-        // B fragments of two key tiles per ldmatrix: (keys 0-7, k 0-7), (keys 0-7, k 8-15), (keys 8-15, k 0-7), (keys 8-15, k 8-15)
-        const uint32_t kb = k_st + (uint32_t)((mi >> 1) * 8 + mr) * kpitch + (uint32_t)(mi & 1) * 16u;
-#pragma unroll 4
-        for (int kk = 0; kk < KS; kk++) {
-            uint32_t af[4];
-            lt_ldmatrix_x4(af, q_addr + (uint32_t)kk * 32u);
-#pragma unroll
-            for (int jp = 0; jp < 4; jp++) {
-                uint32_t b[4];
-                lt_ldmatrix_x4(b, kb + (uint32_t)(jp * 16) * kpitch + (uint32_t)kk * 32u);
-                lt_mma(s[2 * jp], af, b[0], b[1]);
-                lt_mma(s[2 * jp + 1], af, b[2], b[3]);
-            }
-        }
-        const int key0 = t * LA_KEYS + 2 * tq;
-        const bool need_mask = t * LA_KEYS + LA_KEYS - 1 > min(pos[0], pos[1]);
-        float mx[2] = {-INFINITY, -INFINITY};
-#pragma unroll
-        for (int j = 0; j < 8; j++)
-#pragma unroll
-            for (int e = 0; e < 4; e++) {
-                float x = s[j][e] * sl2;
-                if (need_mask && key0 + j * 8 + (e & 1) > pos[e >> 1]) x = -INFINITY;
-                s[j][e] = x;
-                mx[e >> 1] = fmaxf(mx[e >> 1], x);
-            }
-        float corr[2], m_use[2], rs[2] = {0.f, 0.f};
-#pragma unroll
-        for (int e = 0; e < 2; e++) {
-            mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 1));
-            mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 2));
-            const float mn = fmaxf(m_run[e], mx[e]);
-            m_use[e] = mn == -INFINITY ? 0.f : mn;
-            corr[e] = exp2f(m_run[e] - m_use[e]);
-            m_run[e] = mn;
-        }
-        uint32_t ph[4][4], pl[4][4];
-#pragma unroll
-        for (int j = 0; j < 8; j++) {
-            const float p0 = exp2f(s[j][0] - m_use[0]), p1 = exp2f(s[j][1] - m_use[0]);
-            const float p2 = exp2f(s[j][2] - m_use[1]), p3 = exp2f(s[j][3] - m_use[1]);
-            rs[0] += p0 + p1;
-            rs[1] += p2 + p3;
-            lt_split(p0, p1, ph[j >> 1][2 * (j & 1)], pl[j >> 1][2 * (j & 1)]);
-            lt_split(p2, p3, ph[j >> 1][2 * (j & 1) + 1], pl[j >> 1][2 * (j & 1) + 1]);
-        }
-#pragma unroll
-        for (int e = 0; e < 2; e++) {
-            rs[e] += __shfl_xor_sync(0xffffffffu, rs[e], 1);
-            rs[e] += __shfl_xor_sync(0xffffffffu, rs[e], 2);
-            l_run[e] = fmaf(l_run[e], corr[e], rs[e]);
-        }
-#pragma unroll
-        for (int j = 0; j < DVJ; j++) {
-            o[j][0] *= corr[0];
-            o[j][1] *= corr[0];
-            o[j][2] *= corr[1];
-            o[j][3] *= corr[1];
-        }
-#pragma unroll
-        for (int kk = 0; kk < 4; kk++) {
-            const uint32_t vb = v_st + (uint32_t)(kk * 16 + (mi & 1) * 8 + mr) * vpitch + (uint32_t)(mi >> 1) * 16u;
-#pragma unroll
-            for (int jp = 0; jp < DVJ / 2; jp++) {
-                uint32_t b[4];
-                lt_ldmatrix_x4_trans(b, vb + (uint32_t)jp * 32u);
-                lt_mma(o[2 * jp], ph[kk], b[0], b[1]);
-                lt_mma(o[2 * jp], pl[kk], b[0], b[1]);
-                lt_mma(o[2 * jp + 1], ph[kk], b[2], b[3]);
-                lt_mma(o[2 * jp + 1], pl[kk], b[2], b[3]);
-            }
-        }
-        __syncthreads();
-    }
-#pragma unroll
-    for (int e = 0; e < 2; e++) {
-        if (!live[e]) continue;
-        const float inv = 1.0f / l_run[e];
-        bf16 *dst = a.act + ((size_t)qi[e] * d.heads + h) * d.vdim;
-#pragma unroll
-        for (int j = 0; j < DVJ; j++)
-#pragma unroll
-            for (int x = 0; x < 2; x++)
-                if (8 * j + 2 * tq + x < d.vdim) dst[8 * j + 2 * tq + x] = from_f32<bf16>(o[j][2 * e + x] * inv);
     }
 }
 

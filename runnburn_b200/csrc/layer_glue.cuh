@@ -25,31 +25,32 @@ __device__ __forceinline__ void prefetch_l2(const void *p, size_t bytes, int tid
 
 // grid = tokens.  x and (when kept for later passes) emb: [tokens][width] f32
 RNB_GLOBAL void __launch_bounds__(256)
-dense_embed_kernel(const bf16 *__restrict__ table, const uint32_t *__restrict__ token, int width, float *__restrict__ x, float *__restrict__ emb) {
+dense_embed_kernel(const bf16 *__restrict__ table, const uint32_t *__restrict__ token, int width, float scale, float *__restrict__ x, float *__restrict__ emb) {
     pdl_launch_dependents();
     pdl_wait();
     const size_t row = (size_t)token[blockIdx.x] * width, o = (size_t)blockIdx.x * width;
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
-        const float v = to_f32(table[row + i]);
+        const float v = to_f32(table[row + i]) * scale;
         x[o + i] = v;
         if (emb) emb[o + i] = v;
     }
 }
 
 // The end of one sublayer and the start of the next in one pass over the residual rows:
-//   x <- x + mult * (y / rms(y)) * (1 + wb) + emb     (y, emb: may be null)
+//   x <- x + mult * (y / rms(y)) * (1 + wb) + emb     (y, emb: may be null; wb null: x + mult * y + emb)
 //   h <- (x / rms(x)) * (1 + wn)                      (wn null: stop at x)
+//   or, with `center`, the layer norm  h <- (x - mean) / sqrt(mean (x - mean)^2 + eps) * wn + bn
 // With mu [n_mix][width] the output is n_mix token-shifted mixes  h + (h' - h) * mu_s  instead, stream s
 // at h + s * tokens * width; h' is the previous token's h, which the CTA recomputes for the row before its
 // first (from x_in, so x_out must be another buffer when there are several CTAs) or takes from shift_in
 // for the step's first token.  The last token's h goes to shift_out.
 // grid = ceil(tokens / rows_per_cta); dynamic shared memory (mu ? 2 : 1) * width floats.
 struct ResidualNormArgs {
-    const float *x_in, *y, *wb, *emb, *wn, *mu, *shift_in;
+    const float *x_in, *y, *wb, *emb, *wn, *bn, *mu, *shift_in;
     float *x_out, *shift_out;
     void *h;
     float mult, eps;
-    int width, tokens, rows_per_cta, n_mix;
+    int width, tokens, rows_per_cta, n_mix, center;
 };
 template <class HT, int V>   // V: elements per access (4 when width % 4 == 0, else 1)
 RNB_GLOBAL void __launch_bounds__(1024)
@@ -60,6 +61,7 @@ residual_norm_kernel(const __grid_constant__ ResidualNormArgs a) {
     if (gridDim.x == 1) {
         prefetch_l2(a.wb, (size_t)a.width * 4, threadIdx.x, blockDim.x);
         prefetch_l2(a.wn, (size_t)a.width * 4, threadIdx.x, blockDim.x);
+        prefetch_l2(a.bn, (size_t)a.width * 4, threadIdx.x, blockDim.x);
         prefetch_l2(a.mu, (size_t)a.width * 4 * a.n_mix, threadIdx.x, blockDim.x);
     }
     pdl_wait();
@@ -73,7 +75,7 @@ residual_norm_kernel(const __grid_constant__ ResidualNormArgs a) {
         const size_t row = (size_t)t * D;
         const bool mine = t >= t0;
         float ry = 0.f;
-        if (a.y) {
+        if (a.y && a.wb) {
             float ss = 0.f;
             for (int i = threadIdx.x * V; i < D; i += step) {
                 const Vec y = *reinterpret_cast<const Vec *>(a.y + row + i);
@@ -86,9 +88,15 @@ residual_norm_kernel(const __grid_constant__ ResidualNormArgs a) {
         for (int i = threadIdx.x * V; i < D; i += step) {
             Vec x = *reinterpret_cast<const Vec *>(a.x_in + row + i);
             if (a.y) {
-                const Vec y = *reinterpret_cast<const Vec *>(a.y + row + i), w = *reinterpret_cast<const Vec *>(a.wb + i);
+                const Vec y = *reinterpret_cast<const Vec *>(a.y + row + i);
+                if (a.wb) {
+                    const Vec w = *reinterpret_cast<const Vec *>(a.wb + i);
 #pragma unroll
-                for (int e = 0; e < V; e++) x.v[e] += a.mult * (y.v[e] * ry * (1.0f + w.v[e]));
+                    for (int e = 0; e < V; e++) x.v[e] += a.mult * (y.v[e] * ry * (1.0f + w.v[e]));
+                } else {
+#pragma unroll
+                    for (int e = 0; e < V; e++) x.v[e] = fmaf(a.mult, y.v[e], x.v[e]);
+                }
             }
             if (a.emb) {
                 const Vec z = *reinterpret_cast<const Vec *>(a.emb + row + i);
@@ -98,15 +106,30 @@ residual_norm_kernel(const __grid_constant__ ResidualNormArgs a) {
             if (mine && (a.y || a.emb || a.x_out != a.x_in)) *reinterpret_cast<Vec *>(a.x_out + row + i) = x;
             *reinterpret_cast<Vec *>(cur + i) = x;
 #pragma unroll
-            for (int e = 0; e < V; e++) ss = fmaf(x.v[e], x.v[e], ss);
+            for (int e = 0; e < V; e++) ss = a.center ? ss + x.v[e] : fmaf(x.v[e], x.v[e], ss);
         }
         if (!a.wn) continue;
+        float mean = 0.f;
+        if (a.center) {
+            mean = block_sum(ss, red) / (float)D;
+            ss = 0.f;
+            for (int i = threadIdx.x * V; i < D; i += step) {
+                const Vec c = *reinterpret_cast<const Vec *>(cur + i);   // this thread's own elements
+#pragma unroll
+                for (int e = 0; e < V; e++) ss = fmaf(c.v[e] - mean, c.v[e] - mean, ss);
+            }
+        }
         const float rx = 1.0f / sqrtf(block_sum(ss, red) / (float)D + a.eps);
         for (int i = threadIdx.x * V; i < D; i += step) {
             Vec c = *reinterpret_cast<const Vec *>(cur + i);   // this thread's own elements
             const Vec w = *reinterpret_cast<const Vec *>(a.wn + i);
 #pragma unroll
-            for (int e = 0; e < V; e++) c.v[e] = c.v[e] * rx * (1.0f + w.v[e]);
+            for (int e = 0; e < V; e++) c.v[e] = a.center ? (c.v[e] - mean) * rx * w.v[e] : c.v[e] * rx * (1.0f + w.v[e]);
+            if (a.bn) {
+                const Vec b = *reinterpret_cast<const Vec *>(a.bn + i);
+#pragma unroll
+                for (int e = 0; e < V; e++) c.v[e] += b.v[e];
+            }
             if (a.mu) {
                 Vec p;
                 if (t == 0) p = *reinterpret_cast<const Vec *>(a.shift_in + i);
@@ -131,20 +154,26 @@ residual_norm_kernel(const __grid_constant__ ResidualNormArgs a) {
     }
 }
 
-// Norm of selected residual rows (the final norm of the positions whose logits are wanted).
+// Norm of selected residual rows (the final norm of the positions whose logits are wanted): with b the
+// layer norm of weight w and bias b, without it the root-mean-square norm of weight 1 + w.
 // rows null: row blockIdx.x itself.  grid = rows, dynamic shared memory none.
 template <class HT>
 RNB_GLOBAL void __launch_bounds__(512)
-norm_rows_kernel(const float *__restrict__ x, const int *__restrict__ rows, const float *__restrict__ w, float eps, int width, HT *__restrict__ h) {
+norm_rows_kernel(const float *__restrict__ x, const int *__restrict__ rows, const float *__restrict__ w, const float *__restrict__ b, float eps, int width,
+                 HT *__restrict__ h) {
     __shared__ float red[32];
     pdl_launch_dependents();
     pdl_wait();
     const float *xs = x + (size_t)(rows ? rows[blockIdx.x] : (int)blockIdx.x) * width;
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) ss = fmaf(xs[i], xs[i], ss);
+    float mean = 0.f, ss = 0.f;
+    if (b) {
+        for (int i = threadIdx.x; i < width; i += blockDim.x) mean += xs[i];
+        mean = block_sum(mean, red) / (float)width;
+    }
+    for (int i = threadIdx.x; i < width; i += blockDim.x) ss = fmaf(xs[i] - mean, xs[i] - mean, ss);
     const float r = 1.0f / sqrtf(block_sum(ss, red) / (float)width + eps);
     HT *hs = h + (size_t)blockIdx.x * width;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) hs[i] = from_f32<HT>(xs[i] * r * (1.0f + w[i]));
+    for (int i = threadIdx.x; i < width; i += blockDim.x) hs[i] = from_f32<HT>(b ? (xs[i] - mean) * r * w[i] + b[i] : xs[i] * r * (1.0f + w[i]));
 }
 
 // ---- rotary positions ---------------------------------------------------------------------------
@@ -205,38 +234,49 @@ rotate_heads_kernel(const __grid_constant__ RotateArgs a) {
         }
 }
 
-// act = (o / rms(o over the head)) * w * silu(g); w null: 1.  `lanes` (a power of two up to 32) per
-// (token, head), V elements per access (4 when vdim % 4 == 0, else 1).
-template <class GT, class HT, int V>
+// act = (o / rms(o over the head)) * w * silu(g) * mul; w null: 1, else `w_head` elements from one head's to the
+// next (0: shared by the heads).  `lanes` (a power of two up to 32) per (token, head), V elements per
+// access (4 when vdim and the row strides are multiples of 4, else 1).
+struct HeadNormGateArgs {
+    const float *o, *w;      // [tokens][heads][vdim]
+    const void *g;           // token t's rows at g + t * ldg, act + t * lda
+    void *act;
+    size_t units;            // tokens * heads
+    float eps, mul;
+    int heads, vdim, lanes, w_head, ldg, lda;
+};
+template <class HT, int V>
 RNB_GLOBAL void __launch_bounds__(256)
-head_norm_gate_kernel(const float *__restrict__ o, const float *__restrict__ w, const GT *__restrict__ g, float eps, size_t units, int heads, int vdim, int lanes,
-                      HT *__restrict__ act) {
+head_norm_gate_kernel(const __grid_constant__ HeadNormGateArgs a) {
     pdl_launch_dependents();
     pdl_wait();
     struct alignas(4 * V) Vec { float v[V]; };
-    struct alignas(sizeof(GT) * V) GVec { GT v[V]; };
     struct alignas(sizeof(HT) * V) HVec { HT v[V]; };
+    const int lanes = a.lanes, vdim = a.vdim;
     const size_t unit = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) / lanes;
     const int l = threadIdx.x & (lanes - 1);
-    const bool in = unit < units;
-    const size_t at = (in ? unit : 0) * vdim;
-    const int hw = (int)((in ? unit : 0) % heads) * vdim;
+    const bool in = unit < a.units;
+    const size_t u = in ? unit : 0, t = u / a.heads;
+    const int h = (int)(u % a.heads);
+    const float *o = a.o + u * vdim, *w = a.w ? a.w + (size_t)h * a.w_head : nullptr;
     float ss = 0.f;
     for (int j = l * V; j < vdim; j += lanes * V) {
-        const Vec x = *reinterpret_cast<const Vec *>(o + at + j);
+        const Vec x = *reinterpret_cast<const Vec *>(o + j);
 #pragma unroll
         for (int e = 0; e < V; e++) ss = fmaf(x.v[e], x.v[e], ss);
     }
     for (int d = 1; d < lanes; d <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
-    const float r = 1.0f / sqrtf(ss / (float)vdim + eps);
+    const float r = a.mul / sqrtf(ss / (float)vdim + a.eps);
     if (!in) return;
+    const HT *g = reinterpret_cast<const HT *>(a.g) + t * a.ldg + (size_t)h * vdim;
+    HT *act = reinterpret_cast<HT *>(a.act) + t * a.lda + (size_t)h * vdim;
     for (int j = l * V; j < vdim; j += lanes * V) {
-        const Vec x = *reinterpret_cast<const Vec *>(o + at + j);
-        const GVec y = *reinterpret_cast<const GVec *>(g + at + j);
+        const Vec x = *reinterpret_cast<const Vec *>(o + j);
+        const HVec y = *reinterpret_cast<const HVec *>(g + j);
         HVec out;
 #pragma unroll
-        for (int e = 0; e < V; e++) out.v[e] = from_f32<HT>(x.v[e] * r * (w ? w[hw + j + e] : 1.0f) * silu_f32(to_f32(y.v[e])));
-        *reinterpret_cast<HVec *>(act + at + j) = out;
+        for (int e = 0; e < V; e++) out.v[e] = from_f32<HT>(x.v[e] * r * (w ? w[j + e] : 1.0f) * silu_f32(to_f32(y.v[e])));
+        *reinterpret_cast<HVec *>(act + j) = out;
     }
 }
 

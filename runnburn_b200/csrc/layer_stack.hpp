@@ -1,5 +1,5 @@
-// Layers of a mixed stack (RWKV-style time mixing, retention, latent attention; dense gated feed-forward):
-// weights, per-run state and the launches of a step.  The decoder (decoder.inc) owns the step itself -
+// Layers of a mixed stack (RWKV-style time mixing, retention, latent attention, gated linear attention, window
+// attention, gated delta rule; dense gated feed-forward): weights, per-run state and the launches of a step.  The decoder (decoder.inc) owns the step itself -
 // token and position hand-over, graphs, LM-head argmax, timing - and calls in here for the layers.
 #pragma once
 #include <string>
@@ -16,21 +16,40 @@ struct DenseMat {
     bool tiled = false;                            // map is valid: rows are 16-byte aligned
 };
 
-struct StackLayer {
+// A mixer's weights.  Time mixing, retention and latent attention project through one matrix per tensor; the
+// others through `in` (their tensors' rows one after the other, at in_at, each padded to 8 rows) and, where
+// an f32 result is wanted, `aux`.
+struct StackMixer {
     rnb_b200_mixer_cfg c;
+    std::string prefix;
     std::vector<float> decay_host;
-    float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr;
-    DenseMat r, k, v, g, w1, w2, w2x /* [w2 | w2] */, q, dkv, uk, uv, o, gate, up, down;
-    float *mu = nullptr, *w0 = nullptr, *u = nullptr, *head_norm = nullptr, *dkv_norm = nullptr, *decay = nullptr;
+    DenseMat r, k, v, g, w1, w2, w2x /* [w2 | w2] */, q, dkv, uk, uv, in, aux;
+    int in_at[4] = {}, in_rows = 0, aux_rows = 0;
+    int act_at = 0, act_cols = 0;      // the output's columns in the input of the layer's output matrix
+    float *mu = nullptr, *w0 = nullptr, *u = nullptr, *head_norm = nullptr, *dkv_norm = nullptr, *decay = nullptr, *conv = nullptr, *a_log = nullptr, *dt = nullptr;
     const void *rot_table = nullptr;   // float2 [max_ctx][dims / 2]
 };
 
+struct StackLayer {
+    std::vector<StackMixer> mixers;
+    int n_ff = 0, weights_of = -1;
+    int ff_at = 0, out_cols = 0;       // parallel layers: the feed-forward shares the output matrix, from column ff_at on
+    float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr;
+    DenseMat out, gate, up, down;      // out: [width][out_cols], the mixers' output projections (and down) side by side
+    bool shifts() const { return mixers[0].c.mixer == RNB_B200_MIXER_WKV; }
+};
+
+struct MixerState {
+    float *state = nullptr, *shift = nullptr, *shift_out = nullptr;   // recurrent state, last normed input
+    void *cache = nullptr;                                           // latent rows [max_ctx][ld]; keys [ring][kv_heads * dim]
+    void *values = nullptr;                                          // values [ring][kv_heads * vdim]
+    float *conv_ring = nullptr;                                      // last inputs of the short convolutions
+};
 // One execution of a layer in a step; a looped layer has one per pass, each with its own state.
 struct LayerRun {
-    int layer = 0;
+    int layer = 0;                     // whose weights
     bool add_embedding = false;
-    float *state = nullptr, *shift = nullptr, *shift_out = nullptr;   // recurrent state, last normed input
-    void *cache = nullptr;                                           // latent rows [max_ctx][ld]
+    std::vector<MixerState> m;
 };
 
 struct StackScratch {
@@ -38,8 +57,10 @@ struct StackScratch {
     float *x[2] = {nullptr, nullptr}, *emb = nullptr, *y = nullptr, *z = nullptr, *w = nullptr, *o = nullptr, *qf = nullptr, *part = nullptr, *starts = nullptr,
           *decays = nullptr, *logits = nullptr;
     uint16_t *th = nullptr;   // tanh of the low-rank decay input as bf16 hi + lo
-    void *h = nullptr, *p[4] = {nullptr, nullptr, nullptr, nullptr}, *act = nullptr;
-    uint16_t *kn = nullptr, *vx = nullptr;
+    void *h = nullptr, *p[4] = {nullptr, nullptr, nullptr, nullptr}, *act = nullptr, *qn = nullptr;
+    float *aux[2] = {nullptr, nullptr};
+    uint16_t *kn = nullptr, *vx = nullptr, *cq = nullptr, *ck = nullptr, *cv = nullptr;
+    uint8_t *rec = nullptr;
     int *rows = nullptr;
     uint32_t *tok = nullptr;
     std::vector<void *> allocs;
@@ -79,6 +100,7 @@ private:
         float **vec = nullptr;
         size_t vec_off = 0, vec_total = 0;   // where in the vector's buffer, and its size
         int64_t rows = 0, cols = 0;          // cols 0: a vector of `rows` values; -1: taken from the tensor
+        int64_t row0 = 0, col0 = 0, all_rows = 0, all_cols = 0;   // all_rows > 0: a block of a larger matrix, zeros between the blocks
         float synth_mean = 0.f, synth_sigma = 0.f;
         bool set = false;
     };
@@ -88,22 +110,40 @@ private:
         size_t ldx;
         void *y;
         bool f32_out;
-        const float *decay_bias = nullptr;
+        size_t ldy = 0;                      // 0: rows
+        const float *decay_bias = nullptr;   // y: decays of the mixer `decay`
+        const rnb_b200_mixer_cfg *decay = nullptr;
     };
     explicit LayerStack(const rnb_b200_stack_cfg &c) : cfg(c) {}
     int init(const rnb_b200_mixer_cfg *layers);
     int alloc(void **p, size_t bytes, std::vector<void *> *owner = nullptr);
     int alloc_scratch(StackScratch &b, int cap);
     int rotation_table(const rnb_b200_rotation &r, const void **out);
-    int place(Slot &slot, int64_t rows, int64_t cols);
+    int place(cudaStream_t s, Slot &slot, int64_t rows, int64_t cols);
     void slots_of_layer(int i);
     int matmul(cudaStream_t s, int n, const Mm *jobs, int n_jobs, int *err);
-    int boundary(cudaStream_t s, int n, StackScratch &b, int &cur, const float *y, const float *wb, bool emb, const float *wn, const StackLayer *shift, LayerRun *run);
-    int mixer_linear(cudaStream_t s, int n, StackScratch &b, StackLayer &L, LayerRun &R, const int *pos_dev, int *err);
-    int mixer_latent(cudaStream_t s, int n, StackScratch &b, StackLayer &L, LayerRun &R, const int *pos_dev, int pos_host, int *err);
+    int in_jobs(int n, StackScratch &b, StackLayer &L, Mm *jobs);   // the projections that read the layer's normed input
+    Mm out_job(StackScratch &b, StackLayer &L);
+    int boundary(cudaStream_t s, int n, StackScratch &b, int &cur, const float *y, const float *wb, bool emb, const float *wn, const float *bn, const StackLayer *shift, LayerRun *run);
+    int run_mixer(cudaStream_t s, int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev, int pos_host, int *err);
+    int mixer_linear(cudaStream_t s, int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev, int *err);
+    int mixer_latent(cudaStream_t s, int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev, int pos_host, int *err);
+    int mixer_attention(cudaStream_t s, int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev);
+    int mixer_delta(cudaStream_t s, int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev);
+    int head_norm_gate(cudaStream_t s, int n, StackScratch &b, const StackLayer &L, const StackMixer &M, const void *g, int ldg);
+    void *act_of(StackScratch &b, const StackMixer &M, int n) const { return (char *)b.act + (size_t)M.act_at * (narrow(n) ? 2 : 4); }
+    int attention_ring(const rnb_b200_mixer_cfg &m) const;
+    int attention_chunks(const rnb_b200_mixer_cfg &m) const;
+    bool attention_tiled(const rnb_b200_mixer_cfg &m) const;
+    bool parallel() const { return cfg.block == RNB_B200_BLOCK_PARALLEL; }
+    template <class Fn>
+    void each_mixer(Fn fn) const {
+        for (const StackLayer &L : layers_)
+            for (const StackMixer &M : L.mixers) fn(L, M);
+    }
     bool narrow(int n) const { return n > SMALL && !cfg.f32_math; }   // bf16 activations
-    bool absorbed(const StackLayer &L, int n) const;
-    int latent_ld(const StackLayer &L) const { return (L.c.kv_rank + L.c.rot_dim + 7) & ~7; }
+    bool absorbed(const rnb_b200_mixer_cfg &m, int n) const;
+    static int latent_ld(const rnb_b200_mixer_cfg &m) { return (m.kv_rank + m.rot_dim + 7) & ~7; }
 
     std::vector<StackLayer> layers_;
     std::vector<LayerRun> runs_;
@@ -111,7 +151,7 @@ private:
     std::vector<void *> allocs_;
     std::vector<std::pair<rnb_b200_rotation, const void *>> tables_;
     DenseMat embed_;
-    float *final_norm_ = nullptr;
+    float *final_norm_ = nullptr, *final_bias_ = nullptr;
     StackScratch small_, big_;
     int *counters_ = nullptr;
     bool ready_ = false, loops_ = false;

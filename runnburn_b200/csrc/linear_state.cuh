@@ -1,7 +1,9 @@
-// Linear recurrences with a matrix state per head (RWKV-style time mixing, retention), all in f32:
+// Linear recurrences with a matrix state per head (RWKV-style time mixing, retention, gated linear
+// attention), all in f32:
 //   o_t = rs * S^T r_t + (sum_i r_t[i] u[i] k_t[i]) v_t,      S <- diag(w_t) S + k_t v_t^T
 // Time mixing: w_t per key channel, u the bonus of the current token, rs = 1.  Retention, whose output
-// reads the updated state S_t = decay S + k v^T: w_t = decay of the head, u = 1, rs = decay.
+// reads the updated state S_t = decay S + k v^T: w_t = decay of the head, u = 1, rs = decay.  Gated linear
+// attention reads the updated state too, with w_t per key channel: the first term takes w_t r_t, u = 1.
 // State [heads][dim][vdim] f32.
 //
 //   linear_state_step_kernel    1..8 tokens, one launch: rotations or decays, recurrence, head norm, gate
@@ -18,13 +20,15 @@
 
 namespace rnb {
 
+enum LinearMode { LS_BONUS = 0, LS_HEAD_DECAY = 1, LS_UPDATED = 2 };   // time mixing, retention, gated linear attention
 struct LinearChunkArgs {
-    const void *r, *k, *v;     // [tokens][heads][dim], same, [tokens][heads][vdim] (AT)
-    const float *w;            // [tokens][heads][dim]; null: decay[head]
+    const void *r, *k, *v;     // [tokens][heads][dim], same, [tokens][heads][vdim] (AT); a token's row is ldr (r, k), ldv long
+    const float *w;            // [tokens][heads][dim]; LS_HEAD_DECAY: decay[head] instead
     const float *decay, *u;    // [heads]; [heads][dim], null: 1
+    float o_mul;               // multiplies the outputs
     float *state, *o;          // [heads][dim][vdim]; [tokens][heads][vdim]
     float *starts, *decays;    // [chunks][heads][dim][vdim]; [chunks][heads][dim]
-    int tokens, heads, dim, vdim, chunk, n_chunks;
+    int tokens, heads, dim, vdim, ldr, ldv, chunk, n_chunks;
     int G, JG;                 // lanes along dim (16 channels each), groups of 4 value columns per CTA
 };
 constexpr int LS_TI = 16, LS_TS = 16;   // channels per thread; tokens staged at a time
@@ -32,9 +36,10 @@ __host__ __device__ inline size_t linear_chunk_smem(int G, int JG) { return size
 
 // grid = (chunks, heads, column blocks); G * JG threads rounded up to a warp.
 // Thread (jg, g): value columns 4 jg .. + 3, channels 4 (q G + g) .. + 3 for q = 0..3.
-template <class AT, bool OUT, bool CONST_W>
+template <class AT, bool OUT, int MODE>
 RNB_GLOBAL void __launch_bounds__(256)
 linear_state_chunk_kernel(const __grid_constant__ LinearChunkArgs a) {
+    constexpr bool CONST_W = MODE == LS_HEAD_DECAY;
     extern __shared__ __align__(16) float ls_smem[];
     pdl_launch_dependents();
     pdl_wait();
@@ -76,14 +81,14 @@ linear_state_chunk_kernel(const __grid_constant__ LinearChunkArgs a) {
         for (int i = tid; i < nt * DP; i += blockDim.x) {
             const int t = i / DP, ch = i % DP;
             const bool in = ch < a.dim;
-            const size_t at = ((size_t)(t0 + t) * a.heads + h) * a.dim + ch;
+            const size_t at = (size_t)(t0 + t) * a.ldr + h * a.dim + ch;
             if (OUT) sr[i] = in ? to_f32(rp[at]) : 0.f;
             sk[i] = in ? to_f32(kp[at]) : 0.f;
-            if (!CONST_W) sw[i] = in ? a.w[at] : 0.f;
+            if (!CONST_W) sw[i] = in ? a.w[((size_t)(t0 + t) * a.heads + h) * a.dim + ch] : 0.f;
         }
         for (int i = tid; i < nt * VB; i += blockDim.x) {
             const int t = i / VB, col = j0 + i % VB;
-            sv[i] = col < a.vdim ? to_f32(vp[((size_t)(t0 + t) * a.heads + h) * a.vdim + col]) : 0.f;
+            sv[i] = col < a.vdim ? to_f32(vp[(size_t)(t0 + t) * a.ldv + h * a.vdim + col]) : 0.f;
         }
         __syncthreads();
         if (OUT) {
@@ -119,7 +124,7 @@ linear_state_chunk_kernel(const __grid_constant__ LinearChunkArgs a) {
                 for (int i = 0; i < 4; i++) {
 #pragma unroll
                     for (int e = 0; e < 4; e++) {
-                        if (OUT) acc[e] = fmaf(rr[i], S[4 * q + i][e], acc[e]);
+                        if (OUT) acc[e] = fmaf(MODE == LS_UPDATED ? rr[i] * ww[i] : rr[i], S[4 * q + i][e], acc[e]);
                         S[4 * q + i][e] = fmaf(ww[i], S[4 * q + i][e], kk[i] * vv[e]);
                     }
                     if (!OUT && !CONST_W) P[4 * q + i] *= ww[i];
@@ -134,7 +139,7 @@ linear_state_chunk_kernel(const __grid_constant__ LinearChunkArgs a) {
                     float *o = a.o + ((size_t)(t0 + t) * a.heads + h) * a.vdim + j;
 #pragma unroll
                     for (int e = 0; e < 4; e++)
-                        if (j + e < a.vdim) o[e] = fmaf(rs, acc[e], sb[t] * vv[e]);
+                        if (j + e < a.vdim) o[e] = fmaf(rs, acc[e], sb[t] * vv[e]) * a.o_mul;
                 }
             }
         }
@@ -186,18 +191,19 @@ linear_state_scan_kernel(const float *__restrict__ state, float *starts, const f
     *reinterpret_cast<Vec *>(starts + (size_t)(n_chunks - 1) * n + i) = S;
 }
 
-// Decays of time mixing: out[t][c] = exp(-exp(sum_j w2[c][j] tanh(z[t][j]) + w0[c])).
+// Decays from their low-rank input: out[t][c] = decay_of(sum_j w2[c][j] f(z[t][j]) + w0[c]); f: tanh for DECAY_EXP, else none.
 // grid = (ceil(channels / 128), ceil(tokens / 16)), 128 threads; dynamic shared memory 16 * rank floats.
 RNB_GLOBAL void __launch_bounds__(128)
-decay_rows_kernel(const float *__restrict__ z, const bf16 *__restrict__ w2, const float *__restrict__ w0, int tokens, int rank, int channels,
-                  float *__restrict__ out) {
+decay_rows_kernel(const float *__restrict__ z, const bf16 *__restrict__ w2, const float *__restrict__ w0, int tokens, int rank, int channels, int kind,
+                  float inv_tau, float *__restrict__ out) {
     extern __shared__ __align__(16) float dr_smem[];   // [rank][16]
     pdl_launch_dependents();
     pdl_wait();
     const int t0 = blockIdx.y * 16;
     for (int i = threadIdx.x; i < rank * 16; i += blockDim.x) {
         const int t = i / rank, j = i % rank;
-        dr_smem[j * 16 + t] = t0 + t < tokens ? tanhf(z[(size_t)(t0 + t) * rank + j]) : 0.f;
+        const float v = t0 + t < tokens ? z[(size_t)(t0 + t) * rank + j] : 0.f;
+        dr_smem[j * 16 + t] = kind == DECAY_EXP ? tanhf(v) : v;
     }
     __syncthreads();
     const int c = blockIdx.x * 128 + threadIdx.x;
@@ -219,18 +225,18 @@ decay_rows_kernel(const float *__restrict__ z, const bf16 *__restrict__ w2, cons
     }
 #pragma unroll
     for (int t = 0; t < 16; t++)
-        if (t0 + t < tokens) out[(size_t)(t0 + t) * channels + c] = expf(-expf(acc[t] + b));
+        if (t0 + t < tokens) out[(size_t)(t0 + t) * channels + c] = decay_of(kind, acc[t] + b, inv_tau);
 }
 
-// z [tokens][rank] f32 -> [tanh z rounded to bf16 | what the rounding left] [tokens][2 rank]: against [w2 | w2] the
-// tensor-core matmul gives w2 tanh(z) to f32 accuracy.
+// z [tokens][rank] f32 -> [f(z) rounded to bf16 | what the rounding left] [tokens][2 rank], f = tanh or none: against
+// [w2 | w2] the tensor-core matmul gives w2 f(z) to about f32 accuracy.
 RNB_GLOBAL void __launch_bounds__(256)
-tanh_split_kernel(const float *__restrict__ z, int rank, size_t n, bf16 *__restrict__ out) {
+split_rows_kernel(const float *__restrict__ z, int rank, size_t n, int kind, bf16 *__restrict__ out) {
     pdl_launch_dependents();
     pdl_wait();
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= n) return;
-    const float v = tanhf(z[i]);
+    const float v = kind == DECAY_EXP ? tanhf(z[i]) : z[i];
     const bf16 hi = from_f32<bf16>(v);
     bf16 *row = out + (i / rank) * 2 * rank + i % rank;
     row[0] = hi;
@@ -265,12 +271,14 @@ __host__ __device__ inline LinearTileSmem linear_tile_smem(int DT, int NW) {
 // Per tile of 16 tokens, with S^T (value column x channel) in each warp's accumulators:
 //   o^T = S^T r~^T + v^T A^T          r~_t = r_t times the decays before t,  A: pairs inside the tile
 //   S^T <- S^T D + v^T k~             k~_t = k_t times the decays after t,   D: all decays of the tile
+// (gated linear attention: r~_t takes the decay of t itself too, and so do the pairs of A)
 // Time mixing computes A below the diagonal pair by pair (running products of w), with r u k on it;
 // retention masks and scales q k^T by powers of its decay, and scales S^T q^T by them afterwards.
 // grid = (chunks, heads, column blocks), blockDim = 32 * NW.  dim <= 16 DT, dim and vdim multiples of 8.
-template <int DT, bool OUT, bool CONST_W>
+template <int DT, bool OUT, int MODE>
 RNB_GLOBAL void __launch_bounds__(256)
 linear_state_tile_kernel(const __grid_constant__ LinearChunkArgs a) {
+    constexpr bool CONST_W = MODE == LS_HEAD_DECAY;
     extern __shared__ __align__(128) uint8_t lt_smem[];
     pdl_launch_dependents();
     pdl_wait();
@@ -283,7 +291,7 @@ linear_state_tile_kernel(const __grid_constant__ LinearChunkArgs a) {
     const bf16 *rp = reinterpret_cast<const bf16 *>(a.r) + (size_t)h * a.dim, *kp = reinterpret_cast<const bf16 *>(a.k) + (size_t)h * a.dim;
     const bf16 *vp = reinterpret_cast<const bf16 *>(a.v) + (size_t)h * a.vdim;
     const float *wp = CONST_W ? nullptr : a.w + (size_t)h * a.dim;
-    const size_t ldk = (size_t)a.heads * a.dim, ldv = (size_t)a.heads * a.vdim;
+    const size_t ldk = (size_t)a.ldr, ldw = (size_t)a.heads * a.dim, ldv = (size_t)a.ldv;
     float *sD = reinterpret_cast<float *>(lt_smem + L.d), *sP = reinterpret_cast<float *>(lt_smem + L.p), *pw = reinterpret_cast<float *>(lt_smem + L.pw);
     auto cp16 = [&](uint32_t dst, const void *src, bool in) {
         asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(in ? 16u : 0u) : "memory");
@@ -305,7 +313,7 @@ linear_state_tile_kernel(const __grid_constant__ LinearChunkArgs a) {
                 if (OUT) cp16(st + (uint32_t)t * L.kp + (uint32_t)q * 16u, rp + row * ldk + at, ok);
             }
             if (!CONST_W)
-                for (int q = q0; q < CWF; q += qs) cp16(st + L.w + (uint32_t)(t * DP + q * 4) * 4u, wp + row * ldk + min(q * 4, a.dim - 4), in && q * 4 < a.dim);
+                for (int q = q0; q < CWF; q += qs) cp16(st + L.w + (uint32_t)(t * DP + q * 4) * 4u, wp + row * ldw + min(q * 4, a.dim - 4), in && q * 4 < a.dim);
             for (int q = q0; q < 2 * NW; q += qs) {
                 const int col = j0 + q * 8;
                 cp16(st + L.v + (uint32_t)t * L.vp + (uint32_t)q * 16u, vp + row * ldv + min(col, a.vdim - 8), in && col < a.vdim);
@@ -417,8 +425,9 @@ linear_state_tile_kernel(const __grid_constant__ LinearChunkArgs a) {
                 } else {
 #pragma unroll
                     for (int t = 0; t < 16; t++) {
+                        if (MODE == LS_UPDATED) p *= w16[t];
                         lt_split_store(rhi + t * KE + ch, rlo + t * KE + ch, raw16[t] * p);
-                        p *= w16[t];
+                        if (MODE != LS_UPDATED) p *= w16[t];
                     }
                 }
             }
@@ -440,7 +449,7 @@ linear_state_tile_kernel(const __grid_constant__ LinearChunkArgs a) {
                         float r4[4];
                         row4(kk + s * KE, i, x[i]);
                         row4(rr + s * KE, i, r4);
-                        const float4 u4 = ch < a.dim ? *reinterpret_cast<const float4 *>(a.u + h * a.dim + ch) : make_float4(0.f, 0.f, 0.f, 0.f);
+                        const float4 u4 = !a.u ? make_float4(1.f, 1.f, 1.f, 1.f) : ch < a.dim ? *reinterpret_cast<const float4 *>(a.u + h * a.dim + ch) : make_float4(0.f, 0.f, 0.f, 0.f);
                         b = fmaf(r4[0] * u4.x, x[i][0], b);
                         b = fmaf(r4[1] * u4.y, x[i][1], b);
                         b = fmaf(r4[2] * u4.z, x[i][2], b);
@@ -456,14 +465,13 @@ linear_state_tile_kernel(const __grid_constant__ LinearChunkArgs a) {
                                 float r4[4];
                                 row4(rr + t * KE, i, r4);
                                 const float4 w4 = *reinterpret_cast<const float4 *>(ww + t * DP + 4 * (q + 8 * i));
-                                v[t] = fmaf(r4[0], x[i][0], v[t]);
-                                v[t] = fmaf(r4[1], x[i][1], v[t]);
-                                v[t] = fmaf(r4[2], x[i][2], v[t]);
-                                v[t] = fmaf(r4[3], x[i][3], v[t]);
-                                x[i][0] *= w4.x;
-                                x[i][1] *= w4.y;
-                                x[i][2] *= w4.z;
-                                x[i][3] *= w4.w;
+                                const float wv[4] = {w4.x, w4.y, w4.z, w4.w};
+#pragma unroll
+                                for (int e = 0; e < 4; e++) {
+                                    if (MODE == LS_UPDATED) x[i][e] *= wv[e];
+                                    v[t] = fmaf(r4[e], x[i][e], v[t]);
+                                    if (MODE != LS_UPDATED) x[i][e] *= wv[e];
+                                }
                             }
                         }
                     }
@@ -525,7 +533,7 @@ linear_state_tile_kernel(const __grid_constant__ LinearChunkArgs a) {
 #pragma unroll
                 for (int e = 0; e < 4; e++) {
                     const int t = n * 8 + 2 * tq + (e & 1), j = jw + g + 8 * (e >> 1);
-                    if (t < nt && j < a.vdim) a.o[((size_t)(t0 + t) * a.heads + h) * a.vdim + j] = o[n][e];
+                    if (t < nt && j < a.vdim) a.o[((size_t)(t0 + t) * a.heads + h) * a.vdim + j] = o[n][e] * a.o_mul;
                 }
         }
 #pragma unroll
@@ -562,17 +570,49 @@ linear_state_tile_kernel(const __grid_constant__ LinearChunkArgs a) {
 }
 
 // ---- few tokens: everything between the projections in one launch -------------------------------
+// True for the one of n CTAs that arrives last at the counter (zero between launches); what the others wrote before is
+// then visible to it through L2.
+__device__ __forceinline__ bool last_of_head(int *counter, int n) {
+    __shared__ int s_last;
+    __threadfence();
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        const int before = n > 1 ? atomicAdd(counter, 1) : 0;
+        s_last = before == n - 1;
+        if (n > 1 && s_last) *counter = 0;
+        __threadfence();
+    }
+    __syncthreads();
+    return s_last != 0;
+}
+// Head h of head_norm_gate_kernel for T tokens, f32, by one CTA; o [T][heads][vdim] is read through L2.
+__device__ __forceinline__ void head_norm_gate_rows(const float *o, const float *g, const float *norm, float *act, int T, int heads, int h, int vdim, int norm_head,
+                                                    int ldg, int lda, float eps, float mul) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+    for (int t = warp; t < T; t += nw) {
+        const float *x = o + ((size_t)t * heads + h) * vdim;
+        float ss = 0.f;
+        for (int i = lane; i < vdim; i += 32) {
+            const float v = __ldcg(x + i);
+            ss = fmaf(v, v, ss);
+        }
+        const float r = mul / sqrtf(warp_sum(ss) / (float)vdim + eps);
+        const float *gt = g + (size_t)t * ldg + (size_t)h * vdim;
+        float *at = act + (size_t)t * lda + (size_t)h * vdim;
+        for (int i = lane; i < vdim; i += 32) at[i] = __ldcg(x + i) * r * (norm ? norm[(size_t)h * norm_head + i] : 1.0f) * silu_f32(gt[i]);
+    }
+}
 struct LinearStepArgs {
-    const float *r, *k, *v, *g;      // projections of the tokens, f32: [tokens][heads * dim] (v, g: heads * vdim)
-    const float *z, *w0, *decay, *u; // time mixing: z [tokens][rank], w0 and u [heads * dim]; retention: decay [heads]
+    const float *r, *k, *v, *g;      // projections of the tokens, f32: [tokens][heads * dim] (v, g: heads * vdim), rows of ldr, ldv
+    const float *z, *w0, *decay, *u; // low-rank decays: z [tokens][rank], w0 [heads * dim]; u [heads * dim] or null; retention: decay [heads]
     const bf16 *w2;                  // [heads * dim][rank]
-    const float *norm;               // [heads * vdim] or null
+    const float *norm;               // null: 1, else `norm_head` elements from one head's to the next
     Rotation rot;                    // of r and k (table null: none)
     const int *pos0;
-    float k_mul, eps;
-    float *state, *o, *act;          // o: scratch [tokens][heads * vdim]; act: the output
+    float k_mul, o_mul, out_mul, inv_tau, eps;   // o_mul before the norm, out_mul after the gate
+    float *state, *o, *act;          // o: scratch [tokens][heads * vdim]; act: the output, rows of lda
     int *counters;                   // [heads], zero between launches
-    int tokens, heads, dim, vdim, rank;
+    int tokens, heads, dim, vdim, rank, mode, norm_head, ldr, ldv, lda;
 };
 __host__ inline size_t linear_step_smem(int tokens, int dim, int rank) {
     return sizeof(float) * ((size_t)tokens * (3 * dim + rank + 32 + 1) + 8 * 32);
@@ -583,7 +623,6 @@ template <int TI>
 RNB_GLOBAL void __launch_bounds__(256)
 linear_state_step_kernel(const __grid_constant__ LinearStepArgs a) {
     extern __shared__ __align__(16) float st_smem[];
-    __shared__ int s_last;
     pdl_launch_dependents();
     const int T = a.tokens, dim = a.dim, vdim = a.vdim, h = blockIdx.x, j0 = blockIdx.y * 32;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, j = j0 + lane;
@@ -613,17 +652,18 @@ linear_state_step_kernel(const __grid_constant__ LinearStepArgs a) {
     const int p0 = a.rot.table ? *a.pos0 : 0;
     for (int i = tid; i < T * dim; i += 256) {
         const int t = i / dim, ch = i % dim;
-        const float *rr = a.r + ((size_t)t * a.heads + h) * dim, *kk = a.k + ((size_t)t * a.heads + h) * dim;
+        const float *rr = a.r + (size_t)t * a.ldr + h * dim, *kk = a.k + (size_t)t * a.ldr + h * dim;
         sr[i] = rotated_element(a.rot, p0 + t, ch, [&](int e) { return rr[e]; });
         sk[i] = rotated_element(a.rot, p0 + t, ch, [&](int e) { return kk[e]; }) * a.k_mul;
         if (a.decay) sw[i] = a.decay[h];
     }
     for (int i = tid; i < T * 32; i += 256) {
         const int col = j0 + (i & 31);
-        sv[i] = col < vdim ? a.v[((size_t)(i >> 5) * a.heads + h) * vdim + col] : 0.f;
+        sv[i] = col < vdim ? a.v[(size_t)(i >> 5) * a.ldv + h * vdim + col] : 0.f;
     }
-    for (int i = tid; i < T * a.rank; i += 256) sz[i] = tanhf(a.z[i]);
+    for (int i = tid; i < T * a.rank; i += 256) sz[i] = a.mode == LS_BONUS ? tanhf(a.z[i]) : a.z[i];
     __syncthreads();
+    const int dkind = a.mode == LS_UPDATED ? DECAY_SIGMOID_ROOT : DECAY_EXP;
     if (dvec) {
         for (int ch = dch; ch < (dim + 63) / 64 * 64; ch += 64) {
             if (ch != dch && ch < dim)
@@ -646,7 +686,7 @@ linear_state_step_kernel(const __grid_constant__ LinearStepArgs a) {
                         }
                 s += __shfl_xor_sync(0xffffffffu, s, 1);
                 s += __shfl_xor_sync(0xffffffffu, s, 2);
-                if (dl == 0 && ch < dim) sw[t * dim + ch] = expf(-expf(s + a.w0[h * dim + ch]));
+                if (dl == 0 && ch < dim) sw[t * dim + ch] = decay_of(dkind, s + a.w0[h * dim + ch], a.inv_tau);
             }
         }
     } else if (!a.decay) {
@@ -656,7 +696,7 @@ linear_state_step_kernel(const __grid_constant__ LinearStepArgs a) {
                 float s = 0.f;
                 for (int q = lane; q < a.rank; q += 32) s = fmaf(to_f32(w[q]), sz[t * a.rank + q], s);
                 s = warp_sum(s);
-                if (lane == 0) sw[t * dim + ch] = expf(-expf(s + a.w0[h * dim + ch]));
+                if (lane == 0) sw[t * dim + ch] = decay_of(dkind, s + a.w0[h * dim + ch], a.inv_tau);
             }
         }
     }
@@ -675,7 +715,7 @@ linear_state_step_kernel(const __grid_constant__ LinearStepArgs a) {
         for (int q = 0; q < TI; q++) {
             const int ch = warp + 8 * q;
             if (ch < dim) {
-                acc = fmaf(sr[t * dim + ch], S[q], acc);
+                acc = fmaf(a.mode == LS_UPDATED ? sr[t * dim + ch] * sw[t * dim + ch] : sr[t * dim + ch], S[q], acc);
                 S[q] = fmaf(sw[t * dim + ch], S[q], sk[t * dim + ch] * v);
             }
         }
@@ -685,7 +725,7 @@ linear_state_step_kernel(const __grid_constant__ LinearStepArgs a) {
             float s = 0.f;
 #pragma unroll
             for (int i = 0; i < 8; i++) s += red[i * 32 + lane];
-            if (live) __stcg(a.o + ((size_t)t * a.heads + h) * vdim + j, fmaf(rs, s, sb[t] * v));
+            if (live) __stcg(a.o + ((size_t)t * a.heads + h) * vdim + j, fmaf(rs, s, sb[t] * v) * a.o_mul);
         }
         __syncthreads();
     }
@@ -694,27 +734,7 @@ linear_state_step_kernel(const __grid_constant__ LinearStepArgs a) {
         const int ch = warp + 8 * q;
         if (live && ch < dim) sp[(size_t)ch * vdim] = S[q];
     }
-    __threadfence();
-    __syncthreads();
-    if (tid == 0) {
-        const int n = gridDim.y, before = n > 1 ? atomicAdd(a.counters + h, 1) : 0;
-        s_last = before == n - 1;
-        if (n > 1 && s_last) a.counters[h] = 0;
-        __threadfence();
-    }
-    __syncthreads();
-    if (!s_last) return;
-    for (int t = warp; t < T; t += 8) {
-        const size_t at = ((size_t)t * a.heads + h) * vdim;
-        float ss = 0.f;
-        for (int i = lane; i < vdim; i += 32) {
-            const float v = __ldcg(a.o + at + i);
-            ss = fmaf(v, v, ss);
-        }
-        const float r = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + a.eps);
-        for (int i = lane; i < vdim; i += 32)
-            a.act[at + i] = __ldcg(a.o + at + i) * r * (a.norm ? a.norm[h * vdim + i] : 1.0f) * silu_f32(a.g[at + i]);
-    }
+    if (last_of_head(a.counters + h, gridDim.y)) head_norm_gate_rows(a.o, a.g, a.norm, a.act, T, a.heads, h, vdim, a.norm_head, a.ldv, a.lda, a.eps, a.out_mul);
 }
 
 }  // namespace rnb

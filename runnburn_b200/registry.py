@@ -11,10 +11,10 @@ from pathlib import Path
 
 from .decoder import Decoder
 from .safetensors import SafetensorsFile
-from .stack import punisun_config
+from .stack import dutivik_config, punisun_config
 
 # architecture -> function(config.json, max_ctx, dtype) that builds the decoder's configuration
-ARCHITECTURES = {"Punisun": punisun_config}
+ARCHITECTURES = {"Punisun": punisun_config, "Dutivik": dutivik_config}
 
 
 def read_config(folder, max_ctx: int, dtype: str = "bfloat16"):

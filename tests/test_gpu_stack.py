@@ -13,36 +13,11 @@ import stack_util as su
 
 pytestmark = pytest.mark.gpu
 ROOT = Path(__file__).resolve().parent.parent
-TOL = {"float32": 2e-5, "bfloat16": 3e-2}
+TOL = su.TOL
 DTYPES = ["float32", "bfloat16"]
 
 
-def _bad(got, want, dtype):
-    """Empty when the rows agree.  f32: every row.  bf16 rounds the projections, and a head's norm amplifies that
-    where its output nearly cancels: the rows together are held to TOL, a single one to four times as much."""
-    worst = su.rel(got, want)
-    mean = float(np.sqrt(np.mean((np.asarray(got, np.float64) - want) ** 2) / np.mean(np.asarray(want, np.float64) ** 2)))
-    ok = worst < TOL[dtype] if dtype == "float32" else mean < TOL[dtype] and worst < 4 * TOL[dtype]
-    return "" if ok else f"worst row {worst:.3g}, together {mean:.3g}"
-
-
-def _tokens(cfg, n, seed=0):
-    return np.random.default_rng(seed).integers(0, cfg["vocab"], n)
-
-
-def _feed(dec, toks, cuts):
-    """Logits of all tokens, fed in portions of the sizes `cuts` (repeated until the end)."""
-    out, at, i = [], 0, 0
-    while at < len(toks):
-        n = min(cuts[i % len(cuts)], len(toks) - at)
-        i += 1
-        if n == 1 and at > 0:
-            out.append(dec.step(int(toks[at]), at, want_logits=True)[1][None])
-        else:
-            out.append(dec.prefill_logits(toks[at:at + n], at, list(range(n)))[0])
-        at += n
-    return np.concatenate(out)
-
+_bad, _tokens, _feed = su.bad, su.tokens, su.feed
 
 MIXED = [su.wkv(), su.retention(), su.latent(scaling=su.YARN), su.wkv(ff=0), su.retention(heads=1, dim=64, vdim=24, dims=32)]
 MECHANISMS = {

@@ -8,7 +8,7 @@ import hybrid_ref as ref
 import stack_util as su
 from runnburn_b200 import registry
 from runnburn_b200.safetensors import SafetensorsFile
-from runnburn_b200.stack import StackConfig, punisun_config
+from runnburn_b200.stack import StackConfig, dutivik_config, punisun_config
 
 
 def _mixed(**kw):
@@ -91,3 +91,76 @@ def test_reference_rotation_keeps_relative_positions():
             c1, s1 = ref.rotation_tables({"dims": 8, "base": 100.0}, [11 + shift])
             dots.append(float(np.sum(ref.rotate_pairs(q, c0, s0, inter) * ref.rotate_pairs(k, c1, s1, inter))))
         assert abs(dots[0] - dots[1]) < 1e-12
+
+
+def test_dutivik_config_reads_every_size_and_constant():
+    layers = [su.parallel(left=su.window(heads=6, kv_heads=3, dim=10, vdim=12, size=77, dims=4, base=50.0, factor=3.0, scale=0.3), right=su.delta(heads=4, kv_heads=1, dim=20, vdim=28, conv=5),
+                          left_scale=0.25, right_scale=2.0, ff=36),
+              su.gla(heads=5, dim=14, vdim=18, tau=9.0, ff=0)]
+    cfg = su.dutivik(layers + [su.again(layers[1], 1), su.again(layers[0], 0)], eps=1e-4, scale=7.0)
+    c = dutivik_config(json.loads(json.dumps(cfg)), 123, "float32")
+    assert (c.width, c.vocab, c.max_ctx, c.dtype, c.loop) == (72, 97, 123, "float32", (0, 0, 1))
+    assert (c.norm_eps, c.embed_scale, c.residual_mult, c.block, c.norm, c.act) == (1e-4, 7.0, 1.0, "parallel", "layer", "silu")
+    assert [(ly.mixer, ly.join, ly.weights_of, ly.n_ff) for ly in c.layers] == [
+        ("attention", False, None, 36), ("delta", True, None, 0), ("gla", False, None, 0), ("gla", False, 1, 0), ("attention", False, 0, 36), ("delta", True, 0, 0)]
+    a, d, g = (ly.to_c([]) for ly in c.layers[:3])
+    assert (a.heads, a.kv_heads, a.dim, a.vdim, a.window, a.qk_norm, a.head_gate, a.prefix, a.weights_of) == (6, 3, 10, 12, 77, 1, 1, b"mix.left.", -1)
+    assert (a.rot.dims, a.rot.base, a.rot.interleaved, a.rot.scaled, a.rot.factor) == (4, 50.0, 1, 2, 3.0)
+    assert abs(a.scale - 0.3) < 1e-7 and (a.out_scale, d.out_scale) == (0.25, 2.0)
+    assert (d.heads, d.kv_heads, d.dim, d.vdim, d.conv, d.join, d.prefix) == (4, 1, 20, 28, 5, 1, b"mix.right.")
+    assert (g.heads, g.dim, g.vdim, g.tau, g.prefix, g.out_scale) == (5, 14, 18, 9.0, b"mix.", 1.0)
+    assert c.layers[4].to_c([]).weights_of == 0
+
+
+def test_dutivik_bad_configs():
+    with pytest.raises(ValueError, match="unknown mixer 'other'"):
+        dutivik_config(su.dutivik([dict(su.gla(), type="other")]), 8, "bfloat16")
+    with pytest.raises(ValueError, match="sparse"):
+        dutivik_config(su.dutivik([dict(su.gla(), mlp={"kind": "sparse", "ff": 8})]), 8, "bfloat16")
+
+
+def test_dutivik_registry(tmp_path):
+    cfg = su.dutivik([su.gla(), su.parallel(), su.again(su.gla(), 0)])
+    w = su.weights(cfg, 3)
+    assert not any(n.startswith("l2.") for n in w)
+    su.save(tmp_path, cfg, w)
+    assert registry.read_config(tmp_path, 64).embed_scale == 3.0
+    assert set(SafetensorsFile(tmp_path / "model.safetensors").tensors) == set(w)
+
+
+def test_dutivik_reference_does_not_depend_on_portions():
+    layers = [su.parallel(), su.gla()]
+    cfg = su.dutivik(layers + [su.again(layers[0], 0)])
+    w = su.weights(cfg, 1)
+    toks = np.random.default_rng(0).integers(0, cfg["vocab"], 40)
+    whole = ref.Model(cfg, w).forward(toks)
+    m = ref.Model(cfg, w)
+    parts, at = [], 0
+    for n in (1, 2, 13, 1, 23):
+        parts.append(m.forward(toks[at:at + n]))
+        at += n
+    assert np.allclose(np.concatenate(parts), whole, rtol=0, atol=1e-10)
+
+
+def test_reference_mechanisms_against_their_definitions():
+    rng = np.random.default_rng(0)
+    # a window of one token returns the value itself, whatever the scores
+    q, k, v = rng.standard_normal((3, 5, 2, 4))
+    assert np.allclose(ref.window_softmax(q, k, v, 3.0, 0, 0, 1), v)
+    # the delta rule with beta 1 and no decay stores v at a unit key exactly, and a second write replaces it
+    e = np.zeros((2, 1, 4))
+    e[:, 0, 1] = 1.0
+    v = rng.standard_normal((2, 1, 3))
+    o, S = ref.delta_recurrence(e, e, v, np.ones((2, 1)), np.ones((2, 1)), np.zeros((1, 4, 3)))
+    assert np.allclose(o, v) and np.allclose(S[0, 1], v[1, 0])
+    # the last column of the taps belongs to the current input
+    x, taps = rng.standard_normal((6, 2)), np.array([[0.0, 0.0, 1.0], [1.0, 0.0, 0.0]])
+    y, last = ref.short_convolution(x, np.zeros((2, 2)), taps)
+    assert np.allclose(y[:, 0], x[:, 0]) and np.allclose(y[2:, 1], x[:-2, 1]) and np.allclose(y[:2, 1], 0) and np.allclose(last, x[-2:])
+    # gated linear attention with decays of one is a running sum
+    q, k, v = rng.standard_normal((3, 7, 1, 2))
+    o, _ = ref.gla_recurrence(q, k, v, np.ones((7, 1, 2)), np.zeros((1, 2, 2)))
+    assert np.allclose(o[-1, 0], sum((k[t, 0] @ q[-1, 0]) * v[t, 0] for t in range(7)))
+    assert np.allclose(ref.channel_decay(np.array([0.3]), 4.0), ref.sigmoid(0.3) ** 0.25)
+    z = ref.layer_norm(rng.standard_normal((3, 8)) + 5.0, np.ones(8), np.zeros(8), 0.0)
+    assert np.allclose(z.mean(-1), 0) and np.allclose((z * z).mean(-1), 1)
