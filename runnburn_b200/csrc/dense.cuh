@@ -371,6 +371,7 @@ dense_gemm_simt_kernel(const __grid_constant__ DenseSimtJobs jobs) {
             if (pair) us[k][r] = win ? to_f32(job.w2[(size_t)(n0 + r) * job.cols + k0 + k]) : 0.f;
         }
         __syncthreads();
+        float c[4][4] = {}, d[4][4] = {};   // sums of sums: rounding grows with the depth of one tile and the number of tiles
 #pragma unroll
         for (int k = 0; k < DS_K; k++) {
             const float4 xv = *reinterpret_cast<const float4 *>(&xs[k][ty * 4]), wv = *reinterpret_cast<const float4 *>(&ws[k][tx * 4]);
@@ -378,16 +379,20 @@ dense_gemm_simt_kernel(const __grid_constant__ DenseSimtJobs jobs) {
 #pragma unroll
             for (int i = 0; i < 4; i++)
 #pragma unroll
-                for (int j = 0; j < 4; j++) a[i][j] = fmaf(xr[i], wr[j], a[i][j]);
+                for (int j = 0; j < 4; j++) c[i][j] = fmaf(xr[i], wr[j], c[i][j]);
             if (pair) {
                 const float4 uv = *reinterpret_cast<const float4 *>(&us[k][tx * 4]);
                 const float ur[4] = {uv.x, uv.y, uv.z, uv.w};
 #pragma unroll
                 for (int i = 0; i < 4; i++)
 #pragma unroll
-                    for (int j = 0; j < 4; j++) b[i][j] = fmaf(xr[i], ur[j], b[i][j]);
+                    for (int j = 0; j < 4; j++) d[i][j] = fmaf(xr[i], ur[j], d[i][j]);
             }
         }
+#pragma unroll
+        for (int i = 0; i < 4; i++)
+#pragma unroll
+            for (int j = 0; j < 4; j++) a[i][j] += c[i][j], b[i][j] += d[i][j];
         __syncthreads();
     }
 #pragma unroll

@@ -191,7 +191,10 @@ def test_long_memory(dtype, kind):
     if kind == "gla":
         w["l0.mix.a2.b"][:] = 6.0
         w["l0.mix.a2"][:] *= 0.25
-        names = ["l0.mix.k", "l0.mix.v"]
+        w["embed"][:, 1] = 6.0            # every query follows one direction, and the first key lies along it
+        w["l0.mix.q"][:, 1] = 1.0
+        w["l0.mix.k"][:, 0] = 2.0
+        names = ["l0.mix.v"]
     else:
         p = "l0.mix.right."
         w[p + "A_log"][:] = -4.0
@@ -206,7 +209,7 @@ def test_long_memory(dtype, kind):
     w["embed"][:31, 0] = 0.0
     w["embed"][31, 0] = 12.0
     for n in names:
-        w[n][:, 0] *= 40.0
+        w[n][:, 0] *= 8.0
     w["l0.mix.o" if kind == "gla" else "l0.mix.right.o"][:] *= 6.0
     w = {k: su.bf16_round(v) for k, v in w.items()}
     toks = su.tokens(dict(cfg, vocab=31), 1200, seed=1)
