@@ -56,12 +56,32 @@ def punisun_shape(n_layer: int, width: int, n_ff: int, vocab: int, loop=(0, 0, 1
     return dict(stack=[(wkv, ret, wkv, lat)[i % 4] for i in range(n_layer)], n_layer=n_layer, hidden=width, vocab=vocab, loop=loop)
 
 
+def dutivik_shape(n_layer: int, width: int, n_ff: int, vocab: int) -> dict:
+    """A mixed stack (Dutivik design) of the widths of a common dense model, in bf16: two parallel layers (window attention
+    over 1024 tokens, 128-wide heads, four query heads per key head; gated delta rule, 128-wide heads, two per key head) for
+    every one with gated linear attention.  The last layers use the weights of the first ones."""
+    h = width // 128
+    att = dict(mixer="attention", heads=h, kv_heads=max(h // 4, 1), dim=128, vdim=128, rot=dict(dims=128, base=2e5, scaling=dict(factor=4.0)), scale=128 ** -0.5,
+               window=1024, qk_norm=True, head_gate=True, out_scale=0.7, prefix="mix.left.", n_ff=n_ff)
+    dlt = dict(mixer="delta", heads=h, kv_heads=max(h // 2, 1), dim=128, vdim=128, conv=4, out_scale=0.9, prefix="mix.right.", join=True)
+    gla = dict(mixer="gla", heads=h, dim=64, vdim=128, tau=12.0, decay_rank=64, n_ff=n_ff)
+    recs = []
+    for i in range(n_layer):
+        of = i % 3 if n_layer >= 6 and i >= n_layer - 2 else None
+        recs += [dict(gla, weights_of=of)] if i % 3 == 2 else [dict(att, weights_of=of), dict(dlt, weights_of=of)]
+    return dict(stack=recs, n_layer=n_layer, hidden=width, vocab=vocab, loop=(0, 0, 1), form=dict(block="parallel", norm="layer", act="silu", embed_scale=8.0))
+
+
 WORKLOADS.update({
     # the layer widths of the 8B shape above; two layers run twice
     "punisun-8b-ctx4096": (punisun_shape(32, 4096, 14336, 128256, (0, 2, 2)), 4096),
     "punisun-1b-ctx4096": (punisun_shape(16, 2048, 8192, 128256, (0, 2, 2)), 4096),
     # one group of four layers of the 8B widths: the capture-sized case for ncu
     "punisun-4layers-ctx4096": (punisun_shape(4, 4096, 14336, 32768), 4096),
+    "dutivik-8b-ctx4096": (dutivik_shape(24, 4096, 14336, 128256), 4096),
+    "dutivik-1b-ctx4096": (dutivik_shape(12, 2048, 8192, 128256), 4096),
+    # two parallel layers and one of gated linear attention: the capture-sized case for ncu
+    "dutivik-3layers-ctx4096": (dutivik_shape(3, 4096, 14336, 32768), 4096),
     # the 1B widths of the closest other model, for the comparison at equal size
     "llama3-1b-q4km-ctx4096": (dict(n_layer=16, hidden=2048, n_head=16, n_kv_head=8, n_ff=8192, vocab=128256), 4096),
 })
@@ -90,7 +110,18 @@ def algorithmic_bytes_per_token(shape: dict, ctx: int) -> dict:
         for i in runs:
             m = shape["stack"][i]
             hd, hv = m["heads"] * m["dim"], m["heads"] * m.get("vdim", m["dim"])
-            if m["mixer"] == "latent_attention":
+            if m["mixer"] == "attention":
+                kd, kv = m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"]
+                mats = [(hd, H), (kd, H), (kv, H), (m["heads"], H), (H, hv)]
+                state += (min(ctx + 1, m["window"] or ctx + 1) + 1) * (kd + kv) * 2
+            elif m["mixer"] == "delta":
+                kd = m["kv_heads"] * m["dim"]
+                mats = [(kd, H), (kd, H), (hv, H), (hv, H), (2 * m["heads"], H), (H, hv)]
+                state += 2 * hd * m["vdim"] * 4 + m["conv"] * (2 * kd + hv) * 4
+            elif m["mixer"] == "gla":
+                mats = [(hd, H), (hd, H), (hv, H), (hv, H), (m["decay_rank"], H), (hd, m["decay_rank"]), (H, hv)]
+                state += 2 * hd * m["vdim"] * 4
+            elif m["mixer"] == "latent_attention":
                 row = m["kv_rank"] + m["rot_dim"]
                 mats = [(m["heads"] * (m["dim"] + m["rot_dim"]), H), (row, H), (hd, m["kv_rank"]), (hv, m["kv_rank"]), (H, hv)]
                 state += (ctx + 1) * row * 2
@@ -99,7 +130,8 @@ def algorithmic_bytes_per_token(shape: dict, ctx: int) -> dict:
                 if m["mixer"] == "wkv":
                     mats += [(m["decay_rank"], H), (hd, m["decay_rank"])]
                 state += 2 * hd * m.get("vdim", m["dim"]) * 4
-            mats += [(m["n_ff"], H), (m["n_ff"], H), (H, m["n_ff"])]
+            if m.get("n_ff"):
+                mats += [(m["n_ff"], H), (m["n_ff"], H), (H, m["n_ff"])]
             w += sum(r * c for r, c in mats) * 2
             act += sum(r + c for r, c in mats) * 4
         return {"weights": w, "kv": state, "activations": act, "total": w + state + act}
@@ -477,7 +509,7 @@ def run_gpu(args, shape, ctx, name, rank, world, local_rank):
             raise SystemExit("mixed stacks run on one GPU")
         from runnburn_b200.stack import MixerLayer
         cfg = r.StackConfig(width=shape["hidden"], vocab=shape["vocab"], layers=[MixerLayer(**m) for m in shape["stack"]], norm_eps=1e-6,
-                            residual_mult=0.5, loop=shape["loop"], max_ctx=max_ctx)
+                            loop=shape["loop"], max_ctx=max_ctx, **shape.get("form", dict(residual_mult=0.5)))
     else:
         cfg = r.ModelConfig(max_ctx=max_ctx, world_size=world, rank=rank, **shape)
     dec = r.Decoder(cfg)
@@ -599,7 +631,7 @@ def run_gpu(args, shape, ctx, name, rank, world, local_rank):
         "ms_per_step": ms / K, "repeats": R, "ms_per_step_all": [m / K for m in all_ms], "timing": "median of %d timed regions of %d steps each, max over ranks per region" % (R, K),
         "higher_is_better": True, "scaling": "strong" if world > 1 else "weak",
         "vs_baseline": None, "dtype": "bf16 weights, f32 activations and accumulate" if stack else "int8xint4->int32, f32 accumulate", "data": "synthetic",
-        "config": {"workload": name, "context": ctx, "kv_cache": "bf16 latent rows, f32 recurrent states" if stack else "f16", "weights": "random-init N(0,0.02), bf16, generated on device" if stack else ("random-init N(0,0.02): attention and LM head Q6_K, f32 router, experts Q4_K, generated on device" if shape.get("n_expert", 0) else "random-init N(0,0.02), Q4_K_M layout (attn_v/ffn_down/output Q6_K), generated on device"),
+        "config": {"workload": name, "context": ctx, "kv_cache": "bf16 latent rows or key and value rings, f32 recurrent states" if stack else "f16", "weights": "random-init N(0,0.02), bf16, generated on device" if stack else ("random-init N(0,0.02): attention and LM head Q6_K, f32 router, experts Q4_K, generated on device" if shape.get("n_expert", 0) else "random-init N(0,0.02), Q4_K_M layout (attn_v/ffn_down/output Q6_K), generated on device"),
                    "parallelism": (f"row-sharded x{world}, all-gather by " + ("ncclAllGather" if transport == "nccl" else "peer-memory stores over NVLink from the producing kernels' epilogues, consumers wait on arrival flags (no exchange launch)")) if world > 1 else "single GPU",
                    "l2": "each step streams its whole weight set and KV cache (GBs), far more than the 126 MB L2: no flush needed",
                    "algorithmic_bytes_per_token": alg},
@@ -640,7 +672,7 @@ def run_gpu(args, shape, ctx, name, rank, world, local_rank):
             dec.prefill(ids, 0, timed=True)
             _, pms = dec.prefill(ids, 0, timed=True)
             out["prefill"] = {"tokens": int(n_tok), "ms": pms, "tok_per_s": n_tok / (pms / 1000.0),
-                              "what": "embed, layers (projections and feed-forward on tcgen05 in bf16, chunked recurrences in f32, causal latent attention on mma.sync), "
+                              "what": "embed, layers (projections and feed-forward on tcgen05 in bf16, chunked recurrences in f32, causal attention on mma.sync), "
                                       "final norm + LM head + argmax of the last token" if stack else "embed, 32 x (RMSNorm, q/k/v matmul, RoPE + f16 KV append, causal attention, o_proj, RMSNorm, gate/up, SiLU*up, down), "
                                       "final norm + LM head + argmax of the last token; matmuls on tcgen05 (bf16), causal attention on mma.sync tensor cores (split-f16 operands, fp32 accumulate)"}
         except Exception as e:   # a secondary figure must not lose the headline line

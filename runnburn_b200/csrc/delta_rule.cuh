@@ -121,7 +121,7 @@ delta_step_kernel(const __grid_constant__ DeltaArgs a) {
         if (tid < T) {
             const float *ba = a.ba + (size_t)(t0 + tid) * a.ld_ba;
             sb[tid] = sigmoid_f32(ba[h]);
-            sg[tid] = expf(decay * softplus_f32(ba[a.a_at + h] + dt));
+            sg[tid] = expm1f(decay * softplus_f32(ba[a.a_at + h] + dt));   // g - 1: over many tokens the rounding of a g near 1 adds up
         }
         __syncthreads();
         for (int t = warp; t < T; t += 8) {
@@ -137,13 +137,13 @@ delta_step_kernel(const __grid_constant__ DeltaArgs a) {
         }
         __syncthreads();
         for (int t = 0; t < T; t++) {
-            const float g = sg[t];
+            const float g1 = sg[t];
             float kd = 0.f, qd = 0.f;
 #pragma unroll
             for (int q = 0; q < TI; q++) {
                 const int ch = warp + 8 * q;
                 if (ch < dim) {
-                    S[q] *= g;
+                    S[q] = fmaf(S[q], g1, S[q]);
                     kd = fmaf(sk[t * dim + ch], S[q], kd);
                     qd = fmaf(sq[t * dim + ch], S[q], qd);
                 }
