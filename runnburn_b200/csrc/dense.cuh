@@ -44,10 +44,11 @@ constexpr int ACT_GELU_TANH = 0, ACT_SILU = 1;
 __device__ __forceinline__ float gate_act(int act, float z) { return act == ACT_SILU ? silu_f32(z) : gelu_tanh_f32(z); }
 __device__ __forceinline__ float gate_act_fast(int act, float z) { return act == ACT_SILU ? silu_fast(z) : gelu_tanh_fast(z); }
 
-// A decay in (0, 1) from its projection x: exp(-exp(x)), or sigmoid(x)^inv_tau taken through the logarithm of the sigmoid.
+// A decay in (0, 1) from its projection x: exp(-exp(x)), or sigmoid(x)^inv_tau taken through the logarithm of the sigmoid
+// (whose absolute error is what counts for the power).
 constexpr int DECAY_EXP = 0, DECAY_SIGMOID_ROOT = 1;
 __device__ __forceinline__ float decay_of(int kind, float x, float inv_tau) {
-    return kind == DECAY_SIGMOID_ROOT ? expf((fminf(x, 0.f) - log1pf(expf(-fabsf(x)))) * inv_tau) : expf(-expf(x));
+    return kind == DECAY_SIGMOID_ROOT ? expf((fminf(x, 0.f) - logf(1.0f + expf(-fabsf(x)))) * inv_tau) : expf(-expf(x));
 }
 
 constexpr int DENSE_MAX_JOBS = 6;

@@ -219,8 +219,9 @@ int LayerStack::init(const rnb_b200_mixer_cfg *layers) {
             }
             r.m.push_back(st);
         }
-    RNB_TRY(alloc((void **)&counters_, (size_t)counters * 4));
-    RNB_CU(cudaMemset(counters_, 0, (size_t)counters * 4));
+    counters_of_mixer_ = counters;   // two mixers may run in one launch
+    RNB_TRY(alloc((void **)&counters_, (size_t)2 * counters * 4));
+    RNB_CU(cudaMemset(counters_, 0, (size_t)2 * counters * 4));
     RNB_CU(cudaStreamSynchronize(nullptr));
     attend_chunks_ = std::max(1, std::min((c.max_ctx + 127) / 128, 64));
     return RNB_B200_OK;
@@ -644,6 +645,12 @@ int LayerStack::ready(cudaStream_t s) {
                          (const void *)attention_step_kernel<float, float>, (const void *)attention_step_kernel<float, bf16>, (const void *)attention_step_kernel<bf16, bf16>,
                          (const void *)delta_prepare_kernel, (const void *)delta_tile_kernel<2>, (const void *)delta_tile_kernel<4>, (const void *)delta_tile_kernel<8>,
                          (const void *)delta_tile_kernel<16>};
+    const void *pairs[] = {
+#define RNB_AD(TI) (const void *)attention_delta_step_kernel<float, TI>, (const void *)attention_delta_step_kernel<bf16, TI>
+        RNB_AD(4), RNB_AD(8), RNB_AD(16), RNB_AD(32), RNB_AD(64)
+#undef RNB_AD
+    };
+    for (const void *f : pairs) RNB_TRY(raise(f));
     for (const void *f : fns) RNB_TRY(raise(f));
     const void *linear[] = {
 #define RNB_LC(AT, MODE) (const void *)linear_state_chunk_kernel<AT, false, MODE>, (const void *)linear_state_chunk_kernel<AT, true, MODE>
@@ -676,6 +683,16 @@ int LayerStack::ready(cudaStream_t s) {
             }
     RNB_TRY(alloc_scratch(small_, SMALL));
     RNB_TRY(reset(s));
+    for (StackLayer &L : layers_)
+        for (StackMixer &M : L.mixers)
+            if (M.conv) {   // [channels][taps] as the tensors have them -> [taps][channels]
+                const size_t taps = (size_t)M.c.conv, C = (size_t)2 * M.c.kv_heads * M.c.dim + (size_t)M.c.heads * M.c.vdim;
+                std::vector<float> in(C * taps), out(C * taps);
+                RNB_CU(cudaMemcpy(in.data(), M.conv, in.size() * 4, cudaMemcpyDeviceToHost));
+                for (size_t c = 0; c < C; c++)
+                    for (size_t t = 0; t < taps; t++) out[t * C + c] = in[c * taps + t];
+                RNB_CU(cudaMemcpy(M.conv, out.data(), out.size() * 4, cudaMemcpyHostToDevice));
+            }
     ready_ = true;
     return RNB_B200_OK;
 }
@@ -935,7 +952,7 @@ int LayerStack::mixer_linear(cudaStream_t s, int n, StackScratch &b, StackLayer 
         a.k_mul = k_mul, a.o_mul = o_mul, a.out_mul = m.out_scale, a.eps = cfg.norm_eps;
         a.inv_tau = gla ? 1.f / m.tau : 0.f;
         a.state = R.state, a.o = b.o, a.act = (float *)act_of(b, M, n);
-        a.counters = counters_;
+        a.counters = counters_ + i * counters_of_mixer_;
         a.tokens = n, a.heads = m.heads, a.dim = m.dim, a.vdim = m.vdim, a.rank = rank, a.mode = mode;
         a.ldr = ldr, a.ldv = ldv, a.lda = L.out_cols;
         const dim3 grid((unsigned)m.heads, (unsigned)((m.vdim + 31) / 32)), block(256);
@@ -984,7 +1001,7 @@ int LayerStack::mixer_linear(cudaStream_t s, int n, StackScratch &b, StackLayer 
     return head_norm_gate(s, n, b, L, M, part(3), ldv);
 }
 
-int LayerStack::mixer_attention(cudaStream_t s, int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev) {
+WindowAttentionArgs LayerStack::attention_args(int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev) const {
     const StackMixer &M = L.mixers[i];
     const rnb_b200_mixer_cfg &m = M.c;
     const bool nb = narrow(n);
@@ -995,27 +1012,37 @@ int LayerStack::mixer_attention(cudaStream_t s, int n, StackScratch &b, StackLay
     a.q = p, a.k = p + M.in_at[1] * es, a.v = p + M.in_at[2] * es;
     a.qn = b.qn, a.kc = R.cache, a.vc = R.values;
     a.gate = m.head_gate ? b.aux[i] : nullptr, a.ldg = M.aux_rows;
-    a.part = b.part, a.counters = counters_, a.act = act_of(b, M, n);
+    a.part = b.part, a.counters = counters_ + i * counters_of_mixer_, a.act = act_of(b, M, n);
+    a.fresh = n <= SMALL;
     a.pos0 = pos_dev;
     a.rot = Rotation{(const float2 *)M.rot_table, m.rot.dims, m.rot.interleaved};
     a.eps = cfg.norm_eps, a.scale = m.scale, a.out_mul = m.out_scale;
     a.tokens = n, a.heads = m.heads, a.kv_heads = m.kv_heads, a.dim = m.dim, a.vdim = m.vdim, a.ld = M.in_rows, a.lda = L.out_cols;
     a.ring = attention_ring(m), a.window = m.window, a.qk_norm = m.qk_norm;
+    return a;
+}
+
+int LayerStack::mixer_attention(cudaStream_t s, int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev) {
+    const rnb_b200_mixer_cfg &m = L.mixers[i].c;
+    const bool nb = narrow(n);
+    const WindowAttentionArgs a = attention_args(n, b, L, i, R, pos_dev);
     const size_t smem = attention_step_bytes(m, cfg.f32_math != 0);
     if (n <= SMALL) {
-        a.fresh = 1;
         const dim3 grid((unsigned)attention_chunks(m), (unsigned)m.kv_heads, (unsigned)n);
         if (cfg.f32_math) RNB_CU(launch_k(attention_step_kernel<float, float>, grid, dim3(AS_THREADS), smem, s, a));
         else RNB_CU(launch_k(attention_step_kernel<float, bf16>, grid, dim3(AS_THREADS), smem, s, a));
         return RNB_B200_OK;
     }
     const dim3 pg((unsigned)n, (unsigned)((m.heads + 2 * m.kv_heads + 7) / 8)), one(1, (unsigned)m.kv_heads, (unsigned)n);
+    const bool fours = m.dim <= 512 && m.dim % 4 == 0 && a.rot.dims % 4 == 0 && (a.rot.interleaved || !a.rot.table);
     if (!nb) {
-        RNB_CU(launch_k(attention_prepare_kernel<float, float>, pg, dim3(256), 0, s, a));
+        if (fours) RNB_CU(launch_k(attention_prepare_kernel<float, float, true>, pg, dim3(256), 0, s, a));
+        else RNB_CU(launch_k(attention_prepare_kernel<float, float, false>, pg, dim3(256), 0, s, a));
         RNB_CU(launch_k(attention_step_kernel<float, float>, one, dim3(AS_THREADS), smem, s, a));
         return RNB_B200_OK;
     }
-    RNB_CU(launch_k(attention_prepare_kernel<bf16, bf16>, pg, dim3(256), 0, s, a));
+    if (fours) RNB_CU(launch_k(attention_prepare_kernel<bf16, bf16, true>, pg, dim3(256), 0, s, a));
+    else RNB_CU(launch_k(attention_prepare_kernel<bf16, bf16, false>, pg, dim3(256), 0, s, a));
     if (!attention_tiled(m)) {
         RNB_CU(launch_k(attention_step_kernel<bf16, bf16>, one, dim3(AS_THREADS), smem, s, a));
         return RNB_B200_OK;
@@ -1032,31 +1059,36 @@ int LayerStack::mixer_attention(cudaStream_t s, int n, StackScratch &b, StackLay
     return launch_causal_attention(s, c);
 }
 
-int LayerStack::mixer_delta(cudaStream_t s, int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev) {
+DeltaArgs LayerStack::delta_args(int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev) const {
     const StackMixer &M = L.mixers[i];
     const rnb_b200_mixer_cfg &m = M.c;
-    const bool nb = narrow(n);
     DeltaArgs a;
     memset(&a, 0, sizeof(a));
     a.p = b.p[i], a.ba = b.aux[i], a.conv = M.conv, a.a_log = M.a_log, a.dt = M.dt, a.norm = M.head_norm;
-    a.ring = R.conv_ring, a.state = R.state, a.o = b.o, a.counters = counters_, a.pos0 = pos_dev;
+    a.ring = R.conv_ring, a.state = R.state, a.o = b.o, a.counters = counters_ + i * counters_of_mixer_, a.pos0 = pos_dev;
+    if (n <= SMALL) a.act = (float *)act_of(b, M, n);
     a.cq = reinterpret_cast<bf16 *>(b.cq), a.ck = reinterpret_cast<bf16 *>(b.ck), a.cv = reinterpret_cast<bf16 *>(b.cv), a.rec = b.rec;
     a.eps = cfg.norm_eps, a.out_mul = m.out_scale, a.q_mul = 1.0f / sqrtf((float)m.dim);
     a.tokens = n, a.heads = m.heads, a.kv_heads = m.kv_heads, a.dim = m.dim, a.vdim = m.vdim, a.taps = m.conv;
     a.k_at = M.in_at[1], a.v_at = M.in_at[2], a.g_at = M.in_at[3], a.a_at = m.heads, a.ld = M.in_rows, a.ld_ba = M.aux_rows, a.lda = L.out_cols;
+    return a;
+}
+
+int LayerStack::mixer_delta(cudaStream_t s, int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev) {
+    const StackMixer &M = L.mixers[i];
+    const rnb_b200_mixer_cfg &m = M.c;
+    const bool nb = narrow(n);
+    const DeltaArgs a = delta_args(n, b, L, i, R, pos_dev);
     if (nb && delta_tiled(m)) {
-        RNB_CU(launch_k(delta_prepare_kernel, dim3((unsigned)((n + 15) / 16), (unsigned)m.kv_heads), dim3(256), delta_prepare_smem(m.dim), s, a));
-        // one warp per 16 value columns; few per CTA, so that the heads spread over the SMs
-        const int cols = (m.vdim + 15) / 16;
-        int nw = std::min(cols, 8);
-        while (nw > 2 && m.heads * ((cols + nw - 1) / nw) < sm_ / 2) nw = (nw + 1) / 2;
-        const dim3 grid((unsigned)m.heads, (unsigned)((cols + nw - 1) / nw)), block((unsigned)(32 * nw));
-        if (m.dim <= 32) RNB_CU(launch_k(delta_tile_kernel<2>, grid, block, delta_tile_smem(2, nw).bytes, s, a));
-        else if (m.dim <= 64) RNB_CU(launch_k(delta_tile_kernel<4>, grid, block, delta_tile_smem(4, nw).bytes, s, a));
-        else if (m.dim <= 128) RNB_CU(launch_k(delta_tile_kernel<8>, grid, block, delta_tile_smem(8, nw).bytes, s, a));
-        else RNB_CU(launch_k(delta_tile_kernel<16>, grid, block, delta_tile_smem(16, nw).bytes, s, a));
+        RNB_CU(launch_k(delta_prepare_kernel, dim3((unsigned)((n + DP_TOKENS - 1) / DP_TOKENS), (unsigned)m.kv_heads), dim3(256), delta_prepare_smem(m.dim), s, a));
+        const int cols = (m.vdim + 15) / 16, cw = std::min(cols, 2);   // few columns per CTA, so that the heads spread over the SMs
+        const dim3 grid((unsigned)m.heads, (unsigned)((cols + cw - 1) / cw));
+        auto block = [&](int dt) { return dim3((unsigned)(32 * delta_tile_split(dt) * cw)); };
+        if (m.dim <= 32) RNB_CU(launch_k(delta_tile_kernel<2>, grid, block(2), delta_tile_smem(2, cw).bytes, s, a));
+        else if (m.dim <= 64) RNB_CU(launch_k(delta_tile_kernel<4>, grid, block(4), delta_tile_smem(4, cw).bytes, s, a));
+        else if (m.dim <= 128) RNB_CU(launch_k(delta_tile_kernel<8>, grid, block(8), delta_tile_smem(8, cw).bytes, s, a));
+        else RNB_CU(launch_k(delta_tile_kernel<16>, grid, block(16), delta_tile_smem(16, cw).bytes, s, a));
     } else {
-        if (n <= SMALL) a.act = (float *)act_of(b, M, n);
         const dim3 grid((unsigned)m.heads, (unsigned)((m.vdim + 31) / 32)), block(256);
         const size_t smem = delta_step_smem(m.dim);
         const int ti = (m.dim + 7) / 8;
@@ -1086,6 +1118,25 @@ static int launch_causal_attention(cudaStream_t s, const CausalAttentionArgs &a)
     }
     return RNB_B200_OK;
 }
+// A few tokens of window attention and the delta rule side by side: one launch.
+int LayerStack::mixers_attention_delta(cudaStream_t s, int n, StackScratch &b, StackLayer &L, LayerRun &R, const int *pos_dev) {
+    const rnb_b200_mixer_cfg &m = L.mixers[0].c, &k = L.mixers[1].c;
+    const WindowAttentionArgs a = attention_args(n, b, L, 0, R.m[0], pos_dev);
+    const DeltaArgs d = delta_args(n, b, L, 1, R.m[1], pos_dev);
+    const int chunks = attention_chunks(m), n_att = chunks * m.kv_heads * n, n_jb = (k.vdim + 31) / 32, ti = (k.dim + 7) / 8;
+    const dim3 grid((unsigned)(n_att + k.heads * n_jb));
+    const size_t smem = std::max(attention_step_bytes(m, cfg.f32_math != 0), delta_step_smem(k.dim));
+#define RNB_AD(TI) RNB_CU(cfg.f32_math ? launch_k(attention_delta_step_kernel<float, TI>, grid, dim3(256), smem, s, a, d, chunks, n_att, n_jb) \
+                                       : launch_k(attention_delta_step_kernel<bf16, TI>, grid, dim3(256), smem, s, a, d, chunks, n_att, n_jb))
+    if (ti <= 4) RNB_AD(4);
+    else if (ti <= 8) RNB_AD(8);
+    else if (ti <= 16) RNB_AD(16);
+    else if (ti <= 32) RNB_AD(32);
+    else RNB_AD(64);
+#undef RNB_AD
+    return RNB_B200_OK;
+}
+
 static bool latent_mma_fits(const LatentDims &d) { return d.rank % 8 == 0 && d.rank <= 640 && latent_mma_smem(d).bytes <= 220 * 1024; }
 static int launch_latent_attend_mma(cudaStream_t s, const bf16 *qf, const bf16 *cache, const LatentDims &d, float scale, const int *pos, float *part, int n, int chunks) {
     const dim3 grid((unsigned)chunks, (unsigned)((d.heads + 15) / 16), (unsigned)n), block(LM_THREADS);
@@ -1225,7 +1276,10 @@ int LayerStack::forward(cudaStream_t s, const uint32_t *tokens_dev, int n, const
         RNB_TRY(boundary(s, n, b, cur, y, wb, R.add_embedding, L.norm1, parallel() ? L.norm1b : nullptr, L.shifts() ? &L : nullptr, &R));
         Mm jobs[DENSE_MAX_JOBS];
         RNB_TRY(matmul(s, n, jobs, in_jobs(n, b, L, jobs), err));
-        for (size_t m = 0; m < L.mixers.size(); m++) RNB_TRY(run_mixer(s, n, b, L, (int)m, R.m[m], pos_dev, pos_host, err));
+        if (n <= SMALL && L.mixers.size() == 2 && L.mixers[0].c.mixer == RNB_B200_MIXER_ATTENTION && L.mixers[1].c.mixer == RNB_B200_MIXER_DELTA)
+            RNB_TRY(mixers_attention_delta(s, n, b, L, R, pos_dev));
+        else
+            for (size_t m = 0; m < L.mixers.size(); m++) RNB_TRY(run_mixer(s, n, b, L, (int)m, R.m[m], pos_dev, pos_host, err));
         const Mm out = out_job(b, L);
         RNB_TRY(matmul(s, n, &out, 1, err));
         y = b.y, wb = parallel() ? nullptr : L.norm1b;

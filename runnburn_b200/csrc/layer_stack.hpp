@@ -9,6 +9,9 @@
 
 namespace rnb {
 
+struct WindowAttentionArgs;
+struct DeltaArgs;
+
 struct DenseMat {
     uint16_t *w = nullptr;   // bf16 [rows][cols]
     int rows = 0, cols = 0;
@@ -129,6 +132,9 @@ private:
     int mixer_linear(cudaStream_t s, int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev, int *err);
     int mixer_latent(cudaStream_t s, int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev, int pos_host, int *err);
     int mixer_attention(cudaStream_t s, int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev);
+    WindowAttentionArgs attention_args(int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev) const;
+    DeltaArgs delta_args(int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev) const;
+    int mixers_attention_delta(cudaStream_t s, int n, StackScratch &b, StackLayer &L, LayerRun &R, const int *pos_dev);
     int mixer_delta(cudaStream_t s, int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev);
     int head_norm_gate(cudaStream_t s, int n, StackScratch &b, const StackLayer &L, const StackMixer &M, const void *g, int ldg);
     void *act_of(StackScratch &b, const StackMixer &M, int n) const { return (char *)b.act + (size_t)M.act_at * (narrow(n) ? 2 : 4); }
@@ -153,7 +159,7 @@ private:
     DenseMat embed_;
     float *final_norm_ = nullptr, *final_bias_ = nullptr;
     StackScratch small_, big_;
-    int *counters_ = nullptr;
+    int *counters_ = nullptr, counters_of_mixer_ = 0;
     bool ready_ = false, loops_ = false;
     uint64_t weight_bytes_ = 0;
     int sm_ = 148, attend_chunks_ = 1;

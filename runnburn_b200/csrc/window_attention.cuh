@@ -6,9 +6,12 @@
 //   causal_attention_kernel    then runs over the rings (bf16, tensor cores; causal_attention.cuh)
 //   attention_step_kernel      1..8 tokens, one launch: rotation, norm, append, attention split over the
 //                              visible keys, merge, gate.  With fresh = 0 it reads prepared rings only (prompts in f32).
+//   attention_delta_step_kernel  the same and the delta rule's step (delta_rule.cuh) side by side
 #pragma once
+#include <type_traits>
+
 #include "causal_attention.cuh"
-#include "linear_state.cuh"
+#include "delta_rule.cuh"
 
 namespace rnb {
 
@@ -54,8 +57,44 @@ __device__ __forceinline__ void rotated_normed_row(const AT *x, const Rotation &
     }
 }
 
-// grid = (tokens, ceil((heads + 2 kv_heads) / 8)), 256 threads: a warp per query, key or value vector
+// The same for vectors whose rotated pairs (2i, 2i + 1) and accesses of four elements do not straddle anything
+// (dim <= 512, dim and rotated dims multiples of 4, rows aligned): four elements per lane and access.
+template <class AT>
+struct alignas(4 * sizeof(AT)) Four { AT v[4]; };
 template <class AT, class CT>
+__device__ __forceinline__ void rotated_normed_fours(const AT *x, const Rotation &rot, int pos, int dim, bool norm, float eps, CT *out) {
+    const int lane = threadIdx.x & 31;
+    float v[4][4], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        const int e = 4 * (lane + 32 * i);
+        if (e >= dim) continue;
+        const Four<AT> a = *reinterpret_cast<const Four<AT> *>(x + e);
+#pragma unroll
+        for (int q = 0; q < 4; q++) v[i][q] = to_f32(a.v[q]);
+        if (rot.table && e < rot.dims) {
+            const float4 cs = *reinterpret_cast<const float4 *>(rot.table + (size_t)pos * (rot.dims / 2) + e / 2);
+            const float a0 = v[i][0], a1 = v[i][1], a2 = v[i][2], a3 = v[i][3];
+            v[i][0] = fmaf(a0, cs.x, -(a1 * cs.y)), v[i][1] = fmaf(a1, cs.x, a0 * cs.y);
+            v[i][2] = fmaf(a2, cs.z, -(a3 * cs.w)), v[i][3] = fmaf(a3, cs.z, a2 * cs.w);
+        }
+#pragma unroll
+        for (int q = 0; q < 4; q++) ss = fmaf(v[i][q], v[i][q], ss);
+    }
+    const float r = norm ? 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps) : 1.0f;
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        const int e = 4 * (lane + 32 * i);
+        if (e >= dim) continue;
+        Four<CT> o;
+#pragma unroll
+        for (int q = 0; q < 4; q++) o.v[q] = from_f32<CT>(v[i][q] * r);
+        *reinterpret_cast<Four<CT> *>(out + e) = o;
+    }
+}
+
+// grid = (tokens, ceil((heads + 2 kv_heads) / 8)), 256 threads: a warp per query, key or value vector.  FOURS: the form above.
+template <class AT, class CT, bool FOURS>
 RNB_GLOBAL void __launch_bounds__(256)
 attention_prepare_kernel(const __grid_constant__ WindowAttentionArgs a) {
     pdl_launch_dependents();
@@ -63,18 +102,25 @@ attention_prepare_kernel(const __grid_constant__ WindowAttentionArgs a) {
     const int t = blockIdx.x, unit = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, pos = *a.pos0 + t;
     if (unit >= a.heads + 2 * a.kv_heads) return;
     const size_t row = (size_t)t * a.ld, slot = (size_t)(pos % a.ring);
+    auto finish = [&](const AT *x, auto *out) {
+        typedef typename std::remove_pointer<decltype(out)>::type OT;
+        if (FOURS) rotated_normed_fours<AT, OT>(x, a.rot, pos, a.dim, a.qk_norm, a.eps, out);
+        else rotated_normed_row(x, a.rot, pos, a.dim, a.qk_norm, a.eps, [&](int e, float v) { out[e] = from_f32<OT>(v); });
+    };
     if (unit < a.heads) {
-        AT *out = reinterpret_cast<AT *>(a.qn) + ((size_t)t * a.heads + unit) * a.dim;
-        rotated_normed_row(reinterpret_cast<const AT *>(a.q) + row + (size_t)unit * a.dim, a.rot, pos, a.dim, a.qk_norm, a.eps, [&](int e, float v) { out[e] = from_f32<AT>(v); });
+        finish(reinterpret_cast<const AT *>(a.q) + row + (size_t)unit * a.dim, reinterpret_cast<AT *>(a.qn) + ((size_t)t * a.heads + unit) * a.dim);
     } else if (unit < a.heads + a.kv_heads) {
         const int g = unit - a.heads;
-        CT *out = reinterpret_cast<CT *>(a.kc) + (slot * a.kv_heads + g) * a.dim;
-        rotated_normed_row(reinterpret_cast<const AT *>(a.k) + row + (size_t)g * a.dim, a.rot, pos, a.dim, a.qk_norm, a.eps, [&](int e, float v) { out[e] = from_f32<CT>(v); });
+        finish(reinterpret_cast<const AT *>(a.k) + row + (size_t)g * a.dim, reinterpret_cast<CT *>(a.kc) + (slot * a.kv_heads + g) * a.dim);
     } else {
         const int g = unit - a.heads - a.kv_heads;
         const AT *src = reinterpret_cast<const AT *>(a.v) + row + (size_t)g * a.vdim;
         CT *out = reinterpret_cast<CT *>(a.vc) + (slot * a.kv_heads + g) * a.vdim;
-        for (int e = lane; e < a.vdim; e += 32) out[e] = from_f32<CT>(to_f32(src[e]));
+        if (FOURS && sizeof(AT) == sizeof(CT) && a.vdim % 4 == 0) {
+            for (int e = 4 * lane; e < a.vdim; e += 128) *reinterpret_cast<Four<CT> *>(out + e) = *reinterpret_cast<const Four<CT> *>(src + e);
+        } else {
+            for (int e = lane; e < a.vdim; e += 32) out[e] = from_f32<CT>(to_f32(src[e]));
+        }
     }
 }
 
@@ -103,13 +149,10 @@ __host__ __device__ inline AttentionStepSmem<CT> attention_step_smem(int rep, in
 // keys per chunk when n of them are split over at most `chunks` CTAs
 __device__ __forceinline__ int attention_chunk_keys(int n, int chunks) { return max(AS_KEYS, ((n + chunks - 1) / chunks + AS_KEYS - 1) / AS_KEYS * AS_KEYS); }
 
-// grid = (chunks, kv_heads, tokens)
+// Block (chunk, g, t) of chunks x kv_heads x tokens.  Waits for the previous launch itself.
 template <class AT, class CT>
-RNB_GLOBAL void __launch_bounds__(AS_THREADS)
-attention_step_kernel(const __grid_constant__ WindowAttentionArgs a) {
-    extern __shared__ __align__(16) uint8_t as_smem[];
-    pdl_launch_dependents();
-    const int rep = a.heads / a.kv_heads, dim = a.dim, vdim = a.vdim, g = blockIdx.y, t = blockIdx.z, chunks = gridDim.x;
+__device__ __forceinline__ void attention_step_block(const WindowAttentionArgs &a, int chunk, int g, int t, int chunks, uint8_t *as_smem) {
+    const int rep = a.heads / a.kv_heads, dim = a.dim, vdim = a.vdim;
     const AttentionStepSmem<CT> L = attention_step_smem<CT>(rep, dim, vdim);
     CT *sk = reinterpret_cast<CT *>(as_smem + L.k), *sv = reinterpret_cast<CT *>(as_smem + L.v);
     float *sq = reinterpret_cast<float *>(as_smem + L.q), *ss = reinterpret_cast<float *>(as_smem + L.s), *acc = reinterpret_cast<float *>(as_smem + L.acc);
@@ -120,23 +163,25 @@ attention_step_kernel(const __grid_constant__ WindowAttentionArgs a) {
     pdl_wait();
     const int pos0 = *a.pos0, pos = pos0 + t;
     const int n = a.window > 0 ? min(pos + 1, a.window) : pos + 1, per = attention_chunk_keys(n, chunks), active = (n + per - 1) / per;
-    if ((int)blockIdx.x >= active) return;
-    const int lo = pos + 1 - n + (int)blockIdx.x * per, hi = min(lo + per, pos + 1);
+    if (chunk >= active) return;
+    const int lo = pos + 1 - n + chunk * per, hi = min(lo + per, pos + 1);
     const int fresh = a.fresh ? pos0 : pos + 1;   // keys from here on come from the projections
     const CT *kc = reinterpret_cast<const CT *>(a.kc) + (size_t)g * dim, *vc = reinterpret_cast<const CT *>(a.vc) + (size_t)g * vdim;
     const size_t ldk = (size_t)a.kv_heads * dim, ldv = (size_t)a.kv_heads * vdim;
     auto load = [&](int base) {
         const int cached = min(min(hi, fresh) - base, AS_KEYS);   // rows that the rings hold
         if (vec) {
-            const int qk = dim / E, all = qk + vdim / E;
-            for (int i = tid; i < AS_KEYS * all; i += AS_THREADS) {
-                const int r = i / all, c = i % all, key = base + r;
-                const bool val = c >= qk, in = r < cached;
-                if (!in && key >= fresh && key < hi) continue;   // written below
+            // four threads walk along a key's rows
+            const int r = tid >> 2, q0 = tid & 3, key = base + r;
+            const bool in = r < cached;
+            if (in || key < fresh || key >= hi) {   // else written below
                 const size_t slot = (size_t)((in ? key : lo) % a.ring);
-                const CT *src = val ? vc + slot * ldv + (c - qk) * E : kc + slot * ldk + c * E;
-                const uint32_t dst = val ? smem_u32(sv + r * L.vp + (c - qk) * E) : smem_u32(sk + r * L.kp + c * E);
-                asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(in ? 16u : 0u) : "memory");
+                auto row = [&](CT *dst, const CT *src, int n) {
+                    for (int c = q0; c < n; c += 4)
+                        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + c * E)), "l"(src + c * E), "r"(in ? 16u : 0u) : "memory");
+                };
+                row(sk + r * L.kp, kc + slot * ldk, dim / E);
+                row(sv + r * L.vp, vc + slot * ldv, vdim / E);
             }
         } else {
             const int all = dim + vdim;
@@ -228,9 +273,16 @@ attention_step_kernel(const __grid_constant__ WindowAttentionArgs a) {
                 const float4 *p = reinterpret_cast<const float4 *>(ss + j * AS_KEYS);
                 const CT *v = sv + c;
                 float o0 = 0.f, o1 = 0.f;
-                auto two = [&](int r, float w) {
-                    o0 = fmaf(w, to_f32(v[r * L.vp]), o0);
-                    o1 = fmaf(w, to_f32(v[r * L.vp + 1]), o1);
+                auto two = [&](int r, float w) {   // rows are padded to 16 bytes: a pair is one access
+                    if (E == 8) {
+                        const uint32_t x = *reinterpret_cast<const uint32_t *>(v + r * L.vp);
+                        o0 = fmaf(w, bf16_lo(x), o0);
+                        o1 = fmaf(w, bf16_hi(x), o1);
+                    } else {
+                        const float2 x = *reinterpret_cast<const float2 *>(v + r * L.vp);
+                        o0 = fmaf(w, x.x, o0);
+                        o1 = fmaf(w, x.y, o1);
+                    }
                 };
 #pragma unroll 4
                 for (int r = 0; r < n4; r++) {
@@ -261,19 +313,26 @@ attention_step_kernel(const __grid_constant__ WindowAttentionArgs a) {
         return;
     }
     const size_t pl = (size_t)rep * (vdim + 2);
-    float *part = a.part + ((size_t)t * a.kv_heads + g) * chunks * pl, *mine = part + blockIdx.x * pl;
+    float *part = a.part + ((size_t)t * a.kv_heads + g) * chunks * pl, *mine = part + (size_t)chunk * pl;
     for (int i = tid; i < rep * vdim; i += AS_THREADS) __stcg(mine + i, acc[i]);
     for (int j = tid; j < rep; j += AS_THREADS) __stcg(mine + rep * vdim + j, s_m[j]), __stcg(mine + rep * (vdim + 1) + j, s_l[j]);
     if (!last_of_head(a.counters + t * a.kv_heads + g, active)) return;
     // the chunks' weights, then their weighted sum; ss is free and holds up to AS_KEYS of them per query head
     for (int j = warp; j < rep; j += AS_THREADS / 32) {
-        float m = -INFINITY, l = 0.f;
-        for (int c = lane; c < active; c += 32) m = fmaxf(m, __ldcg(part + c * pl + rep * vdim + j));
+        float mc[2], lc[2], m = -INFINITY, l = 0.f;
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            const int c = lane + 32 * i;
+            mc[i] = c < active ? __ldcg(part + c * pl + rep * vdim + j) : -INFINITY;
+            lc[i] = c < active ? __ldcg(part + c * pl + rep * (vdim + 1) + j) : 0.f;
+            m = fmaxf(m, mc[i]);
+        }
         m = warp_max(m);
-        for (int c = lane; c < active; c += 32) {
-            const float w = expf(__ldcg(part + c * pl + rep * vdim + j) - m);
-            ss[j * AS_KEYS + c] = w;
-            l = fmaf(w, __ldcg(part + c * pl + rep * (vdim + 1) + j), l);
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            const float w = expf(mc[i] - m);
+            ss[j * AS_KEYS + lane + 32 * i] = w;
+            l = fmaf(w, lc[i], l);
         }
         l = warp_sum(l);
         if (lane == 0) s_l[j] = gate_of(g * rep + j) / l;
@@ -286,6 +345,27 @@ attention_step_kernel(const __grid_constant__ WindowAttentionArgs a) {
         for (int c = 0; c < active; c++) o = fmaf(ss[j * AS_KEYS + c], __ldcg(part + c * pl + i), o);
         act[(size_t)(g * rep + j) * vdim + i % vdim] = from_f32<AT>(o * s_l[j]);
     }
+}
+
+// grid = (chunks, kv_heads, tokens)
+template <class AT, class CT>
+RNB_GLOBAL void __launch_bounds__(AS_THREADS)
+attention_step_kernel(const __grid_constant__ WindowAttentionArgs a) {
+    extern __shared__ __align__(16) uint8_t as_smem[];
+    pdl_launch_dependents();
+    attention_step_block<AT, CT>(a, blockIdx.x, blockIdx.y, blockIdx.z, gridDim.x, as_smem);
+}
+
+// Both mixers of a parallel layer, 1..8 tokens, in one launch: n_att = chunks * kv_heads * tokens blocks of attention, then
+// heads * n_jb of the delta rule.  Their counters lie apart.
+template <class CT, int TI>
+RNB_GLOBAL void __launch_bounds__(256)
+attention_delta_step_kernel(const __grid_constant__ WindowAttentionArgs a, const __grid_constant__ DeltaArgs d, int chunks, int n_att, int n_jb) {
+    extern __shared__ __align__(16) uint8_t ad_smem[];
+    pdl_launch_dependents();
+    const int b = blockIdx.x;
+    if (b < n_att) attention_step_block<float, CT>(a, b % chunks, b / chunks % a.kv_heads, b / chunks / a.kv_heads, chunks, ad_smem);
+    else delta_step_block<float, TI>(d, (b - n_att) / n_jb, (b - n_att) % n_jb, n_jb, reinterpret_cast<float *>(ad_smem));
 }
 
 }  // namespace rnb
