@@ -11,8 +11,9 @@
 //   delta_tile_kernel      walks the tiles of a head in order on tensor cores, the state in f32 accumulators
 //
 // Within a tile, with G_ts = g_{s+1} .. g_t, raw (unnormalised) keys y and queries x, and their inverse norms a, b:
-//   (I + M) U = beta (V - (G_t0 a_t y_t) S0),   M_ts = beta_t G_ts a_t a_s (y_t . y_s) for s < t
-//   o_t = b_t (G_t0 x_t S0 + sum_{s <= t} G_ts a_s (x_t . y_s) u_s),   S = G_T0 S0 + sum_s G_Ts a_s y_s u_s^T
+//   R = V - (G_t0 a_t y_t) S0,   U = N R with N = (I + M)^-1 beta,   M_ts = beta_t G_ts a_t a_s (y_t . y_s) for s < t
+//   o_t = b_t G_t0 x_t S0 + (P U)_t with P_ts = b_t G_ts a_s (x_t . y_s) for s <= t,   S = G_T0 S0 + sum_s y_s (G_Ts a_s u_s)^T
+// so that the matrices (G_Ts a_s) N and P N of a tile do not depend on the state and are made ahead of time.
 // G is summed in logarithms pair by pair and never divided.
 #pragma once
 #include "linear_state.cuh"
@@ -36,10 +37,13 @@ struct DeltaArgs {
     float *o, *act;            // o [tokens][heads][vdim]; act: rows of lda, null: o only
     int *counters;             // [heads], zero between launches
     const int *pos0;
-    bf16 *cq, *ck, *cv;        // prompts: convolved queries and keys [tokens][kv_heads][dim], values [tokens][heads][vdim]
-    uint8_t *rec;              // prompts: [tiles][heads] records
+    // prompts, as shared memory wants a tile (16 tokens): convolved queries and keys [tiles][kv_heads][2][16][ld_qk], values
+    // [tiles][heads][col_blocks][16][ld_val] (16 cw columns per block), records [tiles][heads]
+    bf16 *cqk, *cv;
+    uint8_t *rec;
+    int *err;                  // prompts: device error flag
     float eps, out_mul, q_mul;
-    int tokens, heads, kv_heads, dim, vdim, taps, k_at, v_at, g_at, a_at, ld, ld_ba, lda;
+    int tokens, heads, kv_heads, dim, vdim, taps, k_at, v_at, g_at, a_at, ld, ld_ba, lda, ld_qk, ld_val, col_blocks, cw;
 };
 
 __device__ __forceinline__ int delta_channels(const DeltaArgs &a) { return 2 * a.kv_heads * a.dim + a.heads * a.vdim; }
@@ -97,6 +101,7 @@ __device__ __forceinline__ void delta_step_block(const DeltaArgs &a, int h, int 
         prefetch_l2(w + qc + hk * dim, (size_t)dim * 4, lane, 32);
         if (lane == 0) prefetch_l2(w + 2 * qc + h * vdim + j0, 4, 0, 1);
     }
+    if (a.norm) prefetch_l2(a.norm, (size_t)vdim * 4, tid, 256);
     pdl_wait();
     float S[TI];
 #pragma unroll
@@ -196,68 +201,118 @@ delta_step_kernel(const __grid_constant__ DeltaArgs a) {
 }
 
 // ---- prompts on tensor cores ---------------------------------------------------------------------
-// Record of a tile and head: T beta (bf16 hi, lo), P (hi, lo): 16 x 16 each, row t, column s; then f32: G_t0 a_t [16],
-// G_t0 b_t [16], G_Tt a_t [16], G_T0 [1].
-constexpr int DR_MAT = 16 * 16 * 2, DR_VEC = 4 * DR_MAT, DR_REC = DR_VEC + 4 * 64;
+// Record of a tile and head: (G_Tt a_t) N (bf16 hi, lo), P N (hi, lo): 16 x 16 each, row t, column s; then f32:
+// G_t0 a_t [16], G_t0 b_t [16], G_T0 [1].
+constexpr int DR_ROW = 48, DR_MAT = 16 * DR_ROW, DR_VEC = 4 * DR_MAT, DR_REC = DR_VEC + 4 * 64;   // rows of 48 bytes: the form shared memory wants
 // tokens of a prepare CTA, and the pitch of its f32 matrices
-constexpr int DP_TILES = 4, DP_TOKENS = 16 * DP_TILES, DP_PITCH = 20, DP_WORK = 16 * DP_PITCH + 32;
+constexpr int DP_TILES = 4, DP_TOKENS = 16 * DP_TILES, DP_PITCH = 20, DP_WORK = 2 * 16 * DP_PITCH + 16;
 __host__ __device__ inline size_t delta_prepare_smem(int dim) {
     return (size_t)2 * DP_TOKENS * (dim + 8) * 2 + ((size_t)2 * DP_TILES * 16 * DP_PITCH + 2 * DP_TOKENS + 16 * DP_WORK) * 4;
 }
 
+// Convolution and silu of 8 channels (column `col` of the projections, taps from channel c on) at the 16 tokens from t on:
+// put(i, eight bf16) for each of them, zeros from token `end` on.  TAPS: their number, 0 for any.
+template <int TAPS, class Put>
+__device__ __forceinline__ void delta_convolve16(const DeltaArgs &a, int c, int col, int t, int end, int pos0, Put put) {
+    const int taps = TAPS ? TAPS : a.taps, C = delta_channels(a);
+    const bf16 *p = reinterpret_cast<const bf16 *>(a.p) + col;
+    auto row = [&](int at, float (&v)[8]) {
+        if (at >= 0) {
+            const uint4 b = *reinterpret_cast<const uint4 *>(p + (size_t)min(at, a.tokens - 1) * a.ld);
+            const uint32_t r[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+            for (int e = 0; e < 4; e++) v[2 * e] = bf16_lo(r[e]), v[2 * e + 1] = bf16_hi(r[e]);
+        } else {
+#pragma unroll
+            for (int e = 0; e < 8; e++) v[e] = delta_input<bf16>(a, c + e, col + e, at, pos0);
+        }
+    };
+    auto weights = [&](int n, float (&w)[8]) {
+        const float4 x = *reinterpret_cast<const float4 *>(a.conv + (size_t)n * C + c), y = *reinterpret_cast<const float4 *>(a.conv + (size_t)n * C + c + 4);
+        w[0] = x.x, w[1] = x.y, w[2] = x.z, w[3] = x.w, w[4] = y.x, w[5] = y.y, w[6] = y.z, w[7] = y.w;
+    };
+    auto finish = [&](int i, const float (&y)[8]) {
+        uint32_t r[4] = {0u, 0u, 0u, 0u};
+        if (t + i < end) {
+#pragma unroll
+            for (int e = 0; e < 4; e++) r[e] = pg_pack_bf16(silu_fast(y[2 * e]), silu_fast(y[2 * e + 1]));
+        }
+        put(i, make_uint4(r[0], r[1], r[2], r[3]));
+    };
+    if (TAPS) {
+        constexpr int N = TAPS ? TAPS : 1;
+        float w[N][8], x[N][8];   // x: a ring of the last rows
+#pragma unroll
+        for (int n = 0; n < N; n++) weights(n, w[n]);
+#pragma unroll
+        for (int n = 0; n < N - 1; n++) row(t - (N - 1) + n, x[n]);
+#pragma unroll
+        for (int i = 0; i < 16; i++) {
+            row(t + i, x[(i + N - 1) % N]);
+            float y[8] = {};
+#pragma unroll
+            for (int n = 0; n < N; n++)
+#pragma unroll
+                for (int e = 0; e < 8; e++) y[e] = fmaf(w[n][e], x[(i + n) % N][e], y[e]);
+            finish(i, y);
+        }
+    } else {
+        for (int i = 0; i < 16; i++) {
+            float y[8] = {};
+            for (int n = 0; n < taps; n++) {
+                float w[8], x[8];
+                weights(n, w);
+                row(t + i - (taps - 1) + n, x);
+#pragma unroll
+                for (int e = 0; e < 8; e++) y[e] = fmaf(w[e], x[e], y[e]);
+            }
+            finish(i, y);
+        }
+    }
+}
+
 // grid = (ceil(tokens / 64), kv_heads), 256 threads.  dim and vdim multiples of 8, dim of 16.
+template <int TAPS>
 RNB_GLOBAL void __launch_bounds__(256, 2)
 delta_prepare_kernel(const __grid_constant__ DeltaArgs a) {
     extern __shared__ __align__(16) uint8_t dp_smem[];
     pdl_launch_dependents();
     pdl_wait();
     const int dim = a.dim, rep = a.heads / a.kv_heads, hk = blockIdx.y, t0 = blockIdx.x * DP_TOKENS, nt = min(DP_TOKENS, a.tokens - t0), pos0 = *a.pos0;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, KE = dim + 8, qc = a.kv_heads * dim, C = delta_channels(a);
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, KE = dim + 8, qc = a.kv_heads * dim;
     bf16 *sx = reinterpret_cast<bf16 *>(dp_smem), *sy = sx + DP_TOKENS * KE;
     float *xy = reinterpret_cast<float *>(sy + DP_TOKENS * KE), *yy = xy + DP_TILES * 16 * DP_PITCH, *nrm = yy + DP_TILES * 16 * DP_PITCH, *work = nrm + 2 * DP_TOKENS;
-    const bf16 *p = reinterpret_cast<const bf16 *>(a.p);
-    // convolutions: 8 channels of 4 tokens at a time; rows past the end become zeros
+    // convolutions: 8 channels of a tile at a time; rows past the end become zeros
     const int units = (2 * dim + rep * a.vdim) / 8;
-    for (int i = tid; i < units * (DP_TOKENS / 4); i += 256) {
-        const int u = i % units, ts = i / units * 4, x = u * 8;
+    for (int i = tid; i < units * DP_TILES; i += 256) {
+        const int u = i % units, ts = i / units * 16, x = u * 8;
+        if (ts >= nt) {   // no such tile: only the rows that the products below read
+            if (x < 2 * dim)
+                for (int k = 0; k < 16; k++) *reinterpret_cast<uint4 *>((x < dim ? sx + x : sy + x - dim) + (ts + k) * KE) = make_uint4(0u, 0u, 0u, 0u);
+            continue;
+        }
         const int c = x < dim ? hk * dim + x : x < 2 * dim ? qc + hk * dim + x - dim : 2 * qc + hk * rep * a.vdim + x - 2 * dim;
-        const int col = delta_col(a, c);
-        float y[4][8] = {};
-        for (int n = 0; n < a.taps; n++) {
-            const float4 wa = *reinterpret_cast<const float4 *>(a.conv + (size_t)n * C + c), wb = *reinterpret_cast<const float4 *>(a.conv + (size_t)n * C + c + 4);
-            const float w[8] = {wa.x, wa.y, wa.z, wa.w, wb.x, wb.y, wb.z, wb.w};
-#pragma unroll
-            for (int q = 0; q < 4; q++) {
-                const int t = t0 + ts + q - (a.taps - 1) + n;
-                if (ts + q >= nt) continue;
-                float v[8];
-                if (t >= 0) {
-                    const uint4 b = *reinterpret_cast<const uint4 *>(p + (size_t)t * a.ld + col);
-                    const uint32_t r[4] = {b.x, b.y, b.z, b.w};
-#pragma unroll
-                    for (int e = 0; e < 4; e++) v[2 * e] = bf16_lo(r[e]), v[2 * e + 1] = bf16_hi(r[e]);
-                } else {
-#pragma unroll
-                    for (int e = 0; e < 8; e++) v[e] = delta_input<bf16>(a, c + e, col + e, t, pos0);
-                }
-#pragma unroll
-                for (int e = 0; e < 8; e++) y[q][e] = fmaf(w[e], v[e], y[q][e]);
-            }
+        const size_t tile = (size_t)blockIdx.x * DP_TILES + (i / units);
+        bf16 *near = nullptr, *far;
+        int ld = a.ld_qk;
+        if (x < 2 * dim) {
+            const int key = x >= dim, ch = key ? x - dim : x;
+            near = (key ? sy : sx) + ts * KE + ch;
+            far = a.cqk + ((tile * a.kv_heads + hk) * 2 + key) * 16 * ld + ch;
+        } else {
+            const int j = (x - 2 * dim) % a.vdim, h = hk * rep + (x - 2 * dim) / a.vdim, w = 16 * a.cw;
+            ld = a.ld_val;
+            far = a.cv + ((tile * a.heads + h) * a.col_blocks + j / w) * 16 * ld + j % w;
         }
-#pragma unroll
-        for (int q = 0; q < 4; q++) {
-            const int t = ts + q;
-            uint32_t r[4];
-#pragma unroll
-            for (int e = 0; e < 4; e++) r[e] = pg_pack_bf16(silu_fast(y[q][2 * e]), silu_fast(y[q][2 * e + 1]));
-            const uint4 b = make_uint4(r[0], r[1], r[2], r[3]);
-            if (x < 2 * dim) *reinterpret_cast<uint4 *>((x < dim ? sx + x : sy + x - dim) + t * KE) = b;
-            if (t >= nt) continue;
-            const size_t row = (size_t)(t0 + t);
-            if (x < dim) *reinterpret_cast<uint4 *>(a.cq + (row * a.kv_heads + hk) * dim + x) = b;
-            else if (x < 2 * dim) *reinterpret_cast<uint4 *>(a.ck + (row * a.kv_heads + hk) * dim + x - dim) = b;
-            else *reinterpret_cast<uint4 *>(a.cv + (row * a.heads + hk * rep) * a.vdim + x - 2 * dim) = b;
-        }
+        delta_convolve16<TAPS>(a, c, delta_col(a, c), t0 + ts, a.tokens, pos0, [&](int k, uint4 b) {
+            if (near) *reinterpret_cast<uint4 *>(near + k * KE) = b;
+            *reinterpret_cast<uint4 *>(far + k * ld) = b;
+        });
+    }
+    if (dim + 8 < a.ld_qk) {   // channels that the tile kernel has beyond dim
+        const int pad = (a.ld_qk - 8 - dim) / 8, rows = (nt + 15) / 16 * 32;
+        for (int i = tid; i < rows * pad; i += 256)
+            *reinterpret_cast<uint4 *>(a.cqk + (((size_t)(blockIdx.x * DP_TILES + i / pad / 32) * a.kv_heads + hk) * 32 + i / pad % 32) * a.ld_qk + dim + i % pad * 8) = make_uint4(0u, 0u, 0u, 0u);
     }
     __syncthreads();
     // inverse norms, queries first, eight lanes per row
@@ -295,19 +350,19 @@ delta_prepare_kernel(const __grid_constant__ DeltaArgs a) {
     __syncthreads();
     // half a warp per tile and head; lane s of it = column s of the matrices
     const int s = lane & 15, half = warp * 2 + (lane >> 4), tasks = min(DP_TILES, (nt + 15) / 16) * rep;
-    float *M = work + half * DP_WORK, *lg = M + 16 * DP_PITCH, *bt = lg + 16;
+    float *M = work + half * DP_WORK, *P = M + 16 * DP_PITCH, *lg = P + 16 * DP_PITCH;
     for (int base = 0; base < tasks; base += 16) {
         const int task = base + half;
         const bool on = task < tasks;
         const int tile = on ? task / rep : 0, h = hk * rep + (on ? task % rep : 0), tk = tile * 16, left = nt - tk;
         const float *nq = nrm + tk, *nk = nrm + DP_TOKENS + tk, *xt = xy + tile * 16 * DP_PITCH, *yt = yy + tile * 16 * DP_PITCH;
         const float *ba = a.ba + (size_t)(t0 + tk + min(s, left - 1)) * a.ld_ba;
-        const float l = s < left ? -expf(a.a_log[h]) * softplus_f32(ba[a.a_at + h] + a.dt[h]) : 0.f, b = s < left ? sigmoid_f32(ba[h]) : 0.f;
-        lg[s] = l;
-        bt[s] = b;
+        const float b = s < left ? sigmoid_f32(ba[h]) : 0.f;
+        lg[s] = s < left ? -expf(a.a_log[h]) * softplus_f32(ba[a.a_at + h] + a.dt[h]) : 0.f;
         __syncwarp();
         uint8_t *rec = a.rec + ((size_t)(blockIdx.x * DP_TILES + tile) * a.heads + h) * DR_REC;
-        bf16 *Thi = reinterpret_cast<bf16 *>(rec), *Tlo = Thi + 256, *Phi = Tlo + 256, *Plo = Phi + 256;
+        constexpr int RE = DR_ROW / 2, ME = DR_MAT / 2;
+        bf16 *Whi = reinterpret_cast<bf16 *>(rec), *Wlo = Whi + ME, *Qhi = Wlo + ME, *Qlo = Qhi + ME;
         float acc = 0.f, head = 0.f;   // logarithms of G_ts, and of G_s0
         const float ns = nk[s];
 #pragma unroll
@@ -315,40 +370,47 @@ delta_prepare_kernel(const __grid_constant__ DeltaArgs a) {
             if (t <= s) head += lg[t];
             else acc += lg[t];
             const float e = t >= s ? expf(acc) * ns : 0.f;
-            M[t * DP_PITCH + s] = t > s ? bt[t] * nk[t] * e * yt[t * DP_PITCH + s] : 0.f;
-            if (on) lt_split_store(Phi + t * 16 + s, Plo + t * 16 + s, nq[t] * e * xt[t * DP_PITCH + s]);
+            const float bt = __shfl_sync(0xffffffffu, b, t, 16);
+            M[t * DP_PITCH + s] = t > s ? bt * nk[t] * e * yt[t * DP_PITCH + s] : 0.f;
+            P[t * DP_PITCH + s] = nq[t] * e * xt[t * DP_PITCH + s];
         }
+        const float from0 = expf(head), to_end = expf(acc) * ns;
         if (on) {
             float *vec = reinterpret_cast<float *>(rec + DR_VEC);
-            const float from0 = expf(head);
             vec[s] = from0 * ns;
             vec[16 + s] = from0 * nq[s];
-            vec[32 + s] = expf(acc) * ns;
-            if (s == 15) vec[48] = from0;
+            if (s == 15) vec[32] = from0;
         }
         __syncwarp();
-        // column s of (I + M)^-1 by forward substitution
+        // column s of N by forward substitution
         float x[16];
+        auto dot = [&](const float *row, int n, float first) {   // first + the first n elements of a row times x
+            float v[4] = {first, 0.f, 0.f, 0.f};
 #pragma unroll
-        for (int t = 0; t < 16; t++) {
-            float v[4] = {t == s ? 1.f : 0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-            for (int q4 = 0; q4 < (t + 3) / 4; q4++) {
-                const float4 m = *reinterpret_cast<const float4 *>(M + t * DP_PITCH + 4 * q4);
+            for (int q4 = 0; q4 < 4; q4++) {
+                if (4 * q4 >= n) break;
+                const float4 m = *reinterpret_cast<const float4 *>(row + 4 * q4);
                 const float mv[4] = {m.x, m.y, m.z, m.w};
 #pragma unroll
                 for (int e = 0; e < 4; e++)
-                    if (4 * q4 + e < t) v[e] = fmaf(-mv[e], x[4 * q4 + e], v[e]);
+                    if (4 * q4 + e < n) v[e] = fmaf(mv[e], x[4 * q4 + e], v[e]);
             }
-            x[t] = (v[0] + v[1]) + (v[2] + v[3]);
-            if (on) lt_split_store(Thi + t * 16 + s, Tlo + t * 16 + s, x[t] * b);
+            return (v[0] + v[1]) + (v[2] + v[3]);
+        };
+#pragma unroll
+        for (int t = 0; t < 16; t++) x[t] = (t == s ? b : 0.f) - dot(M + t * DP_PITCH, t, 0.f);
+#pragma unroll
+        for (int t = 0; t < 16; t++) {
+            const float q = dot(P + t * DP_PITCH, t + 1, 0.f), w = __shfl_sync(0xffffffffu, to_end, t, 16) * x[t];
+            if (!on) continue;
+            lt_split_store(Whi + t * RE + s, Wlo + t * RE + s, w);
+            lt_split_store(Qhi + t * RE + s, Qlo + t * RE + s, q);
         }
         __syncwarp();
     }
 }
 
-constexpr int DT_STAGES = 4;
-__host__ __device__ constexpr int delta_tile_split(int DT) { return DT >= 4 ? 4 : 2; }   // warps that share the channels of 16 value columns
+constexpr int DT_STAGES = 4, DT_SPLIT = 2;   // DT_SPLIT: warps that share the channels of 16 value columns
 struct DeltaTileSmem {
     uint32_t kp, vp, y, v, mat, vec, stage, sums, bytes;
 };
@@ -358,200 +420,229 @@ __host__ __device__ inline DeltaTileSmem delta_tile_smem(int DT, int CW) {
     s.vp = (uint32_t)(16 * CW + 8) * 2;
     s.y = 16 * s.kp;                 // x at 0
     s.v = s.y + 16 * s.kp;
-    s.mat = s.v + 16 * s.vp;         // four matrices, rows of 48 bytes
-    s.vec = s.mat + 4 * 16 * 48;
-    s.stage = s.vec + 256;
+    s.mat = s.v + 16 * s.vp;         // four matrices, rows of 48 bytes, then the record's vectors
+    s.vec = s.mat + DR_VEC;
+    s.stage = s.mat + DR_REC;
     s.sums = DT_STAGES * s.stage;    // partial products [2][CW][split][4][32 lanes] float4
-    s.bytes = s.sums + (uint32_t)(2 * CW * delta_tile_split(DT) * 4 * 32 * 16);
+    s.bytes = s.sums + (uint32_t)(2 * CW * DT_SPLIT * 4 * 32 * 16);
     return s;
 }
-// grid = (heads, column blocks), blockDim = 32 * split * CW: 16 value columns per group of `split` warps, each of which holds
-// S^T for its share of the channels.  The products with the state are summed over the group through shared memory.
+// grid = (heads, column blocks), blockDim = 32 * (DT_SPLIT * cw + 1): 16 value columns per group of DT_SPLIT warps, each of which
+// holds S^T for its share of the channels; the last warp has a tile's queries and keys, values and record copied into a ring of stages
+// (three bulk copies).  The products with the state are summed over the group through shared memory; its first two warps finish
+// eight of a tile's tokens each.
+// Waits are bounded; one that gives up sets the error flag, and every copy that was started is waited for before the CTA ends.
 // dim <= 16 DT a multiple of 16, vdim of 8.
 template <int DT>
-RNB_GLOBAL void __launch_bounds__(256)
+RNB_GLOBAL void __launch_bounds__(160)
 delta_tile_kernel(const __grid_constant__ DeltaArgs a) {
     extern __shared__ __align__(128) uint8_t dt_smem[];
+    __shared__ __align__(8) uint64_t full[DT_STAGES], empty[DT_STAGES];
+    __shared__ int s_failed;
     pdl_launch_dependents();
-    pdl_wait();
-    constexpr int KS = delta_tile_split(DT), DW = DT / KS;   // channel blocks of 16 per warp
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nthr = blockDim.x, CW = nthr / (32 * KS), grp = warp / KS, part = warp % KS;
+    constexpr int KS = DT_SPLIT, DW = DT / KS;   // channel blocks of 16 per warp
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, CW = a.cw, grp = warp / KS, part = warp % KS;
     const DeltaTileSmem L = delta_tile_smem(DT, CW);
     const uint32_t base = smem_u32(dt_smem);
     const int h = blockIdx.x, j0 = blockIdx.y * 16 * CW, hk = h / (a.heads / a.kv_heads), n_tiles = (a.tokens + 15) / 16, vdim = a.vdim;
-    const size_t ldk = (size_t)a.kv_heads * a.dim, ldv = (size_t)a.heads * vdim;
-    const bf16 *xp = a.cq + (size_t)hk * a.dim, *yp = a.ck + (size_t)hk * a.dim, *vp = a.cv + (size_t)h * vdim;
-    auto cp16 = [&](uint32_t dst, const void *src, bool in) {
-        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(in ? 16u : 0u) : "memory");
-    };
-    auto load_tile = [&](int i) {
-        if (i < n_tiles) {
-            const uint32_t st = base + (uint32_t)(i % DT_STAGES) * L.stage;
-            const int t0 = 16 * i;
-            for (int x = tid; x < 16 * 2 * DT; x += nthr) {
-                const int t = x / (2 * DT), q = x % (2 * DT);
-                const bool in = t0 + t < a.tokens && q * 8 < a.dim;
-                const size_t at = (size_t)min(t0 + t, a.tokens - 1) * ldk + min(q * 8, a.dim - 8);
-                cp16(st + (uint32_t)t * L.kp + (uint32_t)q * 16u, xp + at, in);
-                cp16(st + L.y + (uint32_t)t * L.kp + (uint32_t)q * 16u, yp + at, in);
-            }
-            for (int x = tid; x < 16 * 2 * CW; x += nthr) {
-                const int t = x & 15, q = x >> 4, col = j0 + q * 8;
-                cp16(st + L.v + (uint32_t)t * L.vp + (uint32_t)q * 16u, vp + (size_t)min(t0 + t, a.tokens - 1) * ldv + min(col, vdim - 8), t0 + t < a.tokens && col < vdim);
-            }
-            const uint8_t *rec = a.rec + ((size_t)i * a.heads + h) * DR_REC;
-            for (int x = tid; x < DR_REC / 16; x += nthr)
-                cp16(x < DR_VEC / 16 ? st + L.mat + (uint32_t)(x >> 1) * 48u + (uint32_t)(x & 1) * 16u : st + L.vec + (uint32_t)(x - DR_VEC / 16) * 16u, rec + x * 16, true);
+    const size_t ldv = (size_t)a.heads * vdim;
+    if (tid == 0) {
+        for (int i = 0; i < DT_STAGES; i++) {
+            mbar_init(&full[i], 1);
+            mbar_init(&empty[i], (uint32_t)(KS * CW));
         }
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    };
-    for (int i = 0; i < DT_STAGES - 1; i++) load_tile(i);
-    {   // the ring for the next call's convolutions: every column block takes its share of the head's channels
-        const int rep = a.heads / a.kv_heads, qc = a.kv_heads * a.dim, pos0 = *a.pos0, step = nthr * gridDim.y, first = blockIdx.y * nthr + tid;
-        if (h % rep == 0) {
-            delta_ring_store<bf16>(a, hk * a.dim + first, step, (hk + 1) * a.dim, pos0);
-            delta_ring_store<bf16>(a, qc + hk * a.dim + first, step, qc + (hk + 1) * a.dim, pos0);
-        }
-        delta_ring_store<bf16>(a, 2 * qc + h * vdim + first, step, 2 * qc + (h + 1) * vdim, pos0);
+        mbar_fence_init();
+        s_failed = 0;
     }
-    const int g = lane >> 2, tq = lane & 3, mi = lane >> 3, mr = lane & 7, jw = j0 + grp * 16, c0 = part * DW * 16;
-    float S[2 * DW][4];
-    auto state_io = [&](bool store) {
+    __syncthreads();
+    pdl_wait();
+    if (warp == KS * CW) {
+        int issued = 0;
+        bool ok = true;
+        if (lane == 0) {
+            const uint32_t qk = 32 * L.kp, val = 16 * L.vp;
+            for (int i = 0; i < n_tiles; i++) {
+                const int sl = i % DT_STAGES;
+                ok = mbar_wait_bounded(&empty[sl], (uint32_t)(((i / DT_STAGES) & 1) ^ 1));
+                if (!ok) break;
+                uint8_t *st = dt_smem + (size_t)sl * L.stage;
+                mbar_arrive_expect_tx(&full[sl], qk + val + DR_REC);
+                bulk_g2s(st, a.cqk + ((size_t)i * a.kv_heads + hk) * 32 * a.ld_qk, qk, &full[sl]);
+                bulk_g2s(st + L.v, a.cv + (((size_t)i * a.heads + h) * a.col_blocks + blockIdx.y) * 16 * a.ld_val, val, &full[sl]);
+                bulk_g2s(st + L.mat, a.rec + ((size_t)i * a.heads + h) * DR_REC, DR_REC, &full[sl]);
+                issued = i + 1;
+            }
+        }
+        if (!ok && lane == 0) atomicExch(&s_failed, 1);
+        // a CTA ends after its copies
+        for (int i = max(0, issued - DT_STAGES); i < issued; i++) mbar_wait_bounded(&full[i % DT_STAGES], (uint32_t)((i / DT_STAGES) & 1));
+    } else {
+        {   // the ring for the next call's convolutions: every column block takes its share of the head's channels
+            const int rep = a.heads / a.kv_heads, qc = a.kv_heads * a.dim, pos0 = *a.pos0, step = 32 * KS * CW * gridDim.y, first = blockIdx.y * 32 * KS * CW + tid;
+            if (h % rep == 0) {
+                delta_ring_store<bf16>(a, hk * a.dim + first, step, (hk + 1) * a.dim, pos0);
+                delta_ring_store<bf16>(a, qc + hk * a.dim + first, step, qc + (hk + 1) * a.dim, pos0);
+            }
+            delta_ring_store<bf16>(a, 2 * qc + h * vdim + first, step, 2 * qc + (h + 1) * vdim, pos0);
+        }
+        const int g = lane >> 2, tq = lane & 3, mi = lane >> 3, mr = lane & 7, jw = j0 + grp * 16, c0 = part * DW * 16;
+        float S[2 * DW][4];
+        auto state_io = [&](bool store) {
 #pragma unroll
-        for (int n = 0; n < 2 * DW; n++)
+            for (int n = 0; n < 2 * DW; n++)
 #pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const int ch = c0 + n * 8 + 2 * tq + (e & 1), j = jw + g + 8 * (e >> 1);
-                const bool in = j < vdim && ch < a.dim;
-                float *p = a.state + ((size_t)h * a.dim + ch) * vdim + j;
-                if (store) {
-                    if (in) *p = S[n][e];
+                for (int e = 0; e < 4; e++) {
+                    const int ch = c0 + n * 8 + 2 * tq + (e & 1), j = jw + g + 8 * (e >> 1);
+                    const bool in = j < vdim && ch < a.dim;
+                    float *p = a.state + ((size_t)h * a.dim + ch) * vdim + j;
+                    if (store) {
+                        if (in) *p = S[n][e];
+                    } else {
+                        S[n][e] = in ? *p : 0.f;
+                    }
+                }
+        };
+        state_io(false);
+        const uint32_t b_plain = (uint32_t)((mi >> 1) * 8 + mr) * L.kp + (uint32_t)(mi & 1) * 16u + (uint32_t)c0 * 2u;        // rows (n), k contiguous
+        const uint32_t b_trans = (uint32_t)((mi & 1) * 8 + mr) * L.kp + (uint32_t)(mi >> 1) * 16u + (uint32_t)c0 * 2u;        // rows (k), n contiguous
+        const uint32_t b_mat = L.mat + (uint32_t)((mi >> 1) * 8 + mr) * DR_ROW + (uint32_t)(mi & 1) * 16u;
+        const uint32_t b_out = L.mat + (uint32_t)(2 + (mi >> 1)) * DR_MAT + (uint32_t)(part * 8 + mr) * DR_ROW + (uint32_t)(mi & 1) * 16u;   // hi, lo of eight rows
+        const uint32_t b_val = L.v + (uint32_t)((mi >> 1) * 8 + mr) * L.vp + (uint32_t)(grp * 32 + (mi & 1) * 16);
+        float4 *sums = reinterpret_cast<float4 *>(dt_smem + L.sums) + (size_t)grp * KS * 128 + lane;
+        float *to = a.o + (size_t)(part * 8 + 2 * tq) * ldv + (size_t)h * vdim + jw + g;
+        const bool col0 = jw + g < vdim, col1 = jw + g + 8 < vdim;
+        bool ok = true;
+        for (int it = 0; it < n_tiles; it++, to += 16 * ldv) {
+            const int sl = it % DT_STAGES;
+            if (ok) ok = mbar_wait_bounded(&full[sl], (uint32_t)((it / DT_STAGES) & 1));
+            ok = __all_sync(0xffffffffu, ok);
+            const uint32_t st = base + (uint32_t)sl * L.stage;
+            const float *vec = reinterpret_cast<const float *>(dt_smem + (size_t)sl * L.stage + L.vec);
+            // this warp's part of (S0^T y, S0^T x): state hi + lo, exact bf16 rows
+            float X[4][4], Y[4][4];
+#pragma unroll
+            for (int ks = 0; ks < DW; ks++) {
+                uint32_t sh[4], s2[4], by[4], bx[4];
+                lt_ldmatrix_x4(by, st + L.y + b_plain + (uint32_t)ks * 32u);
+                lt_ldmatrix_x4(bx, st + b_plain + (uint32_t)ks * 32u);
+                lt_split(S[2 * ks][0], S[2 * ks][1], sh[0], s2[0]);
+                lt_split(S[2 * ks][2], S[2 * ks][3], sh[1], s2[1]);
+                lt_split(S[2 * ks + 1][0], S[2 * ks + 1][1], sh[2], s2[2]);
+                lt_split(S[2 * ks + 1][2], S[2 * ks + 1][3], sh[3], s2[3]);
+                if (ks == 0) {
+                    lt_mma_zero(X[0], sh, by[0], by[1]);
+                    lt_mma_zero(X[1], sh, by[2], by[3]);
+                    lt_mma_zero(X[2], s2, by[0], by[1]);
+                    lt_mma_zero(X[3], s2, by[2], by[3]);
+                    lt_mma_zero(Y[0], sh, bx[0], bx[1]);
+                    lt_mma_zero(Y[1], sh, bx[2], bx[3]);
+                    lt_mma_zero(Y[2], s2, bx[0], bx[1]);
+                    lt_mma_zero(Y[3], s2, bx[2], bx[3]);
                 } else {
-                    S[n][e] = in ? *p : 0.f;
+                    lt_mma(X[0], sh, by[0], by[1]);
+                    lt_mma(X[1], sh, by[2], by[3]);
+                    lt_mma(X[2], s2, by[0], by[1]);
+                    lt_mma(X[3], s2, by[2], by[3]);
+                    lt_mma(Y[0], sh, bx[0], bx[1]);
+                    lt_mma(Y[1], sh, bx[2], bx[3]);
+                    lt_mma(Y[2], s2, bx[0], bx[1]);
+                    lt_mma(Y[3], s2, bx[2], bx[3]);
                 }
             }
-    };
-    state_io(false);
-    const uint32_t b_plain = (uint32_t)((mi >> 1) * 8 + mr) * L.kp + (uint32_t)(mi & 1) * 16u + (uint32_t)c0 * 2u;        // rows (n), k contiguous
-    const uint32_t b_trans = (uint32_t)((mi & 1) * 8 + mr) * L.kp + (uint32_t)(mi >> 1) * 16u + (uint32_t)c0 * 2u;        // rows (k), n contiguous
-    const uint32_t b_mat = (uint32_t)((mi >> 1) * 8 + mr) * 48u + (uint32_t)(mi & 1) * 16u;
-    float4 *sums = reinterpret_cast<float4 *>(dt_smem + L.sums) + (size_t)grp * KS * 128;
-    for (int it = 0; it < n_tiles; it++) {
-        asm volatile("cp.async.wait_group %0;" ::"n"(DT_STAGES - 2) : "memory");
-        __syncthreads();   // the tile is in, and every warp is through with the one whose stage is loaded next
-        load_tile(it + DT_STAGES - 1);
-        const uint32_t st = base + (uint32_t)(it % DT_STAGES) * L.stage;
-        const uint8_t *raw = dt_smem + (size_t)(it % DT_STAGES) * L.stage;
-        const float *vec = reinterpret_cast<const float *>(raw + L.vec);
-        // this warp's part of (S0^T y, S0^T x): state hi + lo, exact bf16 rows
-        float X[4][4] = {}, Y[4][4] = {};
+            float4 *box = sums + (size_t)(it & 1) * CW * KS * 128;
 #pragma unroll
-        for (int ks = 0; ks < DW; ks++) {
-            uint32_t sh[4], sl[4], by[4], bx[4];
-            lt_split(S[2 * ks][0], S[2 * ks][1], sh[0], sl[0]);
-            lt_split(S[2 * ks][2], S[2 * ks][3], sh[1], sl[1]);
-            lt_split(S[2 * ks + 1][0], S[2 * ks + 1][1], sh[2], sl[2]);
-            lt_split(S[2 * ks + 1][2], S[2 * ks + 1][3], sh[3], sl[3]);
-            lt_ldmatrix_x4(by, st + L.y + b_plain + (uint32_t)ks * 32u);
-            lt_ldmatrix_x4(bx, st + b_plain + (uint32_t)ks * 32u);
-            lt_mma(X[0], sh, by[0], by[1]);
-            lt_mma(X[1], sh, by[2], by[3]);
-            lt_mma(X[2], sl, by[0], by[1]);
-            lt_mma(X[3], sl, by[2], by[3]);
-            lt_mma(Y[0], sh, bx[0], bx[1]);
-            lt_mma(Y[1], sh, bx[2], bx[3]);
-            lt_mma(Y[2], sl, bx[0], bx[1]);
-            lt_mma(Y[3], sl, bx[2], bx[3]);
-        }
-        float4 *mine = sums + (size_t)(it & 1) * CW * KS * 128, *put = mine + part * 128 + lane;
-#pragma unroll
-        for (int n = 0; n < 2; n++) {
-            put[n * 32] = make_float4(X[n][0] + X[n + 2][0], X[n][1] + X[n + 2][1], X[n][2] + X[n + 2][2], X[n][3] + X[n + 2][3]);
-            put[(n + 2) * 32] = make_float4(Y[n][0] + Y[n + 2][0], Y[n][1] + Y[n + 2][1], Y[n][2] + Y[n + 2][2], Y[n][3] + Y[n + 2][3]);
-        }
-        asm volatile("bar.sync %0, %1;" ::"r"(1 + grp), "n"(32 * KS) : "memory");
-        auto total = [&](int n, float (&o)[4]) {
-            o[0] = o[1] = o[2] = o[3] = 0.f;
-#pragma unroll
-            for (int k = 0; k < KS; k++) {
-                const float4 v = mine[k * 128 + n * 32 + lane];
-                o[0] += v.x, o[1] += v.y, o[2] += v.z, o[3] += v.w;
+            for (int n = 0; n < 2; n++) {
+                box[part * 128 + n * 32] = make_float4(X[n][0] + X[n + 2][0], X[n][1] + X[n + 2][1], X[n][2] + X[n + 2][2], X[n][3] + X[n + 2][3]);
+                box[part * 128 + 64 + n * 32] = make_float4(Y[n][0] + Y[n + 2][0], Y[n][1] + Y[n + 2][1], Y[n][2] + Y[n + 2][2], Y[n][3] + Y[n + 2][3]);
             }
-        };
-        // V - G_t0 a_t S0^T y
-        const bf16 *sv = reinterpret_cast<const bf16 *>(raw + L.v);
-        const int VE = (int)(L.vp / 2);
-        float R[2][4];
+            uint32_t v4[4], bh[4], bl[4];
+            lt_ldmatrix_x4_trans(v4, st + b_val);
+            lt_ldmatrix_x4(bh, st + b_mat);
+            lt_ldmatrix_x4(bl, st + b_mat + DR_MAT);
+            asm volatile("bar.sync %0, %1;" ::"r"(1 + grp), "n"(32 * KS) : "memory");
+            auto total = [&](int n) {
+                float4 q = box[n * 32];
 #pragma unroll
-        for (int n = 0; n < 2; n++) {
-            float x[4];
-            total(n, x);
+                for (int k = 1; k < KS; k++) {
+                    const float4 v = box[k * 128 + n * 32];
+                    q.x += v.x, q.y += v.y, q.z += v.z, q.w += v.w;
+                }
+                return q;
+            };
+            // R^T = V^T - G_t0 a_t S0^T y
+            float R[2][4];
 #pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const int t = n * 8 + 2 * tq + (e & 1);
-                R[n][e] = fmaf(-vec[t], x[e], to_f32(sv[t * VE + grp * 16 + g + 8 * (e >> 1)]));
+            for (int n = 0; n < 2; n++) {
+                const float4 q = total(n);
+                const float2 f = *reinterpret_cast<const float2 *>(vec + n * 8 + 2 * tq);
+                R[n][0] = fmaf(-f.x, q.x, bf16_lo(v4[2 * n]));
+                R[n][1] = fmaf(-f.y, q.y, bf16_hi(v4[2 * n]));
+                R[n][2] = fmaf(-f.x, q.z, bf16_lo(v4[2 * n + 1]));
+                R[n][3] = fmaf(-f.y, q.w, bf16_hi(v4[2 * n + 1]));
             }
-        }
-        auto split_tile = [&](const float (&m)[2][4], uint32_t (&hi)[4], uint32_t (&lo)[4]) {
-            lt_split(m[0][0], m[0][1], hi[0], lo[0]);
-            lt_split(m[0][2], m[0][3], hi[1], lo[1]);
-            lt_split(m[1][0], m[1][1], hi[2], lo[2]);
-            lt_split(m[1][2], m[1][3], hi[3], lo[3]);
-        };
-        uint32_t hi[4], lo[4], bh[4], bl[4];
-        split_tile(R, hi, lo);
-        lt_ldmatrix_x4(bh, st + L.mat + b_mat);
-        lt_ldmatrix_x4(bl, st + L.mat + 16 * 48 + b_mat);
-        float U[2][4] = {}, U2[2][4] = {}, W[2][4];
-        lt_mma(U[0], hi, bh[0], bh[1]);
-        lt_mma(U[1], hi, bh[2], bh[3]);
-        lt_mma(U2[0], lo, bh[0], bh[1]);
-        lt_mma(U2[1], lo, bh[2], bh[3]);
-        lt_mma(U2[0], hi, bl[0], bl[1]);
-        lt_mma(U2[1], hi, bl[2], bl[3]);
-#pragma unroll
-        for (int n = 0; n < 2; n++)
-#pragma unroll
-            for (int e = 0; e < 4; e++) {
-                U[n][e] += U2[n][e];
-                W[n][e] = U[n][e] * vec[32 + n * 8 + 2 * tq + (e & 1)];
-            }
-        // the state moves on first: the next tile waits for it
-        uint32_t wh[4], wl[4];
-        split_tile(W, wh, wl);
-        const float decay = vec[48];
-#pragma unroll
-        for (int np = 0; np < DW; np++) {
-            uint32_t kb[4];
-            lt_ldmatrix_x4_trans(kb, st + L.y + b_trans + (uint32_t)np * 32u);
-#pragma unroll
-            for (int e = 0; e < 4; e++) S[2 * np][e] *= decay, S[2 * np + 1][e] *= decay;
-            lt_mma(S[2 * np], wh, kb[0], kb[1]);
-            lt_mma(S[2 * np + 1], wh, kb[2], kb[3]);
-            lt_mma(S[2 * np], wl, kb[0], kb[1]);
-            lt_mma(S[2 * np + 1], wl, kb[2], kb[3]);
-        }
-        // outputs: two warps of the group take eight tokens each
-        if (part < 2) {
+            auto split_tile = [&](const float (&m)[2][4], uint32_t (&hi)[4], uint32_t (&lo)[4]) {
+                lt_split(m[0][0], m[0][1], hi[0], lo[0]);
+                lt_split(m[0][2], m[0][3], hi[1], lo[1]);
+                lt_split(m[1][0], m[1][1], hi[2], lo[2]);
+                lt_split(m[1][2], m[1][3], hi[3], lo[3]);
+            };
+            uint32_t hi[4], lo[4];
+            split_tile(R, hi, lo);
+            float W[2][4], W2[2][4];
+            lt_mma_zero(W[0], hi, bh[0], bh[1]);
+            lt_mma_zero(W[1], hi, bh[2], bh[3]);
+            lt_mma_zero(W2[0], lo, bh[0], bh[1]);
+            lt_mma_zero(W2[1], lo, bh[2], bh[3]);
+            lt_mma(W2[0], hi, bl[0], bl[1]);
+            lt_mma(W2[1], hi, bl[2], bl[3]);
+            // meanwhile the first two warps' eight tokens of the output
             float o[4];
-            total(2 + part, o);
+            if (part < 2) {
+                const float4 y = total(2 + part);
+                const float2 f = *reinterpret_cast<const float2 *>(vec + 16 + part * 8 + 2 * tq);
+                o[0] = f.x * y.x, o[1] = f.y * y.y, o[2] = f.x * y.z, o[3] = f.y * y.w;
+                uint32_t q[4];
+                lt_ldmatrix_x4(q, st + b_out);
+                lt_mma(o, hi, q[0], q[1]);
+                lt_mma(o, lo, q[0], q[1]);
+                lt_mma(o, hi, q[2], q[3]);
+            }
 #pragma unroll
-            for (int e = 0; e < 4; e++) o[e] *= vec[16 + part * 8 + 2 * tq + (e & 1)];
-            split_tile(U, hi, lo);
-            lt_ldmatrix_x4(bh, st + L.mat + 2 * 16 * 48 + b_mat);
-            lt_ldmatrix_x4(bl, st + L.mat + 3 * 16 * 48 + b_mat);
-            const uint32_t h0 = part ? bh[2] : bh[0], h1 = part ? bh[3] : bh[1], l0 = part ? bl[2] : bl[0], l1 = part ? bl[3] : bl[1];
-            lt_mma(o, hi, h0, h1);
-            lt_mma(o, lo, h0, h1);
-            lt_mma(o, hi, l0, l1);
+            for (int n = 0; n < 2; n++)
 #pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const int t = 16 * it + part * 8 + 2 * tq + (e & 1), j = jw + g + 8 * (e >> 1);
-                if (t < a.tokens && j < vdim) a.o[((size_t)t * a.heads + h) * vdim + j] = o[e];
+                for (int e = 0; e < 4; e++) W[n][e] += W2[n][e];
+            split_tile(W, hi, lo);
+            const float decay = vec[32];
+#pragma unroll
+            for (int np = 0; np < DW; np++) {
+                uint32_t kb[4];
+                lt_ldmatrix_x4_trans(kb, st + L.y + b_trans + (uint32_t)np * 32u);
+#pragma unroll
+                for (int e = 0; e < 4; e++) S[2 * np][e] *= decay, S[2 * np + 1][e] *= decay;
+                lt_mma(S[2 * np], hi, kb[0], kb[1]);
+                lt_mma(S[2 * np + 1], hi, kb[2], kb[3]);
+                lt_mma(S[2 * np], lo, kb[0], kb[1]);
+                lt_mma(S[2 * np + 1], lo, kb[2], kb[3]);
+            }
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&empty[sl]);
+            if (part < 2) {
+                const int t = 16 * it + part * 8 + 2 * tq;
+                if (t < a.tokens) {
+                    if (col0) to[0] = o[0];
+                    if (col1) to[8] = o[2];
+                }
+                if (t + 1 < a.tokens) {
+                    if (col0) to[ldv] = o[1];
+                    if (col1) to[ldv + 8] = o[3];
+                }
             }
         }
+        if (!ok) atomicExch(&s_failed, 1);
+        state_io(true);
     }
-    state_io(true);
+    __syncthreads();
+    if (tid == 0 && s_failed && a.err) atomicExch(a.err, DEV_ERR_MBAR_TIMEOUT);
 }
 
 }  // namespace rnb

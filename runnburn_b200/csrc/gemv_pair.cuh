@@ -90,9 +90,6 @@ __device__ __forceinline__ void gp_q4k_block(const uint8_t *blk, const uint8_t *
     A.m[1] = __fmaf_rn(dmin, (float)mp1, A.m[1]);
 }
 
-__device__ __forceinline__ void mbar_arrive(uint64_t *bar) {
-    asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(bar)) : "memory");
-}
 
 // grid = tiles of 16 rows, 32 threads.  Operands must be 16-byte aligned (the host checks).
 // DYN: the expert-gathered instantiation (virtual rows, ids read after the wait on the previous kernel, tails 1 with

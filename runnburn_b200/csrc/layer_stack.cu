@@ -525,6 +525,21 @@ static int linear_chunk(int tokens, int ctas_per_chunk) {
 static bool linear_tiled(const rnb_b200_mixer_cfg &m) { return m.dim % 8 == 0 && m.vdim % 8 == 0 && m.dim <= 256; }
 static int linear_tile_warps(int vdim) { return std::min((vdim + 15) / 16, 8); }
 static bool delta_tiled(const rnb_b200_mixer_cfg &m) { return m.dim % 16 == 0 && m.vdim % 8 == 0 && m.dim <= 256; }
+// Tile kernel of the delta rule: channel blocks it is instantiated for, groups of 16 value columns per CTA (few, so that the heads
+// spread over the SMs), rows of the prepared tiles.
+struct DeltaTileShape {
+    int dt, cw, col_blocks, ld_qk, ld_val;
+};
+static DeltaTileShape delta_tile_shape(const rnb_b200_mixer_cfg &m) {
+    DeltaTileShape s;
+    const int cols = (m.vdim + 15) / 16;
+    s.dt = m.dim <= 32 ? 2 : m.dim <= 64 ? 4 : m.dim <= 128 ? 8 : 16;
+    s.cw = std::min(cols, 2);
+    s.col_blocks = (cols + s.cw - 1) / s.cw;
+    s.ld_qk = 16 * s.dt + 8;
+    s.ld_val = 16 * s.cw + 8;
+    return s;
+}
 // CTAs that work on one chunk of tokens
 static int linear_ctas(const rnb_b200_mixer_cfg &m) { const int w = 16 * linear_tile_warps(m.vdim); return m.heads * ((m.vdim + w - 1) / w); }
 
@@ -533,7 +548,7 @@ int LayerStack::alloc_scratch(StackScratch &b, int cap) {
     b = StackScratch();
     const bool small = cap <= SMALL;
     const size_t T = (size_t)cap, D = (size_t)cfg.width, es = narrow(cap) ? 2 : 4;
-    size_t proj[4] = {1, 1, 1, 1}, zw = 1, ww = 1, ow = 1, aw = 1, auxw[2] = {0, 0}, streams = 1, qfw = 0, partw = 0, st = 0, dc = 0, kn = 0, vx = 0, qn = 0, cq = 0, cv = 0, rec = 0, th = 0;
+    size_t proj[4] = {1, 1, 1, 1}, zw = 1, ww = 1, ow = 1, aw = 1, auxw[2] = {0, 0}, streams = 1, qfw = 0, partw = 0, st = 0, dc = 0, kn = 0, vx = 0, qn = 0, cqk = 0, cv = 0, rec = 0, th = 0;
     auto most = [](size_t &a, size_t b) { a = std::max(a, b); };
     for (const StackLayer &L : layers_) {
         if (!L.norm1) continue;   // uses another layer's weights: the same sizes
@@ -567,8 +582,9 @@ int LayerStack::alloc_scratch(StackScratch &b, int cap) {
                 if (m.mixer == RNB_B200_MIXER_WKV) streams = 5, most(zw, (size_t)M.w1.rows);
                 if (m.mixer == RNB_B200_MIXER_WKV || m.mixer == RNB_B200_MIXER_GLA) most(ww, hd), most(th, (size_t)M.w1.rows);
                 if (m.mixer == RNB_B200_MIXER_DELTA && !small && es == 2 && delta_tiled(m)) {
-                    most(cq, (size_t)m.kv_heads * m.dim);
-                    most(cv, hv);
+                    const DeltaTileShape ts = delta_tile_shape(m);
+                    most(cqk, (size_t)m.kv_heads * 32 * ts.ld_qk);
+                    most(cv, (size_t)m.heads * ts.col_blocks * 16 * ts.ld_val);
                     most(rec, (size_t)m.heads * DR_REC);
                 }
                 if (!small && linear) {
@@ -597,9 +613,8 @@ int LayerStack::alloc_scratch(StackScratch &b, int cap) {
     RNB_CU(cudaMemset(b.act, 0, T * aw * es));   // padding columns meet zero weights: they only have to be finite
     RNB_CU(cudaStreamSynchronize(nullptr));      // the decoder's stream does not wait for the default one
     RNB_TRY(get(&b.qn, T * qn * es));
-    RNB_TRY(get(&b.cq, T * cq * 2));
-    RNB_TRY(get(&b.ck, T * cq * 2));
-    RNB_TRY(get(&b.cv, T * cv * 2));
+    RNB_TRY(get(&b.cqk, (T + 15) / 16 * cqk * 2));
+    RNB_TRY(get(&b.cv, (T + 15) / 16 * cv * 2));
     RNB_TRY(get(&b.rec, (T + 15) / 16 * rec));
     RNB_TRY(get(&b.qf, T * qfw * 4));
     RNB_TRY(get(&b.part, T * partw * 4));
@@ -643,7 +658,8 @@ int LayerStack::ready(cudaStream_t s) {
                          (const void *)linear_state_step_kernel<32>, (const void *)linear_state_step_kernel<64>, (const void *)causal_attention_kernel<4>,
                          (const void *)causal_attention_kernel<8>, (const void *)causal_attention_kernel<16>, (const void *)causal_attention_kernel<32>,
                          (const void *)attention_step_kernel<float, float>, (const void *)attention_step_kernel<float, bf16>, (const void *)attention_step_kernel<bf16, bf16>,
-                         (const void *)delta_prepare_kernel, (const void *)delta_tile_kernel<2>, (const void *)delta_tile_kernel<4>, (const void *)delta_tile_kernel<8>,
+                         (const void *)delta_prepare_kernel<0>, (const void *)delta_prepare_kernel<2>,
+                         (const void *)delta_prepare_kernel<3>, (const void *)delta_prepare_kernel<4>, (const void *)delta_tile_kernel<2>, (const void *)delta_tile_kernel<4>, (const void *)delta_tile_kernel<8>,
                          (const void *)delta_tile_kernel<16>};
     const void *pairs[] = {
 #define RNB_AD(TI) (const void *)attention_delta_step_kernel<float, TI>, (const void *)attention_delta_step_kernel<bf16, TI>
@@ -1067,27 +1083,35 @@ DeltaArgs LayerStack::delta_args(int n, StackScratch &b, StackLayer &L, int i, M
     a.p = b.p[i], a.ba = b.aux[i], a.conv = M.conv, a.a_log = M.a_log, a.dt = M.dt, a.norm = M.head_norm;
     a.ring = R.conv_ring, a.state = R.state, a.o = b.o, a.counters = counters_ + i * counters_of_mixer_, a.pos0 = pos_dev;
     if (n <= SMALL) a.act = (float *)act_of(b, M, n);
-    a.cq = reinterpret_cast<bf16 *>(b.cq), a.ck = reinterpret_cast<bf16 *>(b.ck), a.cv = reinterpret_cast<bf16 *>(b.cv), a.rec = b.rec;
+    const DeltaTileShape ts = delta_tile_shape(m);
+    a.cqk = reinterpret_cast<bf16 *>(b.cqk), a.cv = reinterpret_cast<bf16 *>(b.cv), a.rec = b.rec;
+    a.ld_qk = ts.ld_qk, a.ld_val = ts.ld_val, a.col_blocks = ts.col_blocks, a.cw = ts.cw;
     a.eps = cfg.norm_eps, a.out_mul = m.out_scale, a.q_mul = 1.0f / sqrtf((float)m.dim);
     a.tokens = n, a.heads = m.heads, a.kv_heads = m.kv_heads, a.dim = m.dim, a.vdim = m.vdim, a.taps = m.conv;
     a.k_at = M.in_at[1], a.v_at = M.in_at[2], a.g_at = M.in_at[3], a.a_at = m.heads, a.ld = M.in_rows, a.ld_ba = M.aux_rows, a.lda = L.out_cols;
     return a;
 }
 
-int LayerStack::mixer_delta(cudaStream_t s, int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev) {
+int LayerStack::mixer_delta(cudaStream_t s, int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev, int *err) {
     const StackMixer &M = L.mixers[i];
     const rnb_b200_mixer_cfg &m = M.c;
     const bool nb = narrow(n);
-    const DeltaArgs a = delta_args(n, b, L, i, R, pos_dev);
+    DeltaArgs a = delta_args(n, b, L, i, R, pos_dev);
+    a.err = err;
     if (nb && delta_tiled(m)) {
-        RNB_CU(launch_k(delta_prepare_kernel, dim3((unsigned)((n + DP_TOKENS - 1) / DP_TOKENS), (unsigned)m.kv_heads), dim3(256), delta_prepare_smem(m.dim), s, a));
-        const int cols = (m.vdim + 15) / 16, cw = std::min(cols, 2);   // few columns per CTA, so that the heads spread over the SMs
-        const dim3 grid((unsigned)m.heads, (unsigned)((cols + cw - 1) / cw));
-        auto block = [&](int dt) { return dim3((unsigned)(32 * delta_tile_split(dt) * cw)); };
-        if (m.dim <= 32) RNB_CU(launch_k(delta_tile_kernel<2>, grid, block(2), delta_tile_smem(2, cw).bytes, s, a));
-        else if (m.dim <= 64) RNB_CU(launch_k(delta_tile_kernel<4>, grid, block(4), delta_tile_smem(4, cw).bytes, s, a));
-        else if (m.dim <= 128) RNB_CU(launch_k(delta_tile_kernel<8>, grid, block(8), delta_tile_smem(8, cw).bytes, s, a));
-        else RNB_CU(launch_k(delta_tile_kernel<16>, grid, block(16), delta_tile_smem(16, cw).bytes, s, a));
+        const dim3 pg((unsigned)((n + DP_TOKENS - 1) / DP_TOKENS), (unsigned)m.kv_heads);
+        const size_t psmem = delta_prepare_smem(m.dim);
+        if (m.conv == 2) RNB_CU(launch_k(delta_prepare_kernel<2>, pg, dim3(256), psmem, s, a));
+        else if (m.conv == 3) RNB_CU(launch_k(delta_prepare_kernel<3>, pg, dim3(256), psmem, s, a));
+        else if (m.conv == 4) RNB_CU(launch_k(delta_prepare_kernel<4>, pg, dim3(256), psmem, s, a));
+        else RNB_CU(launch_k(delta_prepare_kernel<0>, pg, dim3(256), psmem, s, a));
+        const dim3 grid((unsigned)m.heads, (unsigned)a.col_blocks), block((unsigned)(32 * (DT_SPLIT * a.cw + 1)));
+        const int dt = delta_tile_shape(m).dt;
+        const size_t smem = delta_tile_smem(dt, a.cw).bytes;
+        if (dt == 2) RNB_CU(launch_k(delta_tile_kernel<2>, grid, block, smem, s, a));
+        else if (dt == 4) RNB_CU(launch_k(delta_tile_kernel<4>, grid, block, smem, s, a));
+        else if (dt == 8) RNB_CU(launch_k(delta_tile_kernel<8>, grid, block, smem, s, a));
+        else RNB_CU(launch_k(delta_tile_kernel<16>, grid, block, smem, s, a));
     } else {
         const dim3 grid((unsigned)m.heads, (unsigned)((m.vdim + 31) / 32)), block(256);
         const size_t smem = delta_step_smem(m.dim);
@@ -1224,7 +1248,7 @@ int LayerStack::run_mixer(cudaStream_t s, int n, StackScratch &b, StackLayer &L,
     switch (L.mixers[i].c.mixer) {
     case RNB_B200_MIXER_LATENT_ATTENTION: return mixer_latent(s, n, b, L, i, R, pos_dev, pos_host, err);
     case RNB_B200_MIXER_ATTENTION: return mixer_attention(s, n, b, L, i, R, pos_dev);
-    case RNB_B200_MIXER_DELTA: return mixer_delta(s, n, b, L, i, R, pos_dev);
+    case RNB_B200_MIXER_DELTA: return mixer_delta(s, n, b, L, i, R, pos_dev, err);
     default: return mixer_linear(s, n, b, L, i, R, pos_dev, err);
     }
 }

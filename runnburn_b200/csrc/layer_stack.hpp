@@ -62,7 +62,7 @@ struct StackScratch {
     uint16_t *th = nullptr;   // tanh of the low-rank decay input as bf16 hi + lo
     void *h = nullptr, *p[4] = {nullptr, nullptr, nullptr, nullptr}, *act = nullptr, *qn = nullptr;
     float *aux[2] = {nullptr, nullptr};
-    uint16_t *kn = nullptr, *vx = nullptr, *cq = nullptr, *ck = nullptr, *cv = nullptr;
+    uint16_t *kn = nullptr, *vx = nullptr, *cqk = nullptr, *cv = nullptr;
     uint8_t *rec = nullptr;
     int *rows = nullptr;
     uint32_t *tok = nullptr;
@@ -135,7 +135,7 @@ private:
     WindowAttentionArgs attention_args(int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev) const;
     DeltaArgs delta_args(int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev) const;
     int mixers_attention_delta(cudaStream_t s, int n, StackScratch &b, StackLayer &L, LayerRun &R, const int *pos_dev);
-    int mixer_delta(cudaStream_t s, int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev);
+    int mixer_delta(cudaStream_t s, int n, StackScratch &b, StackLayer &L, int i, MixerState &R, const int *pos_dev, int *err);
     int head_norm_gate(cudaStream_t s, int n, StackScratch &b, const StackLayer &L, const StackMixer &M, const void *g, int ldg);
     void *act_of(StackScratch &b, const StackMixer &M, int n) const { return (char *)b.act + (size_t)M.act_at * (narrow(n) ? 2 : 4); }
     int attention_ring(const rnb_b200_mixer_cfg &m) const;

@@ -16,6 +16,12 @@ __device__ __forceinline__ void lt_mma(float (&c)[4], const uint32_t (&a)[4], ui
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
+// c = a b
+__device__ __forceinline__ void lt_mma_zero(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%10,%10,%10,%10};"
+                 : "=f"(c[0]), "=f"(c[1]), "=f"(c[2]), "=f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1), "f"(0.f));
+}
 __device__ __forceinline__ void lt_split(float x, float y, uint32_t &hi, uint32_t &lo) {
     hi = pg_pack_bf16(x, y);
     lo = pg_pack_bf16(x - bf16_lo(hi), y - bf16_hi(hi));

@@ -143,7 +143,7 @@ __host__ __device__ inline AttentionStepSmem<CT> attention_step_smem(int rep, in
     L.s = L.q + (uint32_t)(((size_t)rep * dim * 4 + 15) & ~(size_t)15);
     L.acc = L.s + (uint32_t)(rep * AS_KEYS * 4);
     L.stat = L.acc + (uint32_t)(((size_t)rep * vdim * 4 + 15) & ~(size_t)15);
-    L.bytes = L.stat + (uint32_t)(3 * rep * 4);
+    L.bytes = L.stat + (uint32_t)(4 * rep * 4);
     return L;
 }
 // keys per chunk when n of them are split over at most `chunks` CTAs
@@ -156,7 +156,7 @@ __device__ __forceinline__ void attention_step_block(const WindowAttentionArgs &
     const AttentionStepSmem<CT> L = attention_step_smem<CT>(rep, dim, vdim);
     CT *sk = reinterpret_cast<CT *>(as_smem + L.k), *sv = reinterpret_cast<CT *>(as_smem + L.v);
     float *sq = reinterpret_cast<float *>(as_smem + L.q), *ss = reinterpret_cast<float *>(as_smem + L.s), *acc = reinterpret_cast<float *>(as_smem + L.acc);
-    float *s_m = reinterpret_cast<float *>(as_smem + L.stat), *s_l = s_m + rep, *s_c = s_l + rep;
+    float *s_m = reinterpret_cast<float *>(as_smem + L.stat), *s_l = s_m + rep, *s_c = s_l + rep, *s_g = s_c + rep;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     constexpr int E = 16 / (int)sizeof(CT);
     const bool vec = dim % E == 0 && vdim % E == 0;
@@ -217,7 +217,10 @@ __device__ __forceinline__ void attention_step_block(const WindowAttentionArgs &
     for (int j = warp; j < rep; j += AS_THREADS / 32) {
         const int h = g * rep + j;
         rotated_normed_row(reinterpret_cast<const AT *>(a.q) + (size_t)t * a.ld + (size_t)h * dim, a.rot, pos, dim, a.qk_norm, a.eps, [&](int e, float v) { sq[j * dim + e] = v; });
-        if (lane == 0) s_m[j] = -INFINITY, s_l[j] = 0.f;
+        if (lane == 0) {
+            s_m[j] = -INFINITY, s_l[j] = 0.f;
+            s_g[j] = a.gate ? a.out_mul / (1.0f + expf(-a.gate[(size_t)t * a.ldg + h])) : a.out_mul;
+        }
     }
     for (int i = tid; i < rep * vdim; i += AS_THREADS) acc[i] = 0.f;
     for (int base = lo; base < hi; base += AS_KEYS) {
@@ -304,11 +307,10 @@ __device__ __forceinline__ void attention_step_block(const WindowAttentionArgs &
         if (base + AS_KEYS < hi) load(base + AS_KEYS);
     }
     AT *act = reinterpret_cast<AT *>(a.act) + (size_t)t * a.lda;
-    auto gate_of = [&](int h) { return a.gate ? a.out_mul / (1.0f + expf(-a.gate[(size_t)t * a.ldg + h])) : a.out_mul; };
     if (active == 1) {
         for (int i = tid; i < rep * vdim; i += AS_THREADS) {
             const int j = i / vdim, h = g * rep + j;
-            act[(size_t)h * vdim + i % vdim] = from_f32<AT>(acc[i] / s_l[j] * gate_of(h));
+            act[(size_t)h * vdim + i % vdim] = from_f32<AT>(acc[i] / s_l[j] * s_g[j]);
         }
         return;
     }
@@ -335,7 +337,7 @@ __device__ __forceinline__ void attention_step_block(const WindowAttentionArgs &
             l = fmaf(w, lc[i], l);
         }
         l = warp_sum(l);
-        if (lane == 0) s_l[j] = gate_of(g * rep + j) / l;
+        if (lane == 0) s_l[j] = s_g[j] / l;
     }
     __syncthreads();
     for (int i = tid; i < rep * vdim; i += AS_THREADS) {
