@@ -216,16 +216,16 @@ template <int TAPS, class Put>
 __device__ __forceinline__ void delta_convolve16(const DeltaArgs &a, int c, int col, int t, int end, int pos0, Put put) {
     const int taps = TAPS ? TAPS : a.taps, C = delta_channels(a);
     const bf16 *p = reinterpret_cast<const bf16 *>(a.p) + col;
+    auto load = [&](int at) { return *reinterpret_cast<const uint4 *>(p + (size_t)min(at, a.tokens - 1) * a.ld); };
+    auto unpack = [&](uint4 b, float (&v)[8]) {
+        const uint32_t r[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+        for (int e = 0; e < 4; e++) v[2 * e] = bf16_lo(r[e]), v[2 * e + 1] = bf16_hi(r[e]);
+    };
     auto row = [&](int at, float (&v)[8]) {
-        if (at >= 0) {
-            const uint4 b = *reinterpret_cast<const uint4 *>(p + (size_t)min(at, a.tokens - 1) * a.ld);
-            const uint32_t r[4] = {b.x, b.y, b.z, b.w};
-#pragma unroll
-            for (int e = 0; e < 4; e++) v[2 * e] = bf16_lo(r[e]), v[2 * e + 1] = bf16_hi(r[e]);
-        } else {
-#pragma unroll
+        if (at >= 0) unpack(load(at), v);
+        else
             for (int e = 0; e < 8; e++) v[e] = delta_input<bf16>(a, c + e, col + e, at, pos0);
-        }
     };
     auto weights = [&](int n, float (&w)[8]) {
         const float4 x = *reinterpret_cast<const float4 *>(a.conv + (size_t)n * C + c), y = *reinterpret_cast<const float4 *>(a.conv + (size_t)n * C + c + 4);
@@ -240,21 +240,35 @@ __device__ __forceinline__ void delta_convolve16(const DeltaArgs &a, int c, int 
         put(i, make_uint4(r[0], r[1], r[2], r[3]));
     };
     if (TAPS) {
+        // groups of N tokens: their rows are asked for a group ahead, and the last rows form a ring whose places are known
         constexpr int N = TAPS ? TAPS : 1;
-        float w[N][8], x[N][8];   // x: a ring of the last rows
+        float w[N][8], x[N][8];
+        uint4 next[N];
+#pragma unroll
+        for (int n = 0; n < N; n++) next[n] = load(t + n);
 #pragma unroll
         for (int n = 0; n < N; n++) weights(n, w[n]);
 #pragma unroll
         for (int n = 0; n < N - 1; n++) row(t - (N - 1) + n, x[n]);
+#pragma unroll 1
+        for (int i0 = 0; i0 < 16; i0 += N) {
+            uint4 now[N];
 #pragma unroll
-        for (int i = 0; i < 16; i++) {
-            row(t + i, x[(i + N - 1) % N]);
-            float y[8] = {};
+            for (int n = 0; n < N; n++) now[n] = next[n];
+            if (i0 + N < 16)
 #pragma unroll
-            for (int n = 0; n < N; n++)
+                for (int n = 0; n < N; n++) next[n] = load(t + i0 + N + n);
 #pragma unroll
-                for (int e = 0; e < 8; e++) y[e] = fmaf(w[n][e], x[(i + n) % N][e], y[e]);
-            finish(i, y);
+            for (int i = 0; i < N; i++) {
+                if (i0 + i >= 16) break;
+                unpack(now[i], x[(i + N - 1) % N]);
+                float y[8] = {};
+#pragma unroll
+                for (int n = 0; n < N; n++)
+#pragma unroll
+                    for (int e = 0; e < 8; e++) y[e] = fmaf(w[n][e], x[(i + n) % N][e], y[e]);
+                finish(i0 + i, y);
+            }
         }
     } else {
         for (int i = 0; i < 16; i++) {
