@@ -1035,6 +1035,7 @@ WindowAttentionArgs LayerStack::attention_args(int n, StackScratch &b, StackLaye
     a.eps = cfg.norm_eps, a.scale = m.scale, a.out_mul = m.out_scale;
     a.tokens = n, a.heads = m.heads, a.kv_heads = m.kv_heads, a.dim = m.dim, a.vdim = m.vdim, a.ld = M.in_rows, a.lda = L.out_cols;
     a.ring = attention_ring(m), a.window = m.window, a.qk_norm = m.qk_norm;
+    a.fours = m.dim % 4 == 0 && m.rot.dims % 4 == 0 && (m.rot.interleaved || !a.rot.table);
     return a;
 }
 
@@ -1050,15 +1051,12 @@ int LayerStack::mixer_attention(cudaStream_t s, int n, StackScratch &b, StackLay
         return RNB_B200_OK;
     }
     const dim3 pg((unsigned)n, (unsigned)((m.heads + 2 * m.kv_heads + 7) / 8)), one(1, (unsigned)m.kv_heads, (unsigned)n);
-    const bool fours = m.dim <= 512 && m.dim % 4 == 0 && a.rot.dims % 4 == 0 && (a.rot.interleaved || !a.rot.table);
     if (!nb) {
-        if (fours) RNB_CU(launch_k(attention_prepare_kernel<float, float, true>, pg, dim3(256), 0, s, a));
-        else RNB_CU(launch_k(attention_prepare_kernel<float, float, false>, pg, dim3(256), 0, s, a));
+        RNB_CU(launch_k(attention_prepare_kernel<float, float>, pg, dim3(256), 0, s, a));
         RNB_CU(launch_k(attention_step_kernel<float, float>, one, dim3(AS_THREADS), smem, s, a));
         return RNB_B200_OK;
     }
-    if (fours) RNB_CU(launch_k(attention_prepare_kernel<bf16, bf16, true>, pg, dim3(256), 0, s, a));
-    else RNB_CU(launch_k(attention_prepare_kernel<bf16, bf16, false>, pg, dim3(256), 0, s, a));
+    RNB_CU(launch_k(attention_prepare_kernel<bf16, bf16>, pg, dim3(256), 0, s, a));
     if (!attention_tiled(m)) {
         RNB_CU(launch_k(attention_step_kernel<bf16, bf16>, one, dim3(AS_THREADS), smem, s, a));
         return RNB_B200_OK;

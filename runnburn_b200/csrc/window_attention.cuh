@@ -26,7 +26,7 @@ struct WindowAttentionArgs {
     const int *pos0;
     Rotation rot;
     float eps, scale, out_mul;
-    int tokens, heads, kv_heads, dim, vdim, ld, ldg, lda, ring, window, qk_norm, fresh;
+    int tokens, heads, kv_heads, dim, vdim, ld, ldg, lda, ring, window, qk_norm, fresh, fours;   // fours: rotated_normed_fours applies
 };
 
 // One warp: store(e, value) for every element of the rotated (and normed) vector x.
@@ -57,44 +57,57 @@ __device__ __forceinline__ void rotated_normed_row(const AT *x, const Rotation &
     }
 }
 
-// The same for vectors whose rotated pairs (2i, 2i + 1) and accesses of four elements do not straddle anything
-// (dim <= 512, dim and rotated dims multiples of 4, rows aligned): four elements per lane and access.
+// The same for vectors whose rotated pairs (2i, 2i + 1) and accesses of four elements do not straddle anything (dim and
+// rotated dims multiples of 4, rows aligned): put(e, four values) for every fourth element.
 template <class AT>
 struct alignas(4 * sizeof(AT)) Four { AT v[4]; };
-template <class AT, class CT>
-__device__ __forceinline__ void rotated_normed_fours(const AT *x, const Rotation &rot, int pos, int dim, bool norm, float eps, CT *out) {
-    const int lane = threadIdx.x & 31;
-    float v[4][4], ss = 0.f;
+template <class CT>
+__device__ __forceinline__ void store_four(CT *p, const float (&v)[4]) {
+    Four<CT> o;
 #pragma unroll
-    for (int i = 0; i < 4; i++) {
-        const int e = 4 * (lane + 32 * i);
-        if (e >= dim) continue;
+    for (int q = 0; q < 4; q++) o.v[q] = from_f32<CT>(v[q]);
+    *reinterpret_cast<Four<CT> *>(p) = o;
+}
+template <class AT, class Put>
+__device__ __forceinline__ void rotated_normed_fours(const AT *x, const Rotation &rot, int pos, int dim, bool norm, float eps, Put put) {
+    const float2 *table = rot.table + (size_t)pos * (rot.dims / 2);
+    auto four = [&](int e, float (&v)[4]) {
         const Four<AT> a = *reinterpret_cast<const Four<AT> *>(x + e);
+        float u[4];
 #pragma unroll
-        for (int q = 0; q < 4; q++) v[i][q] = to_f32(a.v[q]);
+        for (int q = 0; q < 4; q++) u[q] = v[q] = to_f32(a.v[q]);
         if (rot.table && e < rot.dims) {
-            const float4 cs = *reinterpret_cast<const float4 *>(rot.table + (size_t)pos * (rot.dims / 2) + e / 2);
-            const float a0 = v[i][0], a1 = v[i][1], a2 = v[i][2], a3 = v[i][3];
-            v[i][0] = fmaf(a0, cs.x, -(a1 * cs.y)), v[i][1] = fmaf(a1, cs.x, a0 * cs.y);
-            v[i][2] = fmaf(a2, cs.z, -(a3 * cs.w)), v[i][3] = fmaf(a3, cs.z, a2 * cs.w);
+            const float4 cs = *reinterpret_cast<const float4 *>(table + e / 2);
+            v[0] = fmaf(u[0], cs.x, -(u[1] * cs.y)), v[1] = fmaf(u[1], cs.x, u[0] * cs.y);
+            v[2] = fmaf(u[2], cs.z, -(u[3] * cs.w)), v[3] = fmaf(u[3], cs.z, u[2] * cs.w);
         }
-#pragma unroll
-        for (int q = 0; q < 4; q++) ss = fmaf(v[i][q], v[i][q], ss);
+    };
+    auto squares = [](const float (&v)[4]) { return fmaf(v[0], v[0], v[1] * v[1]) + fmaf(v[2], v[2], v[3] * v[3]); };
+    const int first = 4 * (threadIdx.x & 31);
+    float v[4] = {}, w[4];   // the first 128 elements stay in registers
+    if (first < dim) four(first, v);
+    float ss = squares(v);
+#pragma unroll 1
+    for (int e = first + 128; e < dim; e += 128) {
+        four(e, w);
+        ss += squares(w);
     }
     const float r = norm ? 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps) : 1.0f;
+    auto scaled = [&](int e, float (&v)[4]) {
 #pragma unroll
-    for (int i = 0; i < 4; i++) {
-        const int e = 4 * (lane + 32 * i);
-        if (e >= dim) continue;
-        Four<CT> o;
-#pragma unroll
-        for (int q = 0; q < 4; q++) o.v[q] = from_f32<CT>(v[i][q] * r);
-        *reinterpret_cast<Four<CT> *>(out + e) = o;
+        for (int q = 0; q < 4; q++) v[q] *= r;
+        put(e, v);
+    };
+    if (first < dim) scaled(first, v);
+#pragma unroll 1
+    for (int e = first + 128; e < dim; e += 128) {
+        four(e, w);
+        scaled(e, w);
     }
 }
 
-// grid = (tokens, ceil((heads + 2 kv_heads) / 8)), 256 threads: a warp per query, key or value vector.  FOURS: the form above.
-template <class AT, class CT, bool FOURS>
+// grid = (tokens, ceil((heads + 2 kv_heads) / 8)), 256 threads: a warp per query, key or value vector
+template <class AT, class CT>
 RNB_GLOBAL void __launch_bounds__(256)
 attention_prepare_kernel(const __grid_constant__ WindowAttentionArgs a) {
     pdl_launch_dependents();
@@ -104,7 +117,7 @@ attention_prepare_kernel(const __grid_constant__ WindowAttentionArgs a) {
     const size_t row = (size_t)t * a.ld, slot = (size_t)(pos % a.ring);
     auto finish = [&](const AT *x, auto *out) {
         typedef typename std::remove_pointer<decltype(out)>::type OT;
-        if (FOURS) rotated_normed_fours<AT, OT>(x, a.rot, pos, a.dim, a.qk_norm, a.eps, out);
+        if (a.fours) rotated_normed_fours(x, a.rot, pos, a.dim, a.qk_norm, a.eps, [&](int e, const float (&v)[4]) { store_four(out + e, v); });
         else rotated_normed_row(x, a.rot, pos, a.dim, a.qk_norm, a.eps, [&](int e, float v) { out[e] = from_f32<OT>(v); });
     };
     if (unit < a.heads) {
@@ -116,7 +129,7 @@ attention_prepare_kernel(const __grid_constant__ WindowAttentionArgs a) {
         const int g = unit - a.heads - a.kv_heads;
         const AT *src = reinterpret_cast<const AT *>(a.v) + row + (size_t)g * a.vdim;
         CT *out = reinterpret_cast<CT *>(a.vc) + (slot * a.kv_heads + g) * a.vdim;
-        if (FOURS && sizeof(AT) == sizeof(CT) && a.vdim % 4 == 0) {
+        if (a.fours && sizeof(AT) == sizeof(CT) && a.vdim % 4 == 0) {
             for (int e = 4 * lane; e < a.vdim; e += 128) *reinterpret_cast<Four<CT> *>(out + e) = *reinterpret_cast<const Four<CT> *>(src + e);
         } else {
             for (int e = lane; e < a.vdim; e += 32) out[e] = from_f32<CT>(to_f32(src[e]));
@@ -200,11 +213,18 @@ __device__ __forceinline__ void attention_step_block(const WindowAttentionArgs &
             const bool append = key == pos;   // one CTA per key/value head and token
             const size_t row = (size_t)(key - pos0) * a.ld, slot = (size_t)(key % a.ring);
             CT *ko = reinterpret_cast<CT *>(a.kc) + slot * ldk + (size_t)g * dim, *vo = reinterpret_cast<CT *>(a.vc) + slot * ldv + (size_t)g * vdim;
-            rotated_normed_row(reinterpret_cast<const AT *>(a.k) + row + (size_t)g * dim, a.rot, key, dim, a.qk_norm, a.eps, [&](int e, float v) {
-                const CT x = from_f32<CT>(v);
-                sk[r * L.kp + e] = x;
-                if (append) ko[e] = x;
-            });
+            const AT *kx = reinterpret_cast<const AT *>(a.k) + row + (size_t)g * dim;
+            if (a.fours)
+                rotated_normed_fours(kx, a.rot, key, dim, a.qk_norm, a.eps, [&](int e, const float (&v)[4]) {
+                    store_four(sk + r * L.kp + e, v);
+                    if (append) store_four(ko + e, v);
+                });
+            else
+                rotated_normed_row(kx, a.rot, key, dim, a.qk_norm, a.eps, [&](int e, float v) {
+                    const CT x = from_f32<CT>(v);
+                    sk[r * L.kp + e] = x;
+                    if (append) ko[e] = x;
+                });
             const AT *src = reinterpret_cast<const AT *>(a.v) + row + (size_t)g * vdim;
             for (int e = lane; e < vdim; e += 32) {
                 const CT x = from_f32<CT>(to_f32(src[e]));
@@ -216,7 +236,9 @@ __device__ __forceinline__ void attention_step_block(const WindowAttentionArgs &
     load(lo);
     for (int j = warp; j < rep; j += AS_THREADS / 32) {
         const int h = g * rep + j;
-        rotated_normed_row(reinterpret_cast<const AT *>(a.q) + (size_t)t * a.ld + (size_t)h * dim, a.rot, pos, dim, a.qk_norm, a.eps, [&](int e, float v) { sq[j * dim + e] = v; });
+        const AT *qx = reinterpret_cast<const AT *>(a.q) + (size_t)t * a.ld + (size_t)h * dim;
+        if (a.fours) rotated_normed_fours(qx, a.rot, pos, dim, a.qk_norm, a.eps, [&](int e, const float (&v)[4]) { store_four(sq + j * dim + e, v); });
+        else rotated_normed_row(qx, a.rot, pos, dim, a.qk_norm, a.eps, [&](int e, float v) { sq[j * dim + e] = v; });
         if (lane == 0) {
             s_m[j] = -INFINITY, s_l[j] = 0.f;
             s_g[j] = a.gate ? a.out_mul / (1.0f + expf(-a.gate[(size_t)t * a.ldg + h])) : a.out_mul;

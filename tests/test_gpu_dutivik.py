@@ -71,6 +71,19 @@ SHARED = MIXED + [su.again(MIXED[0], 0), su.again(MIXED[3], 3), su.again(MIXED[2
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("rank", [1, 7, 32, 136])
+def test_low_rank_decay_of_any_width(rank, dtype):
+    cfg = su.dutivik([su.gla(heads=3, dim=24, vdim=16), su.gla(heads=1, dim=96, vdim=8, tau=2.0)], width=64)
+    w = su.weights(cfg, 23, rank=rank)
+    toks = su.tokens(cfg, 70)
+    want = ref.Model(cfg, w).forward(toks)
+    dec = su.decoder(cfg, w, dtype)
+    for cuts in ([70], [30] + [1] * 40):
+        assert not su.bad(su.feed(dec, toks, cuts), want, dtype)
+    dec.close()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("layers", [MIXED, SHARED], ids=["own", "shared"])
 def test_stack(dtype, layers):
     cfg = su.dutivik(layers, eps=1e-3, scale=1.0)
