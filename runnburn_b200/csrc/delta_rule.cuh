@@ -109,7 +109,7 @@ __device__ __forceinline__ void delta_step_block(const DeltaArgs &a, int h, int 
         const int ch = warp + 8 * q;
         S[q] = live && ch < dim ? sp[(size_t)ch * vdim] : 0.f;
     }
-    const int pos0 = *a.pos0;
+    const int pos0 = *a.pos0, R = delta_ring_rows(a.taps), slot0 = (pos0 + R - (a.taps - 1)) % R;   // where position pos0 - (taps - 1) lies
     const float decay = -expf(a.a_log[h]), dt = a.dt[h];
     for (int t0 = 0; t0 < a.tokens; t0 += DR_BLOCK) {
         const int T = min(DR_BLOCK, a.tokens - t0);
@@ -120,9 +120,19 @@ __device__ __forceinline__ void delta_step_block(const DeltaArgs &a, int h, int 
             const int c = x < dim ? hk * dim + x : x < 2 * dim ? qc + hk * dim + x - dim : 2 * qc + h * vdim + j0 + x - 2 * dim;
             float y = 0.f;
             if (x < 2 * dim || j0 + x - 2 * dim < vdim) {
-                const int col = delta_col(a, c);
+                const AT *in = reinterpret_cast<const AT *>(a.p) + delta_col(a, c);
+                const int before = max(0, a.taps - 1 - (t0 + t));   // taps that reach back past this call
+                int slot = slot0 + t0 + t;
+                if (slot >= R) slot -= R;
 #pragma unroll 4
-                for (int n = 0; n < a.taps; n++) y = fmaf(a.conv[(size_t)n * C + c], delta_input<AT>(a, c, col, t0 + t - (a.taps - 1) + n, pos0), y);
+                for (int n = 0; n < a.taps; n++) {
+                    const float w = a.conv[(size_t)n * C + c];
+                    float v;
+                    if (n >= before) v = to_f32(in[(size_t)(t0 + t - (a.taps - 1) + n) * a.ld]);
+                    else v = pos0 + t0 + t - (a.taps - 1) + n >= 0 ? a.ring[(size_t)slot * C + c] : 0.f;
+                    if (++slot == R) slot = 0;
+                    y = fmaf(w, v, y);
+                }
                 y = silu_f32(y);
             }
             if (x < dim) sq[t * dim + x] = y;

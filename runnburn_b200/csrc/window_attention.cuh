@@ -137,12 +137,14 @@ attention_prepare_kernel(const __grid_constant__ WindowAttentionArgs a) {
     }
 }
 
-// A step CTA: 64 keys at a time of one key/value head, for the rep query heads that share it.
-constexpr int AS_KEYS = 64, AS_THREADS = 256;
+// A step CTA: 64 keys at a time of one key/value head, for the rep query heads that share it.  bf16 rings with dim % 32 ==
+// 0 and vdim % 16 == 0: the products run on tensor cores, the query heads as the 16 rows (queries and weights enter as bf16
+// hi + lo parts); else on the CUDA cores.
+constexpr int AS_KEYS = 64, AS_THREADS = 256, AS_PE = AS_KEYS + 8;
 template <class CT>
 struct AttentionStepSmem {
-    int kp, vp;                                // elements per staged key / value row
-    uint32_t k, v, q, s, acc, stat, bytes;
+    int kp, vp, rows;                          // elements per staged key / value row; query rows of the products (0: no tensor cores)
+    uint32_t k, v, q, s, acc, stat, qh, ph, bytes;   // qh, ph: hi parts, the lo parts behind them
 };
 template <class CT>
 __host__ __device__ inline AttentionStepSmem<CT> attention_step_smem(int rep, int dim, int vdim) {
@@ -156,7 +158,10 @@ __host__ __device__ inline AttentionStepSmem<CT> attention_step_smem(int rep, in
     L.s = L.q + (uint32_t)(((size_t)rep * dim * 4 + 15) & ~(size_t)15);
     L.acc = L.s + (uint32_t)(rep * AS_KEYS * 4);
     L.stat = L.acc + (uint32_t)(((size_t)rep * vdim * 4 + 15) & ~(size_t)15);
-    L.bytes = L.stat + (uint32_t)(4 * rep * 4);
+    L.rows = sizeof(CT) == 2 && dim % 32 == 0 && vdim % 16 == 0 ? (rep + 15) & ~15 : 0;
+    L.qh = (L.stat + (uint32_t)(4 * rep * 4) + 15) & ~15u;
+    L.ph = L.qh + (uint32_t)(2 * L.rows * L.kp * 2);
+    L.bytes = L.ph + (uint32_t)(2 * L.rows * AS_PE * 2);
     return L;
 }
 // keys per chunk when n of them are split over at most `chunks` CTAs
@@ -245,10 +250,46 @@ __device__ __forceinline__ void attention_step_block(const WindowAttentionArgs &
         }
     }
     for (int i = tid; i < rep * vdim; i += AS_THREADS) acc[i] = 0.f;
+    bf16 *qhi = reinterpret_cast<bf16 *>(as_smem + L.qh), *qlo = qhi + L.rows * L.kp, *phi = reinterpret_cast<bf16 *>(as_smem + L.ph), *plo = phi + L.rows * AS_PE;
+    if (L.rows) {
+        __syncthreads();
+        for (int i = tid; i < L.rows * dim; i += AS_THREADS) {
+            const int j = i / dim, e = i % dim;
+            lt_split_store(qhi + j * L.kp + e, qlo + j * L.kp + e, j < rep ? sq[i] : 0.f);
+        }
+        for (int i = tid; i < (L.rows - rep) * AS_PE; i += AS_THREADS) phi[rep * AS_PE + i] = plo[rep * AS_PE + i] = from_f32<bf16>(0.f);
+    }
+    const int fg = lane >> 2, tq = lane & 3, mi = lane >> 3, mr = lane & 7;
+    const uint32_t a_row = (uint32_t)((mi & 1) * 8 + mr), a_col = (uint32_t)(mi >> 1) * 16u;
     for (int base = lo; base < hi; base += AS_KEYS) {
         const int nk = min(AS_KEYS, hi - base);
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
+        if (L.rows) {   // keys 8 warp .. + 7
+            const uint32_t kb = smem_u32(sk) + (uint32_t)((warp * 8 + mr) * L.kp) * 2u + (uint32_t)mi * 16u;
+            for (int j0 = 0; j0 < L.rows; j0 += 16) {
+                const uint32_t qa = smem_u32(qhi) + ((uint32_t)j0 + a_row) * (uint32_t)L.kp * 2u + a_col, ql = qa + (uint32_t)(L.rows * L.kp) * 2u;
+                float c[4][4] = {};
+#pragma unroll 2
+                for (int k = 0; k < dim / 32; k++) {
+                    uint32_t b[4], h0[4], h1[4], l0[4], l1[4];
+                    lt_ldmatrix_x4(b, kb + (uint32_t)k * 64u);
+                    lt_ldmatrix_x4(h0, qa + (uint32_t)k * 64u);
+                    lt_ldmatrix_x4(h1, qa + (uint32_t)k * 64u + 32u);
+                    lt_ldmatrix_x4(l0, ql + (uint32_t)k * 64u);
+                    lt_ldmatrix_x4(l1, ql + (uint32_t)k * 64u + 32u);
+                    lt_mma(c[0], h0, b[0], b[1]);
+                    lt_mma(c[1], h1, b[2], b[3]);
+                    lt_mma(c[2], l0, b[0], b[1]);
+                    lt_mma(c[3], l1, b[2], b[3]);
+                }
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    const int j = j0 + fg + 8 * (e >> 1), r = warp * 8 + 2 * tq + (e & 1);
+                    if (j < rep) ss[j * AS_KEYS + r] = r < nk ? ((c[0][e] + c[1][e]) + (c[2][e] + c[3][e])) * a.scale : -INFINITY;
+                }
+            }
+        } else
         for (int i = tid; i < rep * AS_KEYS; i += AS_THREADS) {
             const int r = i % AS_KEYS, j = i / AS_KEYS;
             float s = 0.f;
@@ -281,8 +322,13 @@ __device__ __forceinline__ void attention_step_block(const WindowAttentionArgs &
             const float x0 = ss[j * AS_KEYS + lane], x1 = ss[j * AS_KEYS + lane + 32], old = s_m[j];
             const float m = fmaxf(old, warp_max(fmaxf(x0, x1)));
             const float p0 = expf(x0 - m), p1 = expf(x1 - m), sum = warp_sum(p0 + p1);
-            ss[j * AS_KEYS + lane] = p0;
-            ss[j * AS_KEYS + lane + 32] = p1;
+            if (L.rows) {
+                lt_split_store(phi + j * AS_PE + lane, plo + j * AS_PE + lane, p0);
+                lt_split_store(phi + j * AS_PE + lane + 32, plo + j * AS_PE + lane + 32, p1);
+            } else {
+                ss[j * AS_KEYS + lane] = p0;
+                ss[j * AS_KEYS + lane + 32] = p1;
+            }
             if (lane == 0) {
                 const float c = expf(old - m);
                 s_c[j] = c;
@@ -292,7 +338,35 @@ __device__ __forceinline__ void attention_step_block(const WindowAttentionArgs &
         }
         __syncthreads();
         const int n4 = (nk + 3) / 4;
-        if (vdim % 2 == 0) {
+        if (L.rows) {   // 16 value columns per warp and pass
+            for (int c0 = warp * 16; c0 < vdim; c0 += AS_THREADS / 2)
+                for (int j0 = 0; j0 < L.rows; j0 += 16) {
+                    const uint32_t pa = smem_u32(phi) + ((uint32_t)j0 + a_row) * (AS_PE * 2) + a_col, pl = pa + (uint32_t)(L.rows * AS_PE) * 2u;
+                    const uint32_t vb = smem_u32(sv) + (uint32_t)(((mi & 1) * 8 + mr) * L.vp + c0) * 2u + (uint32_t)(mi >> 1) * 16u;
+                    float o[4][4] = {};
+#pragma unroll
+                    for (int kk = 0; kk < AS_KEYS / 16; kk++) {
+                        uint32_t ph[4], pw[4], b[4];
+                        lt_ldmatrix_x4(ph, pa + (uint32_t)kk * 32u);
+                        lt_ldmatrix_x4(pw, pl + (uint32_t)kk * 32u);
+                        lt_ldmatrix_x4_trans(b, vb + (uint32_t)(kk * 16 * L.vp) * 2u);
+                        lt_mma(o[0], ph, b[0], b[1]);
+                        lt_mma(o[1], ph, b[2], b[3]);
+                        lt_mma(o[2], pw, b[0], b[1]);
+                        lt_mma(o[3], pw, b[2], b[3]);
+                    }
+#pragma unroll
+                    for (int e = 0; e < 4; e++) {
+                        const int j = j0 + fg + 8 * (e >> 1);
+                        if (j >= rep) continue;
+#pragma unroll
+                        for (int n = 0; n < 2; n++) {
+                            float *to = acc + j * vdim + c0 + n * 8 + 2 * tq + (e & 1);
+                            *to = fmaf(*to, s_c[j], o[n][e] + o[n + 2][e]);
+                        }
+                    }
+                }
+        } else if (vdim % 2 == 0) {
             for (int i = tid; i < rep * vdim / 2; i += AS_THREADS) {
                 const int j = i / (vdim / 2), c = i % (vdim / 2) * 2;
                 const float4 *p = reinterpret_cast<const float4 *>(ss + j * AS_KEYS);

@@ -33,6 +33,7 @@ MECHANISMS = {
     "attention_all": (attention_only(size=10 ** 6, kv_heads=1), 72), "attention_64": (attention_only(size=64, dim=64, vdim=64, factor=None), 64),
     "attention_65": (attention_only(size=65, heads=6, kv_heads=3, dim=32, vdim=128, dims=8), 64),
     "attention_no_rotation": (attention_only(size=30, dims=0), 48), "attention_odd": (attention_only(heads=3, kv_heads=1, dim=10, vdim=7, size=33, dims=6), 50),
+    "attention_many": (attention_only(heads=40, kv_heads=2, dim=32, vdim=16, size=90), 64),
     "attention_wide": (attention_only(heads=2, kv_heads=2, dim=288, vdim=264, size=40), 64), "attention_large": (attention_only(heads=4, kv_heads=1, dim=128, vdim=256, size=100, scale=0.1), 64),
     "delta": (delta_only(), 72), "delta_one_tap": (delta_only(conv=1), 72), "delta_two_taps": (delta_only(conv=2, kv_heads=4), 72), "delta_seven_taps": (delta_only(conv=7, kv_heads=1), 64),
     "delta_odd": (delta_only(heads=3, kv_heads=1, dim=9, vdim=5), 50), "delta_64": (delta_only(heads=2, kv_heads=2, dim=64, vdim=48), 64),
