@@ -50,10 +50,9 @@ constexpr int DECAY_EXP = 0, DECAY_SIGMOID_ROOT = 1;
 __device__ __forceinline__ float decay_of(int kind, float x, float inv_tau) {
     return kind == DECAY_SIGMOID_ROOT ? expf((fminf(x, 0.f) - logf(1.0f + expf(-fabsf(x)))) * inv_tau) : expf(-expf(x));
 }
-// The same for tensor-core products, whose operands were rounded to bf16: base-2 exponential and logarithm of the special
-// function unit (absolute error of the logarithm 2^-21).
-__device__ __forceinline__ float decay_of_fast(int kind, float x, float inv_tau) {
-    if (kind != DECAY_SIGMOID_ROOT) return expf(-expf(x));
+// sigmoid(x)^inv_tau for tensor-core products, whose operands were rounded to bf16: the fast exponential and logarithm
+// (absolute error of the logarithm 2^-21).
+__device__ __forceinline__ float sigmoid_root_fast(float x, float inv_tau) {
     return __expf((fminf(x, 0.f) - __logf(1.0f + __expf(-fabsf(x)))) * inv_tau);
 }
 
@@ -317,8 +316,13 @@ dense_gemm_kernel(const __grid_constant__ DenseGemmJobs jobs, const __grid_const
                 if (row < rows) {
                     if (job.decay_bias) {
                         const float b = job.decay_bias[row];
+                        if (job.decay_kind == DECAY_SIGMOID_ROOT) {
 #pragma unroll
-                        for (int i = 0; i < 32; i++) v[i] = __float_as_uint(decay_of_fast(job.decay_kind, __uint_as_float(v[i]) + b, job.inv_tau));
+                            for (int i = 0; i < 32; i++) v[i] = __float_as_uint(sigmoid_root_fast(__uint_as_float(v[i]) + b, job.inv_tau));
+                        } else {
+#pragma unroll
+                            for (int i = 0; i < 32; i++) v[i] = __float_as_uint(expf(-expf(__uint_as_float(v[i]) + b)));
+                        }
                     }
 #pragma unroll
                     for (int i = 0; i < 32; i++) {
