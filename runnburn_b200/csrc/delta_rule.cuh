@@ -434,7 +434,7 @@ delta_prepare_kernel(const __grid_constant__ DeltaArgs a) {
     }
 }
 
-constexpr int DT_STAGES = 4, DT_SPLIT = 2;   // DT_SPLIT: warps that share the channels of 16 value columns
+constexpr int DT_STAGES = 4, DT_SPLIT = 2;   // DT_SPLIT: warps that share the channels of 16 value columns (and the two halves of a tile's tokens)
 struct DeltaTileSmem {
     uint32_t kp, vp, y, v, mat, vec, stage, sums, bytes;
 };
@@ -453,8 +453,8 @@ __host__ __device__ inline DeltaTileSmem delta_tile_smem(int DT, int CW) {
 }
 // grid = (heads, column blocks), blockDim = 32 * (DT_SPLIT * cw + 1): 16 value columns per group of DT_SPLIT warps, each of which
 // holds S^T for its share of the channels; the last warp has a tile's queries and keys, values and record copied into a ring of stages
-// (three bulk copies).  The products with the state are summed over the group through shared memory; its first two warps finish
-// eight of a tile's tokens each.
+// (three bulk copies).  The products with the state are summed over the group through shared memory; each warp finishes eight of a
+// tile's tokens.
 // Waits are bounded; one that gives up sets the error flag, and every copy that was started is waited for before the CTA ends.
 // dim <= 16 DT a multiple of 16, vdim of 8.
 template <int DT>
@@ -612,54 +612,56 @@ delta_tile_kernel(const __grid_constant__ DeltaArgs a) {
             };
             uint32_t hi[4], lo[4];
             split_tile(R, hi, lo);
+            // products that add to the same accumulators lie a few issues apart; the rest of the work fills in
             float W[2][4], W2[2][4];
-            lt_mma_zero(W[0], hi, bh[0], bh[1]);
-            lt_mma_zero(W[1], hi, bh[2], bh[3]);
             lt_mma_zero(W2[0], lo, bh[0], bh[1]);
             lt_mma_zero(W2[1], lo, bh[2], bh[3]);
+            lt_mma_zero(W[0], hi, bh[0], bh[1]);
+            lt_mma_zero(W[1], hi, bh[2], bh[3]);
             lt_mma(W2[0], hi, bl[0], bl[1]);
             lt_mma(W2[1], hi, bl[2], bl[3]);
-            // meanwhile the first two warps' eight tokens of the output
-            float o[4];
-            if (part < 2) {
-                const float4 y = total(2 + part);
-                const float2 f = *reinterpret_cast<const float2 *>(vec + 16 + part * 8 + 2 * tq);
-                o[0] = f.x * y.x, o[1] = f.y * y.y, o[2] = f.x * y.z, o[3] = f.y * y.w;
-                uint32_t q[4];
-                lt_ldmatrix_x4(q, st + b_out);
-                lt_mma(o, hi, q[0], q[1]);
-                lt_mma(o, lo, q[0], q[1]);
-                lt_mma(o, hi, q[2], q[3]);
-            }
+            const float decay = vec[32];
+#pragma unroll
+            for (int n = 0; n < 2 * DW; n++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) S[n][e] *= decay;
+            // the warp's eight tokens of the output
+            const float4 y = total(2 + part);
+            const float2 f = *reinterpret_cast<const float2 *>(vec + 16 + part * 8 + 2 * tq);
+            float o[4] = {f.x * y.x, f.y * y.y, f.x * y.z, f.y * y.w}, o2[4], o3[4];
+            uint32_t q[4], wh[4], wl[4], kb[DW][4];
+            lt_ldmatrix_x4(q, st + b_out);
 #pragma unroll
             for (int n = 0; n < 2; n++)
 #pragma unroll
                 for (int e = 0; e < 4; e++) W[n][e] += W2[n][e];
-            split_tile(W, hi, lo);
-            const float decay = vec[32];
+            split_tile(W, wh, wl);
 #pragma unroll
             for (int np = 0; np < DW; np++) {
-                uint32_t kb[4];
-                lt_ldmatrix_x4_trans(kb, st + L.y + b_trans + (uint32_t)np * 32u);
+                lt_ldmatrix_x4_trans(kb[np], st + L.y + b_trans + (uint32_t)np * 32u);
+                lt_mma(S[2 * np], wh, kb[np][0], kb[np][1]);
+                lt_mma(S[2 * np + 1], wh, kb[np][2], kb[np][3]);
+            }
+            lt_mma(o, hi, q[0], q[1]);
+            lt_mma_zero(o2, lo, q[0], q[1]);
+            lt_mma_zero(o3, hi, q[2], q[3]);
 #pragma unroll
-                for (int e = 0; e < 4; e++) S[2 * np][e] *= decay, S[2 * np + 1][e] *= decay;
-                lt_mma(S[2 * np], hi, kb[0], kb[1]);
-                lt_mma(S[2 * np + 1], hi, kb[2], kb[3]);
-                lt_mma(S[2 * np], lo, kb[0], kb[1]);
-                lt_mma(S[2 * np + 1], lo, kb[2], kb[3]);
+            for (int np = 0; np < DW; np++) {
+                lt_mma(S[2 * np], wl, kb[np][0], kb[np][1]);
+                lt_mma(S[2 * np + 1], wl, kb[np][2], kb[np][3]);
             }
             __syncwarp();
             if (lane == 0) mbar_arrive(&empty[sl]);
-            if (part < 2) {
-                const int t = 16 * it + part * 8 + 2 * tq;
-                if (t < a.tokens) {
-                    if (col0) to[0] = o[0];
-                    if (col1) to[8] = o[2];
-                }
-                if (t + 1 < a.tokens) {
-                    if (col0) to[ldv] = o[1];
-                    if (col1) to[ldv + 8] = o[3];
-                }
+#pragma unroll
+            for (int e = 0; e < 4; e++) o[e] += o2[e] + o3[e];
+            const int t = 16 * it + part * 8 + 2 * tq;
+            if (t < a.tokens) {
+                if (col0) to[0] = o[0];
+                if (col1) to[8] = o[2];
+            }
+            if (t + 1 < a.tokens) {
+                if (col0) to[ldv] = o[1];
+                if (col1) to[ldv + 8] = o[3];
             }
         }
         if (!ok) atomicExch(&s_failed, 1);
